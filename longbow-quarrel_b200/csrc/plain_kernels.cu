@@ -1032,7 +1032,7 @@ rope_partial_kernel(const TI* buf, int stride, TO* qout, int qout_stride, const 
         TO* qd = head < k_first ? qrow + (size_t)head * hd : nullptr;
         TO* kd = (k_pages && head >= k_first) ? k_pages + (at + (size_t)(head - k_first) * page_size) * hd : nullptr;
         const float mul = scaled ? head_mul[head] : 1.f;
-        const float* nw = (unit_norm == 2 && norm_w) ? norm_w + (size_t)head * hd : nullptr;
+        const float* nw = (unit_norm && norm_w) ? norm_w + (size_t)head * hd : nullptr;
         if (j < half) {
             float u = to_f32(p[j]) + (b ? b[j] : 0.f), w = to_f32(p[j + half]) + (b ? b[j + half] : 0.f);
             if (scaled) {
@@ -1160,9 +1160,17 @@ LQ_EXPORT int lq_activation(const void* x, void* out, int dtype, long long total
 
 // out[t, f] = act(gu[t, f] + b[f]) * (gu[t, F + f] + b[F + f]): a gated feed-forward's two halves (gate columns, then up
 // columns) with their biases (float32 [2F], or none), the activation in float32.
+// act 5 clamps both halves: g sigmoid(1.702 g) (u + 1) with g = min(gate, limit), u = clamp(up, -limit, limit).
+__device__ __forceinline__ float gated(float g, float u, int act, float limit) {
+    if (act != 5) return activation(g, act) * u;
+    g = fminf(g, limit);
+    u = fminf(fmaxf(u, -limit), limit);
+    return g / (1.f + expf(-1.702f * g)) * (u + 1.f);
+}
+
 template <typename TI, typename TO>
 __global__ void gated_act_kernel(const TI* __restrict__ gu, const float* __restrict__ bias, TO* __restrict__ out, size_t total,
-                                 int F, int act) {
+                                 int F, int act, float limit) {
     pdl_launch_dependents();
     pdl_wait();
     size_t i = (size_t)blockIdx.x * blockDim.x + threadIdx.x;
@@ -1171,12 +1179,12 @@ __global__ void gated_act_kernel(const TI* __restrict__ gu, const float* __restr
     const int f = i % F;
     float g = to_f32(gu[t * 2 * F + f]), u = to_f32(gu[t * 2 * F + F + f]);
     if (bias) { g += bias[f]; u += bias[F + f]; }
-    out[i] = from_f32<TO>(activation(g, act) * u);
+    out[i] = from_f32<TO>(gated(g, u, act, limit));
 }
 
 // bfloat16 in and out, F a multiple of 8: eight outputs a thread from two 16-byte loads, the same arithmetic.
 __global__ void gated_act_vec_kernel(const uint4* __restrict__ gu, const float* __restrict__ bias, uint4* __restrict__ out,
-                                     size_t total8, int F8, int act) {
+                                     size_t total8, int F8, int act, float limit) {
     pdl_launch_dependents();
     pdl_wait();
     const size_t i = (size_t)blockIdx.x * blockDim.x + threadIdx.x;
@@ -1195,27 +1203,27 @@ __global__ void gated_act_vec_kernel(const uint4* __restrict__ gu, const float* 
             gv.x += bias[f]; gv.y += bias[f + 1];
             uv.x += bias[8 * F8 + f]; uv.y += bias[8 * F8 + f + 1];
         }
-        op[j] = __floats2bfloat162_rn(activation(gv.x, act) * uv.x, activation(gv.y, act) * uv.y);
+        op[j] = __floats2bfloat162_rn(gated(gv.x, uv.x, act, limit), gated(gv.y, uv.y, act, limit));
     }
     out[i] = o;
 }
 
 LQ_EXPORT int lq_gated_act(const void* gu, int in_dtype, const float* bias, void* out, int out_dtype, int T, int F, int act,
-                           cudaStream_t stream) {
+                           float limit, cudaStream_t stream) {
     const size_t total = (size_t)T * F;
     if (total == 0) return LQ_OK;
-    if (act < 0 || act > 4) return LQ_BAD_SIZE;
+    if (act < 0 || act > 5) return LQ_BAD_SIZE;
     if (in_dtype == LQ_BF16 && out_dtype == LQ_BF16 && F % 8 == 0 && (((uintptr_t)gu | (uintptr_t)out) & 15) == 0)
         return launch_pdl(gated_act_vec_kernel, dim3((unsigned)((total / 8 + 255) / 256)), dim3(256), 0, stream, (const uint4*)gu, bias,
-                          (uint4*)out, total / 8, F / 8, act);
+                          (uint4*)out, total / 8, F / 8, act, limit);
     const unsigned blocks = (unsigned)((total + 255) / 256);
     typedef __nv_bfloat16 bf;
     if (in_dtype == LQ_F32 && out_dtype == LQ_F32)
-        return launch_pdl(gated_act_kernel<float, float>, dim3(blocks), dim3(256), 0, stream, (const float*)gu, bias, (float*)out, total, F, act);
+        return launch_pdl(gated_act_kernel<float, float>, dim3(blocks), dim3(256), 0, stream, (const float*)gu, bias, (float*)out, total, F, act, limit);
     if (in_dtype == LQ_F32 && out_dtype == LQ_BF16)
-        return launch_pdl(gated_act_kernel<float, bf>, dim3(blocks), dim3(256), 0, stream, (const float*)gu, bias, (bf*)out, total, F, act);
+        return launch_pdl(gated_act_kernel<float, bf>, dim3(blocks), dim3(256), 0, stream, (const float*)gu, bias, (bf*)out, total, F, act, limit);
     if (in_dtype == LQ_BF16 && out_dtype == LQ_BF16)
-        return launch_pdl(gated_act_kernel<bf, bf>, dim3(blocks), dim3(256), 0, stream, (const bf*)gu, bias, (bf*)out, total, F, act);
+        return launch_pdl(gated_act_kernel<bf, bf>, dim3(blocks), dim3(256), 0, stream, (const bf*)gu, bias, (bf*)out, total, F, act, limit);
     return LQ_BAD_DTYPE;
 }
 

@@ -125,17 +125,19 @@ class Model:
             with linear.recording():
                 return self.forward(ctx, cache)
         states = self._state_entries
-        if "embedding" in states:
+        schedule = self.spec.schedule
+        normed = None           # rows of the next layer's first norm (or the stream itself), when the kernel ahead made them
+        if getattr(self.embedding, "emits_stream", False) and getattr(self.blocks[schedule[0].layer], "reads_stream", False):
+            x, normed = self.embedding.forward(ctx.tokens, emit_stream=True)
+        elif "embedding" in states:
             x = self.embedding.forward(ctx.tokens, ctx=ctx, state=cache.view(states["embedding"][0]))
         else:
             x = self.embedding.forward(ctx.tokens)
-        schedule = self.spec.schedule
         probe = self.probe
         if probe is not None:
             probe(-1, x, ctx)
         # A block that reads the embedding's rows again later (`reads_embedding`) gets a copy: the stream changes in place.
         embedded = x.clone() if self._keeps_embedding else None
-        normed = None           # rows of the next layer's first norm, when this layer's last product made them
         for i, entry in enumerate(schedule):
             block = self.blocks[entry.layer]
             if getattr(block, "replaces_stream", False):
@@ -159,7 +161,8 @@ class Model:
                 continue
             after = self.blocks[schedule[i + 1].layer] if i + 1 < len(schedule) else None
             emit = after.input_norm(x.shape[0]) if getattr(after, "folds_norm", False) else None
-            normed = block.forward(x, ctx, cache.view(entry.cache), entry.writes_cache, normed=normed, emit=emit)
+            more = {"emit_stream": True} if getattr(block, "emits_stream", False) and getattr(after, "reads_stream", False) else {}
+            normed = block.forward(x, ctx, cache.view(entry.cache), entry.writes_cache, normed=normed, emit=emit, **more)
             if probe is not None:
                 probe(i, x, ctx)
         if ctx.want_rows is None or ctx.want_rows.numel() == 0:

@@ -432,6 +432,55 @@ def rmsnorm_add(y: torch.Tensor, gain: torch.Tensor, eps: float, x: torch.Tensor
     return h
 
 
+def embedding_norm(table: torch.Tensor, tokens: torch.Tensor, gain: torch.Tensor, eps: float, rows_dtype: torch.dtype | None = None):
+    """(x, rows): x [T, D] float32 = table[tokens] / rms * gain, and the same numbers in rows_dtype (float32: x itself; None: no rows)."""
+    V, D = table.shape
+    T = tokens.numel()
+    if gain.dtype != torch.float32 or gain.numel() != D or not gain.is_contiguous():
+        raise KernelError("embedding_norm: the gain must be contiguous float32 [D]")
+    x = torch.empty((T, D), dtype=torch.float32, device=table.device)
+    copy = rows_dtype is not None and rows_dtype != torch.float32
+    h = torch.empty((T, D), dtype=rows_dtype, device=table.device) if copy else None
+    fn = _fn("post_norm", "lq_embedding_norm", [c_void_p, c_int, c_void_p, c_void_p, c_float, c_void_p, c_void_p, c_int, c_int, c_int,
+                                                c_int, c_void_p])
+    _check(fn(_p(_contig(table, "table")), dtype_code(table), _p(tokens), _p(gain), float(eps), _p(x), _p(h),
+              dtype_code(h) if copy else F32, T, D, V, _stream()), "embedding_norm")
+    return x, (h if copy else (x if rows_dtype is not None else None))
+
+
+def stream_rows(x: torch.Tensor, out_dtype: torch.dtype) -> torch.Tensor:
+    """The float32 stream x [T, D] in out_dtype (float32: x itself, which changes as branches join it)."""
+    return x if out_dtype == torch.float32 else take_columns(x, 0, x.shape[1], x.shape[1], out_dtype)
+
+
+def join_normed(x: torch.Tensor, branches: tuple, gain: torch.Tensor, eps: float, rows_dtype: torch.dtype | None = None,
+                next_norm: tuple | None = None):
+    """x += y / rms(y) * gain, in place (float32 [T, D]).  branches: ((y, bias),), y float32 [T, D] and bias float32 [D] or None;
+    or two of them that are normed first, ((y1, bias1, w1, m1), (y2, bias2, w2, m2), eps_in): y = m1 (y1 + bias1) / rms * w1 +
+    m2 (y2 + bias2) / rms * w2.  rows_dtype: also returns the rows that the next sublayer reads, the new stream in that dtype
+    (float32: x itself) or, with next_norm = (gain, eps), x / rms(x) * gain."""
+    T, D = x.shape
+    one = len(branches) == 1
+    (y1, b1, w1, m1), (y2, b2, w2, m2), eps_in = ((*branches[0], None, 1.0), (None, None, None, 0.0), 0.0) if one else branches
+    for y in (y1, y2):
+        if y is not None and (y.dtype != torch.float32 or y.shape != x.shape or not y.is_contiguous()):
+            raise KernelError("join_normed: a branch must be contiguous float32 of the stream's shape")
+    if x.dtype != torch.float32 or not x.is_contiguous():
+        raise KernelError("join_normed: the stream must be contiguous float32")
+    next_gain, next_eps = next_norm if next_norm is not None else (None, 0.0)
+    for v in (b1, w1, b2, w2, gain, next_gain):
+        if v is not None and (v.dtype != torch.float32 or v.numel() != D or not v.is_contiguous()):
+            raise KernelError("join_normed: gains and biases must be contiguous float32 [D]")
+    own = rows_dtype is not None and (next_norm is not None or rows_dtype != torch.float32)
+    h = torch.empty((T, D), dtype=rows_dtype, device=x.device) if own else None
+    fn = _fn("post_norm", "lq_join_normed", [c_void_p, c_void_p, c_void_p, c_float, c_void_p, c_void_p, c_void_p, c_float, c_float, c_void_p,
+                                             c_float, c_void_p, c_void_p, c_int, c_void_p, c_float, c_int, c_int, c_void_p])
+    _check(fn(_p(y1), _p(b1), _p(w1), float(m1), _p(y2), _p(b2), _p(w2), float(m2), float(eps_in), _p(gain), float(eps), _p(x), _p(h),
+              dtype_code(h) if own else F32, _p(next_gain), float(next_eps), T, D, _stream()), "join_normed", 1,
+           "join_normed:two" if not one else None)
+    return h if own else (x if rows_dtype is not None else None)
+
+
 def rope_partial(buf: torch.Tensor, bias: torch.Tensor | None, cos, sin, rot: int, tok_pos, tok_seq, slots,
                  page_table, k_pages, v_pages, n_rot: int, k_first: int, Hkv: int, hd: int, vd: int, v_off: int,
                  page_size: int, qout: torch.Tensor | None = None, v_unit_eps: float | None = None,
@@ -444,8 +493,8 @@ def rope_partial(buf: torch.Tensor, bias: torch.Tensor | None, cos, sin, rot: in
     bfloat16 (a product's 32-bit sums, rounded once, after bias and rotation).  v_unit_eps: each value head is divided by
     its root mean square, sqrt(mean(v^2) + v_unit_eps), before it is stored.  unit_norm (32-bit, after the bias and ahead
     of the rotation): "head", every one of the n_rot heads over its own root mean square sqrt(mean(x^2) + norm_eps);
-    "all", the queries over the root mean square of all of them together and the keys likewise, times norm_weight
-    (float32 over the n_rot * hd columns).  q_temp = (coef, every): the queries times 1 + coef ln(floor((p + 1) / every) + 1)."""
+    "all", the queries over the root mean square of all of them together and the keys likewise; either times norm_weight where
+    it is given (float32 over the n_rot * hd columns).  q_temp = (coef, every): the queries times 1 + coef ln(floor((p + 1) / every) + 1)."""
     T = buf.shape[0]
     if buf.stride(1) != 1:
         raise KernelError("rope_partial: rows must be contiguous")
@@ -464,9 +513,9 @@ def rope_partial(buf: torch.Tensor, bias: torch.Tensor | None, cos, sin, rot: in
     if unit_norm not in (None, "head", "all"):
         raise KernelError(f"rope_partial: unit_norm {unit_norm!r} is not one of None, 'head', 'all'")
     mode = {None: 0, "head": 1, "all": 2}[unit_norm]
-    if norm_weight is not None and (mode != 2 or norm_weight.dtype != torch.float32 or norm_weight.numel() != n_rot * hd
+    if norm_weight is not None and (mode == 0 or norm_weight.dtype != torch.float32 or norm_weight.numel() != n_rot * hd
                                     or not norm_weight.is_contiguous()):
-        raise KernelError("rope_partial: the norm's weight goes with unit_norm 'all' and is contiguous float32 over the heads' columns")
+        raise KernelError("rope_partial: the norm's weight goes with unit_norm and is contiguous float32 over the heads' columns")
     if q_temp is not None and not int(q_temp[1]) > 0:
         raise KernelError("rope_partial: the query temperature's step must be positive")
     fn = _fn("plain_kernels", "lq_rope_partial", [c_void_p, c_int, c_int, c_void_p, c_int, c_int, c_void_p, c_void_p, c_void_p,
@@ -482,6 +531,7 @@ def rope_partial(buf: torch.Tensor, bias: torch.Tensor | None, cos, sin, rot: in
 
 
 ACTIVATIONS = {"relu2": 0, "gelu_tanh": 1, "silu": 2, "relu": 3, "gelu": 4}
+GATED = {**ACTIVATIONS, "sigmoid_clamped": 5}       # what `gated_act` makes of a gate and an up half
 
 
 def activation(x: torch.Tensor, kind: str, out: torch.Tensor | None = None) -> torch.Tensor:
@@ -517,17 +567,18 @@ def gate_mul(x: torch.Tensor, gate: torch.Tensor, act: str = "sigmoid", group: i
     return x
 
 
-def gated_act(gu: torch.Tensor, bias: torch.Tensor | None, kind: str, out_dtype: torch.dtype) -> torch.Tensor:
-    """gu [T, 2F] (gate columns, then up columns) -> act(gate + b_gate) * (up + b_up) [T, F]; bias float32 [2F] or None."""
+def gated_act(gu: torch.Tensor, bias: torch.Tensor | None, kind: str, out_dtype: torch.dtype, limit: float = 0.0) -> torch.Tensor:
+    """gu [T, 2F] (gate columns, then up columns) -> act(gate + b_gate) * (up + b_up) [T, F]; bias float32 [2F] or None.
+    "sigmoid_clamped": g sigmoid(1.702 g) (u + 1) with g = min(gate, limit), u = clamp(up, -limit, limit)."""
     T, F2 = gu.shape
     F = F2 // 2
-    if kind not in ACTIVATIONS:
-        raise KernelError(f"activation {kind!r} is not one of {', '.join(ACTIVATIONS)}")
+    if kind not in GATED or (kind == "sigmoid_clamped" and not limit > 0):
+        raise KernelError(f"activation {kind!r} is not one of {', '.join(GATED)} (the clamped one with a limit > 0)")
     if bias is not None and (bias.dtype != torch.float32 or bias.numel() != F2):
         raise KernelError("gated_act: the bias must be float32 [2F]")
     out = torch.empty((T, F), dtype=out_dtype, device=gu.device)
-    fn = _fn("plain_kernels", "lq_gated_act", [c_void_p, c_int, c_void_p, c_void_p, c_int, c_int, c_int, c_int, c_void_p])
-    _check(fn(_p(_contig(gu, "gu")), dtype_code(gu), _p(bias), _p(out), dtype_code(out), T, F, ACTIVATIONS[kind], _stream()), "gated_act")
+    fn = _fn("plain_kernels", "lq_gated_act", [c_void_p, c_int, c_void_p, c_void_p, c_int, c_int, c_int, c_int, c_float, c_void_p])
+    _check(fn(_p(_contig(gu, "gu")), dtype_code(gu), _p(bias), _p(out), dtype_code(out), T, F, GATED[kind], float(limit), _stream()), "gated_act")
     return out
 
 
@@ -923,6 +974,80 @@ def head_norm_gate(raw: torch.Tensor, dv: int, eps: float, out_dtype: torch.dtyp
                                                 c_int, c_int, c_int, c_int, c_float, c_void_p])
     _check(fn(_p(_contig(raw, "raw")), dvx, _p(exp_neg_m), _p(weight), _p(gate), gate.stride(0) if gate is not None else 0,
               GATES[act], _p(out), dtype_code(out_dtype), rows, H, dv, float(eps), _stream()), "head_norm_gate")
+    return out
+
+
+# ------------------------------------------------------------------ gated delta rule
+def take_columns(rows: torch.Tensor, off: int, n: int, width: int, out_dtype: torch.dtype, split: bool = False) -> torch.Tensor:
+    """Columns off .. off + n of float32 rows as [T, width] in out_dtype, zeros behind them.  split (bfloat16): [T, 2 width],
+    every number as two bfloat16 terms, the second `width` columns on: the input of a product whose weight is laid out twice."""
+    T = rows.shape[0]
+    if rows.dtype != torch.float32 or rows.stride(1) != 1 or off + n > rows.shape[1] or n > width:
+        raise KernelError("take_columns: float32 rows that hold the columns")
+    out = torch.empty((T, width * (2 if split else 1)), dtype=out_dtype, device=rows.device)
+    fn = _fn("post_norm", "lq_take_columns", [c_void_p, c_int, c_int, c_int, c_void_p, c_int, c_int, c_int, c_int, c_void_p])
+    _check(fn(_p(rows), rows.stride(0), off, n, _p(out), dtype_code(out_dtype), width, int(split), T, _stream()), "take_columns")
+    return out
+
+
+def _delta_sizes(what: str, rows, b_off, taps_w, ring, z_bias, rate, state, H, G, dk, dv):
+    C, taps = 2 * G * dk + H * dv, taps_w.shape[0]
+    for t, shape, name in ((taps_w, (taps, C), "taps"), (z_bias, (H * dk,), "bias"), (rate, (H,), "rates")):
+        if t.dtype != torch.float32 or tuple(t.shape) != shape or not t.is_contiguous():
+            raise KernelError(f"{what}: the {name} must be contiguous float32 {list(shape)}")
+    for t, shape, name in ((ring, (taps, C), "convolution's state"), (state, (H, dk, dv), "state")):
+        if t.dtype != torch.float32 or tuple(t.shape[1:]) != shape or not t.is_contiguous():
+            raise KernelError(f"{what}: the {name} must be contiguous float32 [slots, {', '.join(map(str, shape))}]")
+    if rows.dtype != torch.float32 or not rows.is_contiguous() or b_off < C or rows.shape[1] < b_off + H:
+        raise KernelError(f"{what}: contiguous float32 rows of q, k, v ({C} columns) and the step sizes")
+    if dk > 256 or H % G:
+        raise KernelError(f"{what}: key size {dk} (at most 256), {H} heads on {G} key heads")
+    return taps
+
+
+def delta_prompt(rows: torch.Tensor, b_off: int, taps_w: torch.Tensor, ring: torch.Tensor, z: torch.Tensor, z_bias: torch.Tensor,
+                 rate: torch.Tensor, state: torch.Tensor, cu_rows, slots, tok_pos, B: int, max_new: int, H: int, G: int, dk: int, dv: int,
+                 q_scale: float, unit_eps: float) -> torch.Tensor:
+    """The gated delta rule over a step's rows (csrc/delta.cu): rows float32 [T, >= C + H], q [G dk], k [G dk], v [H dv] side by
+    side (C columns) and the step sizes' pre-activations [H] at column b_off; taps_w [taps, C]; z [T, H dk] the decays'
+    pre-activations ahead of z_bias, a = exp(-rate_h softplus(z + z_bias)).  state [slots, H, dk, dv] and ring [slots, taps, C]
+    (the convolution's last inputs, position p in row p % taps) are moved on.  Returns S^T q, float32 [T, H, dv]."""
+    taps = _delta_sizes("delta_prompt", rows, b_off, taps_w, ring, z_bias, rate, state, H, G, dk, dv)
+    T = rows.shape[0]
+    if z.dtype != torch.float32 or tuple(z.shape) != (T, H * dk) or not z.is_contiguous():
+        raise KernelError("delta_prompt: z must be contiguous float32 [T, H dk]")
+    size = build.load("delta").lq_delta_record_floats
+    size.argtypes, size.restype = [c_int] * 5, c_longlong
+    records = torch.empty(int(size(T, B, H, dk, dv)), dtype=torch.float32, device=rows.device)
+    raw = torch.empty((T, H, dv), dtype=torch.float32, device=rows.device)
+    fn = _fn("delta", "lq_delta_prompt", [c_void_p, c_int, c_int, c_void_p, c_int, c_void_p, c_void_p, c_void_p, c_void_p, c_void_p, c_void_p,
+                                          c_void_p, c_void_p, c_void_p, c_void_p, c_int, c_int, c_int, c_int, c_int, c_int, c_float, c_float,
+                                          c_void_p])
+    _check(fn(_p(rows), rows.stride(0), b_off, _p(taps_w), taps, _p(ring), _p(z), _p(z_bias), _p(rate), _p(state), _p(cu_rows), _p(slots),
+              _p(tok_pos), _p(records), _p(raw), B, max_new, H, G, dk, dv, float(q_scale), float(unit_eps), _stream()), "delta_prompt", 2)
+    return raw
+
+
+def delta_single(rows: torch.Tensor, b_off: int, taps_w: torch.Tensor, ring: torch.Tensor, z_bias: torch.Tensor, rate: torch.Tensor,
+                 state: torch.Tensor, cu_rows, slots, tok_pos, a_off: int, ra: int, a2: torch.Tensor, g_off: int, rg: int, g2: torch.Tensor,
+                 norm_w: torch.Tensor, norm_eps: float, out_dtype: torch.dtype, B: int, H: int, G: int, dk: int, dv: int, q_scale: float,
+                 unit_eps: float) -> torch.Tensor:
+    """delta_prompt for a step of one token per sequence, with what stands around it: the decays' pre-activations are
+    a2 [H dk, >= ra] times the ra columns of rows at a_off, and each head's output leaves over its root mean square, times
+    norm_w [dv], times sigmoid(g2 [H dv, >= rg] times the rg columns at g_off).  Returns [B, H dv] in out_dtype."""
+    taps = _delta_sizes("delta_single", rows, b_off, taps_w, ring, z_bias, rate, state, H, G, dk, dv)
+    for w, n, r in ((a2, H * dk, ra), (g2, H * dv, rg)):
+        if w.dtype != a2.dtype or w.shape[0] != n or w.shape[1] < r or w.shape[1] % 8 or not w.is_contiguous():
+            raise KernelError("delta_single: the second products' weights must be contiguous, of one dtype, rows in whole eights")
+    if rows.shape[1] < max(a_off + ra, g_off + rg) or norm_w.dtype != torch.float32 or norm_w.numel() != dv:
+        raise KernelError("delta_single: rows with both inner products, a float32 norm weight [dv]")
+    out = torch.empty((rows.shape[0], H * dv), dtype=out_dtype, device=rows.device)
+    fn = _fn("delta", "lq_delta_single", [c_void_p, c_int, c_int, c_void_p, c_int, c_void_p, c_void_p, c_void_p, c_void_p, c_void_p, c_void_p,
+                                          c_void_p, c_int, c_int, c_void_p, c_int, c_int, c_int, c_void_p, c_int, c_int, c_void_p, c_float,
+                                          c_void_p, c_int, c_int, c_int, c_int, c_int, c_int, c_float, c_float, c_void_p])
+    _check(fn(_p(rows), rows.stride(0), b_off, _p(taps_w), taps, _p(ring), _p(z_bias), _p(rate), _p(state), _p(cu_rows), _p(slots),
+              _p(tok_pos), a_off, ra, _p(a2), a2.shape[1], g_off, rg, _p(g2), g2.shape[1], dtype_code(a2), _p(norm_w), float(norm_eps),
+              _p(out), dtype_code(out_dtype), B, H, G, dk, dv, float(q_scale), float(unit_eps), _stream()), "delta_single")
     return out
 
 

@@ -26,8 +26,10 @@ root mean square, sqrt(mean(v^2) + eps), before it is cached); a position part w
 `cache_window` / `cache_keep_first`, what the cache entry keeps when layers that read it see further
 than the layer that writes it (default: the layer's own window and kept positions); `sink="one"` (the
 denominator's one more term is exp(0) = 1 for every head, no tensor); `gate="sigmoid_head"` (one gate per
-head, W_g of H rows: every value of a head times sigmoid of the head's number); `qk_norm` "head" (q and k each
-divided by its root mean square per head, sqrt(mean(x^2) + norm_eps), no weight) or "all" (one norm over the whole
+head, W_g of H rows: every value of a head times sigmoid of the head's number); `out_bias` (the output projection
+with a bias); `qk_norm` "head" (q and k each
+divided by its root mean square per head, sqrt(mean(x^2) + norm_eps), no weight), "head_gain" (the same times a weight of
+the head's size that all heads share, one for q and one for k) or "all" (one norm over the whole
 query projection and one over the whole key projection, each with a weight of that size), in 32-bit on the
 products' 32-bit sums, ahead of the rotation; `q_temp` (coef, every): the queries times
 1 + coef ln(floor((p + 1) / every) + 1) at position p; `chunk` n (instead of a window): position i sees j <= i
@@ -65,7 +67,7 @@ class Attention(Mixer):
                  sink: bool = False, gate: str | None = None, softcap: float | None = None, keep_first: int = 0,
                  value_norm_eps: float | None = None, cache_window: int | None | str = "own",
                  cache_keep_first: int | None = None, qk_norm: str | None = None, norm_eps: float = 0.0,
-                 q_temp: tuple | None = None, chunk: int | None = None):
+                 q_temp: tuple | None = None, chunk: int | None = None, out_bias: bool = False):
         if n_heads % n_kv_heads:
             raise ValueError(f"attention: {n_heads} heads are not a multiple of {n_kv_heads} kv heads")
         if (head_dim % 2 and position is not None) or not 1 <= head_dim <= 256:
@@ -80,8 +82,8 @@ class Attention(Mixer):
             raise ValueError(f"attention: value_dim {self.vd} must be at most 256")
         if gate not in (None, "sigmoid", "sigmoid_head"):
             raise ValueError(f"attention: gate {gate!r} is not supported (supported: 'sigmoid', 'sigmoid_head')")
-        if qk_norm not in (None, "head", "all"):
-            raise ValueError(f"attention: qk_norm {qk_norm!r} is not supported (supported: 'head', 'all')")
+        if qk_norm not in (None, "head", "head_gain", "all"):
+            raise ValueError(f"attention: qk_norm {qk_norm!r} is not supported (supported: 'head', 'head_gain', 'all')")
         if chunk is not None and (window is not None or int(chunk) < 1):
             raise ValueError("attention: blocks of positions (chunk >= 1) or a window, not both")
         if q_temp is not None and not int(q_temp[1]) > 0:
@@ -93,6 +95,7 @@ class Attention(Mixer):
         self.q_temp = (float(q_temp[0]), int(q_temp[1])) if q_temp is not None else None
         self.chunk = int(chunk) if chunk is not None else None
         self.norm_w = None
+        self.out_bias, self.branch_bias = bool(out_bias), None
         self.softcap = float(softcap) if softcap else None
         self.keep_first = int(keep_first or 0) if window is not None else 0
         self.value_norm_eps = None if value_norm_eps is None else float(value_norm_eps)
@@ -101,7 +104,7 @@ class Attention(Mixer):
         if self.cache_window is not None and (window is None or window > self.cache_window or self.keep_first > self.cache_keep_first):
             raise ValueError("attention: the cache entry must keep at least what the layer itself sees")
         self.names = {**DEFAULT_NAMES, **(names or {})}
-        for key in ("q", "k", "v"):
+        for key in ("q", "k", "v", "o"):
             self.names.setdefault(key + "_bias", self.names[key].replace(".weight", "") + ".bias")
         self.names.setdefault("sink", "sinks")
         self.names.setdefault("g", "g_proj.weight")
@@ -111,7 +114,7 @@ class Attention(Mixer):
         self.rot = getattr(self.position, "rotary_dims", head_dim) if self.position is not None else 0
         # The kernels that fuse rotation and cache write into the projections, and the tensor-core attention
         # kernels, know the plain form only; every option above takes the general kernels.
-        self.general = self.bias or self.sink or self.gate is not None or self.vd != head_dim or \
+        self.general = self.bias or self.out_bias or self.sink or self.gate is not None or self.vd != head_dim or \
             (self.position is not None and self.rot != head_dim) or self.softcap is not None or self.keep_first > 0 or \
             self.value_norm_eps is not None or self.qk_norm is not None or self.q_temp is not None or self.chunk is not None
         self.b_qkv = self.sinks = None
@@ -137,14 +140,17 @@ class Attention(Mixer):
             if self.own_kv:
                 out[n["k_bias"]] = WeightSpec((self.Hkv * self.hd,), init="small", full_precision=True)
                 out[n["v_bias"]] = WeightSpec((self.Hkv * self.vd,), init="small", full_precision=True)
+        if self.out_bias:
+            out[n["o_bias"]] = WeightSpec((self.D,), init="small", full_precision=True)
         if self.sink_learned:
             out[n["sink"]] = WeightSpec((self.H,), init=("uniform", 0.0, 4.0), full_precision=True)
         if self.gate is not None:
             out[n["g"]] = WeightSpec((self.H if self.gate_per_head else self.H * self.vd, self.D))
-        if self.qk_norm == "all":
-            out[n["q_norm"]] = WeightSpec((self.H * self.hd,), init="gain", full_precision=True)
+        if self.qk_norm in ("all", "head_gain"):
+            shared = self.qk_norm == "head_gain"          # one weight of the head's size for every head
+            out[n["q_norm"]] = WeightSpec((self.hd if shared else self.H * self.hd,), init="gain", full_precision=True)
             if self.own_kv:
-                out[n["k_norm"]] = WeightSpec((self.Hkv * self.hd,), init="gain", full_precision=True)
+                out[n["k_norm"]] = WeightSpec((self.hd if shared else self.Hkv * self.hd,), init="gain", full_precision=True)
         if self.position is not None:
             out.update(self.position.weights())        # a position encoding may have tensors of its own
         return out
@@ -160,6 +166,10 @@ class Attention(Mixer):
     def load(self, tensors):
         n = self.names
         tensors = dict(tensors)
+        if self.qk_norm == "head_gain":
+            for key, heads in (("q_norm", self.H), ("k_norm", self.Hkv)):
+                if n[key] in tensors:
+                    tensors[n[key]] = tensors[n[key]].repeat(heads)          # the kernels read a weight per column
         for key, heads in (("q", self.H), ("k", self.Hkv)):
             for name in (n[key], n[key + "_bias"], n[key + "_norm"]):
                 if name in tensors and (key == "q" or self.own_kv):
@@ -176,14 +186,16 @@ class Attention(Mixer):
         if self.sink:
             self.sinks = tensors[n["sink"]].to(torch.float32).contiguous() if self.sink_learned else \
                 torch.zeros(self.H, dtype=torch.float32, device=self.runtime.device)
-        if self.qk_norm == "all":
+        if self.out_bias:
+            self.branch_bias = tensors[n["o_bias"]].to(torch.float32).contiguous()
+        if self.qk_norm in ("all", "head_gain"):
             keys = ["q_norm"] + (["k_norm"] if self.own_kv else [])
             self.norm_w = torch.cat([tensors[n[k]].to(torch.float32) for k in keys]).contiguous()
         self.w_o = linear.LinearWeight(tensors[n["o"]])
         if self.position is not None and self.position.weights():
             self.position.load({name: tensors[name] for name in self.position.weights()})
 
-    def _forward_general(self, h, ctx: StepContext, cache_view, residual, store: bool):
+    def _forward_general(self, h, ctx: StepContext, cache_view, residual, store: bool, bias: bool = True):
         """The layer with any of its options: one product for q, k, v and the gate; biases, rotation of
         the rotated dimensions and the cache write in one kernel; attention with the sink in the
         denominator and the gate on the way out; the output projection."""
@@ -203,20 +215,25 @@ class Attention(Mixer):
                          ctx.slots, cache_view.page_table if store else None, cache_view.k_pages if store else None,
                          cache_view.v_pages if store else None, H + (G if self.own_kv else 0), H, G, hd, vd, v_off,
                          cache_view.page_size, qout=q if wide else None, v_unit_eps=self.value_norm_eps,
-                         unit_norm=self.qk_norm, norm_weight=self.norm_w, norm_eps=self.norm_eps, q_temp=self.q_temp)
+                         unit_norm="head" if self.qk_norm == "head_gain" else self.qk_norm, norm_weight=self.norm_w, norm_eps=self.norm_eps, q_temp=self.q_temp)
         g_off = H * hd + (G * (hd + vd) if self.own_kv else 0)
         gate = rows[:, g_off:g_off + (H if self.gate_per_head else H * vd)] if self.gate is not None else None
         out = attention_kernels.attention(q, cache_view, ctx, H, G, hd, self.scale, self.window,
                                           next_w=self.w_o.tensor, vd=vd, sink=self.sinks, gate=gate, softcap=self.softcap,
                                           keep_first=self.keep_first, chunk=self.chunk, gate_per_head=self.gate_per_head)
-        return self._project(out, residual, None)
+        out = self._project(out, residual, None)
+        if self.out_bias and bias:
+            ops.add_bias(out if residual is None else residual, self.branch_bias)
+        return out
 
-    def forward(self, h, ctx: StepContext, cache_view, residual, writes_cache: bool = True, emit=None):
+    takes_bias_later = True       # forward(bias=False) leaves `branch_bias` to the kernel that takes the branch
+
+    def forward(self, h, ctx: StepContext, cache_view, residual, writes_cache: bool = True, emit=None, bias: bool = True):
         store = self.own_kv and writes_cache
         if self.own_kv and not store:
             raise ValueError("attention: a layer with its own k and v must write its cache entry")
         if self.general:
-            return self._forward_general(h, ctx, cache_view, residual, store)
+            return self._forward_general(h, ctx, cache_view, residual, store, bias)
         tables = self.position.tables() if self.position is not None else None
         fused = (store and h.dtype == torch.bfloat16 and self.w_qkv.tensor.dtype == torch.bfloat16 and self.D % 8 == 0
                  and self.hd % 16 == 0 and cache_view.k_pages.dtype == torch.bfloat16 and (self.position is None or tables is not None))

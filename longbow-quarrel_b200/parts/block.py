@@ -13,6 +13,10 @@ the mixer and the feed-forward hand back their branches as float32 rows.
 "stream_mix": no mixer and no feed-forward; the stream is replaced by a product over the stream and the embedding's
 rows side by side, x <- W [x; e] (what a pass over repeated layers starts with).
 
+"post_norm": the sublayers read the stream itself and what they return is normed, x += norm1(mixer(x));
+x += norm2(ffn(x)), a layer may have no feed-forward.  The branch's norm (and, for a mixer of two sides whose outputs are
+normed first, theirs and the sum), the addition and the rows that the next sublayer reads are one kernel.
+
 "sandwich_norm": every branch is normed on both sides, x += norm1b(mixer(norm1(x)));
 x += norm2b(ffn(norm2(x))), and a layer may have no feed-forward.  The branch's own norm,
 the addition and the norm that reads the stream next are one kernel."""
@@ -124,7 +128,7 @@ class PreNormBlock(Part):
             return self._forward_plain(x, ctx, cache_view, writes_cache, state)
         n_rows = x.shape[0]
         h = normed if normed is not None else self.norm1.forward(x)
-        if self.has_ffn and hasattr(self.mixer, "branches") and getattr(self.norm2, "takes_branches", False):
+        if self.has_ffn and getattr(self.mixer, "branches", None) is not None and getattr(self.norm2, "takes_branches", False):
             # A mixer of several sides: its branches join the stream in the kernel that makes the second norm's rows.
             h = self.norm2.forward(x, add=self.mixer.branches(h, ctx, cache_view, writes_cache))
             self.ffn.forward(h, ctx, x)
@@ -223,6 +227,85 @@ class SandwichNormBlock(Part):
         h = ops.rmsnorm_add(y, self.norm1b.gain, self.norm1b.eps, x, (self.norm2.gain, self.norm2.eps), act)
         y = self.ffn.forward(h, ctx, None)
         return ops.rmsnorm_add(y, self.norm2b.gain, self.norm2b.eps, x, emit, act)
+
+
+@register_part("block", "post_norm")
+class PostNormBlock(Part):
+    """Places: mixer, norm1, and (both or neither) ffn, norm2; the norms are RMS norms.  The mixer and the feed-forward hand
+    back their outputs as float32 rows (`returns_branch`, or `normed_branches` for a mixer of two normed sides)."""
+
+    folds_norm = True
+    reads_stream = True          # the rows it starts with are the stream itself, in the activations' dtype
+    emits_stream = True          # forward(emit_stream=True) returns such rows for the layer that follows
+    kernel_libraries = ("post_norm",)
+
+    def __init__(self, runtime: Runtime, layer: LayerSpec):
+        self.prefix, self.runtime = layer.prefix, runtime
+        places = set(layer.parts)
+        unknown = places - {"mixer", "norm1", "ffn", "norm2"}
+        if unknown:
+            raise ValueError(f"layer {layer.prefix!r}: the arrangement 'post_norm' has no place {sorted(unknown)}")
+        if len(places & {"norm2", "ffn"}) == 1:
+            raise ValueError(f"layer {layer.prefix!r}: norm2 and ffn come together or not at all")
+        self.mixer = make_part("mixer", layer.part("mixer"), runtime)
+        self.norm1 = make_part("norm", layer.part("norm1"), runtime)
+        self.has_ffn = "ffn" in places
+        self.ffn = make_part("ffn", layer.part("ffn"), runtime) if self.has_ffn else None
+        self.norm2 = make_part("norm", layer.part("norm2"), runtime) if self.has_ffn else None
+        if not getattr(self.mixer, "returns_branch", False):
+            raise ValueError(f"layer {layer.prefix!r}: the mixer {layer.part('mixer').kind!r} cannot hand back its output for a "
+                             f"norm of its own")
+        for norm in (self.norm1, self.norm2):
+            if norm is not None and not isinstance(norm, RMSNorm):
+                raise ValueError(f"layer {layer.prefix!r}: the arrangement 'post_norm' needs RMS norms with a gain")
+
+    def parts(self):
+        return tuple(p for p in (self.mixer, self.norm1, self.ffn, self.norm2) if p is not None)
+
+    def cache_need(self):
+        return self.mixer.cache_need()
+
+    def step_needs(self):
+        out = {}
+        for part in self.parts():
+            out.update(part.step_needs())
+        return out
+
+    @property
+    def graph_safe(self):
+        return all(p.graph_safe for p in self.parts())
+
+    def weights(self):
+        out = {}
+        for part in self.parts():
+            for name, spec in part.weights().items():
+                if name in out:
+                    raise ValueError(f"layer {self.prefix}: two parts name the tensor {name!r}")
+                out[name] = spec
+        return out
+
+    def load(self, tensors):
+        for part in self.parts():
+            part.load({n: tensors[n] for n in part.weights()})
+
+    def input_norm(self, n_rows: int):
+        return None              # the layer reads the stream itself
+
+    def forward(self, x, ctx: StepContext, cache_view, writes_cache: bool = True, normed=None, emit=None, emit_stream: bool = False):
+        """`normed`: the stream in the activations' dtype when the kernel ahead left it; `emit`: the next layer's input_norm();
+        `emit_stream`: the next layer reads the stream itself.  Returns the next layer's rows, or None."""
+        act = self.runtime.act_dtype
+        h = normed if normed is not None else ops.stream_rows(x, act)
+        rows = act if emit is not None or emit_stream else None
+        if getattr(self.mixer, "out_norms", None) is not None:
+            branches = self.mixer.normed_branches(h, ctx, cache_view, writes_cache)
+        else:
+            branches = ((self.mixer.forward(h, ctx, cache_view, None, writes_cache), None),)
+        if not self.has_ffn:
+            return ops.join_normed(x, branches, self.norm1.gain, self.norm1.eps, rows, emit)
+        h = ops.join_normed(x, branches, self.norm1.gain, self.norm1.eps, act)
+        y = self.ffn.forward(h, ctx, None)
+        return ops.join_normed(x, ((y, None),), self.norm2.gain, self.norm2.eps, rows, emit)
 
 
 @register_part("block", "stream_mix")

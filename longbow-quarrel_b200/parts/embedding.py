@@ -13,25 +13,40 @@ import torch
 from ..kernels import linear, ops
 from ..weights.spec import WeightSpec
 from .base import Part, Runtime, StateNeed
-from .registry import register_part
+from .registry import make_part, register_part
+from .spec import PartSpec
 
 
 @register_part("embedding", "token_embedding")
 class TokenEmbedding(Part):
     graph_safe = True
 
-    def __init__(self, runtime: Runtime, vocab_size: int, hidden_size: int, name: str):
+    def __init__(self, runtime: Runtime, vocab_size: int, hidden_size: int, name: str, norm: PartSpec | None = None):
+        """norm: an RMS norm with a gain that the rows pass before they become the stream."""
         self.runtime, self.vocab_size, self.hidden_size, self.name = runtime, vocab_size, hidden_size, name
+        self.norm = make_part("norm", norm, runtime) if norm is not None else None
+        if self.norm is not None and not (hasattr(self.norm, "gain") and hasattr(self.norm, "eps") and not hasattr(self.norm, "bias")):
+            raise ValueError("token_embedding: the rows' norm must be an RMS norm with a gain")
+        self.emits_stream = self.norm is not None      # forward(emit_stream=True) also returns the rows in the activations' dtype
+        self.kernel_libraries = ("post_norm",) if self.norm is not None else ()
         self.table: torch.Tensor | None = None
 
     def weights(self):
-        return {self.name: WeightSpec((self.vocab_size, self.hidden_size))}
+        out = {self.name: WeightSpec((self.vocab_size, self.hidden_size))}
+        if self.norm is not None:
+            out.update(self.norm.weights())
+        return out
 
     def load(self, tensors):
         self.table = tensors[self.name]
+        if self.norm is not None:
+            self.norm.load({n: tensors[n] for n in self.norm.weights()})
 
-    def forward(self, tokens: torch.Tensor) -> torch.Tensor:
-        return ops.embedding(self.table, tokens)
+    def forward(self, tokens: torch.Tensor, emit_stream: bool = False):
+        if self.norm is None:
+            return ops.embedding(self.table, tokens)
+        x, rows = ops.embedding_norm(self.table, tokens, self.norm.gain, self.norm.eps, self.runtime.act_dtype if emit_stream else None)
+        return (x, rows) if emit_stream else x
 
 
 @register_part("embedding", "pair_hash_embedding")

@@ -2,7 +2,8 @@
 (internal/device/metal.go:1464-1474; internal/device/cpu_ref.go:133-149 CPUSwiGLU).
 Gate and up are one matrix product over the stacked weight [2F, D].
 
-Options that other designs use: `activation` "gelu_tanh" or "gelu" (the erf form) instead of "silu", and
+Options that other designs use: `activation` "gelu_tanh" or "gelu" (the erf form) instead of "silu", or "sigmoid_clamped" with
+a `limit` m (y = W_down (g sigmoid(1.702 g) (u + 1)), g = min(W_gate h, m), u = clamp(W_up h, -m, m)), and
 `bias` (each of the three projections with a bias: y = W_down (act(W_gate h + b_g) * (W_up h + b_u)) + b_d).
 With either the activation is a kernel of its own behind the product (whose sums it reads in 32-bit where
 biases are added); the fused SwiGLU epilogues serve the plain form."""
@@ -23,9 +24,12 @@ class GatedMLP(FeedForward):
     graph_safe = True
 
     def __init__(self, runtime: Runtime, hidden_size: int, intermediate_size: int, activation: str = "silu",
-                 names: dict | None = None, bias: bool = False):
-        if activation not in ("silu", "gelu_tanh", "gelu"):
-            raise ValueError(f"gated_mlp: activation {activation!r} is not supported (supported: 'silu', 'gelu_tanh', 'gelu')")
+                 names: dict | None = None, bias: bool = False, limit: float | None = None):
+        if activation not in ("silu", "gelu_tanh", "gelu", "sigmoid_clamped"):
+            raise ValueError(f"gated_mlp: activation {activation!r} is not supported (supported: 'silu', 'gelu_tanh', 'gelu', 'sigmoid_clamped')")
+        if (activation == "sigmoid_clamped") != (limit is not None) or (limit is not None and not limit > 0):
+            raise ValueError("gated_mlp: the activation 'sigmoid_clamped' comes with a limit > 0, the others without")
+        self.limit = float(limit or 0.0)
         self.runtime, self.D, self.F = runtime, hidden_size, intermediate_size
         self.activation, self.bias = activation, bool(bias)
         self.plain = activation == "silu" and not self.bias
@@ -69,12 +73,12 @@ class GatedMLP(FeedForward):
             if self.plain:
                 return linear.linear(linear.linear_swiglu(h, self.w_gu, self.block), self.w_down, torch.float32)
             gu = linear.linear(h, self.w_gu, torch.float32 if self.bias else self.runtime.act_dtype)
-            out = linear.linear(ops.gated_act(gu, self.b_gu, self.activation, self.runtime.act_dtype), self.w_down, torch.float32)
+            out = linear.linear(ops.gated_act(gu, self.b_gu, self.activation, self.runtime.act_dtype, self.limit), self.w_down, torch.float32)
             return ops.add_bias(out, self.b_down) if self.bias else out
         if not self.plain:
             # Biases meet the product's 32-bit sums before anything is rounded.
             gu = linear.linear(h, self.w_gu, torch.float32 if self.bias else self.runtime.act_dtype)
-            act = ops.gated_act(gu, self.b_gu, self.activation, self.runtime.act_dtype)
+            act = ops.gated_act(gu, self.b_gu, self.activation, self.runtime.act_dtype, self.limit)
             linear.linear(act, self.w_down, self.runtime.act_dtype, residual=residual)
             if self.bias:
                 ops.add_bias(residual, self.b_down)

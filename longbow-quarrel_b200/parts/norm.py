@@ -16,12 +16,14 @@ class RMSNorm(Norm):
     graph_safe = True
 
     def __init__(self, runtime: Runtime, size: int, eps: float, name: str = "weight", offset: float = 0.0,
-                 scalar: bool = False):
+                 scalar: bool = False, multiplier: float = 1.0):
         """offset: what is added to the stored tensor to give the gain (1 for checkpoints that keep their
         gains minus one: y = x / rms(x) * (1 + w)); the sum is made once, in 32-bit, when the tensor is loaded.
-        scalar: the stored gain is one number (a tensor without dimensions) that serves every coordinate."""
+        scalar: the stored gain is one number (a tensor without dimensions) that serves every coordinate.
+        multiplier: the gain is multiplied by this constant, once, in 32-bit (a factor on what the norm feeds, such as
+        the logits' of the final norm)."""
         self.runtime, self.size, self.eps, self.name, self.offset = runtime, size, float(eps), name, float(offset)
-        self.scalar = bool(scalar)
+        self.scalar, self.multiplier = bool(scalar), float(multiplier)
         self.gain: torch.Tensor | None = None
 
     def weights(self):
@@ -29,7 +31,7 @@ class RMSNorm(Norm):
         return {self.name: WeightSpec(shape, init="gain" if self.offset == 0.0 else "small", full_precision=True)}
 
     def load(self, tensors):
-        gain = tensors[self.name].to(torch.float32) + self.offset
+        gain = (tensors[self.name].to(torch.float32) + self.offset) * self.multiplier
         # One number for all coordinates is kept as a row of equal gains: every kernel that reads gains takes it as it is.
         self.gain = (gain.reshape(1).expand(self.size) if self.scalar else gain).contiguous()
 
