@@ -30,7 +30,8 @@ namespace {
 
 constexpr int DW = 8;            // warps per block
 constexpr int TILE = 16;         // keys per warp tile
-constexpr int RING = 3;          // tiles of a warp in shared memory: one in use, two on their way
+// Tiles of a warp in shared memory: one in use, the others on their way (two; one where wide values leave no room).
+constexpr int ring_tiles(int VD) { return VD <= 128 ? 3 : 2; }
 constexpr int PAD = 8;           // elements of padding per shared-memory row (ldmatrix without bank conflicts)
 constexpr int MAX_SPLITS = 32;   // most slices a sequence's keys are cut into
 
@@ -70,23 +71,25 @@ __device__ __forceinline__ float tanh_fast(float x) {
     return fmaf(-2.0f, r, 1.0f);
 }
 
-template <int HD>
-__global__ void __launch_bounds__(DW * 32, HD <= 64 ? 2 : 1)
+// VD: a value head's size rounded up; its real size vd may be another than hd.
+template <int HD, int VD>
+__global__ void __launch_bounds__(DW * 32, HD <= 64 && VD <= 64 ? 2 : 1)
 attn_decode_kernel(const __nv_bfloat16* __restrict__ q, int q_stride, const __nv_bfloat16* __restrict__ k_pages,
                    const __nv_bfloat16* __restrict__ v_pages, const int* __restrict__ page_table, int pt_stride,
                    const int* __restrict__ tok_pos, const int* __restrict__ tok_seq, const int* __restrict__ slots,
                    float* __restrict__ part_o, float* __restrict__ part_ml, int* __restrict__ counters,
                    __nv_bfloat16* __restrict__ out, int H, int Hkv, int hd, int page_size, float scale, int window,
                    int n_splits, int part_stride, const int* __restrict__ work, const char* next_w, unsigned next_piece,
-                   int early_loads, const float* __restrict__ sink, float softcap, int keep_first) {
-    constexpr int LD = HD + PAD;                   // shared-memory row length in elements
+                   int early_loads, const float* __restrict__ sink, float softcap, int keep_first, int vd) {
+    constexpr int LD = HD + PAD, LV = VD + PAD;    // shared-memory row lengths in elements: keys, values
+    constexpr int RING = ring_tiles(VD);
     constexpr int KD = HD / 16;                    // k16 steps over the head dimension
-    constexpr int STAGE = 2 * TILE * LD;           // elements of one tile: K rows, then V rows
+    constexpr int STAGE = TILE * (LD + LV);        // elements of one tile: K rows, then V rows
     extern __shared__ __align__(16) uint8_t smem_raw[];
     __nv_bfloat16* ring = reinterpret_cast<__nv_bfloat16*>(smem_raw);            // [DW][RING][STAGE]
     // After the loop the same memory holds each warp's state for the merge.
-    float (*sm_o)[16][HD + 1] = reinterpret_cast<float (*)[16][HD + 1]>(smem_raw);
-    float (*sm_m)[16] = reinterpret_cast<float (*)[16]>(smem_raw + sizeof(float) * DW * 16 * (HD + 1));
+    float (*sm_o)[16][VD + 1] = reinterpret_cast<float (*)[16][VD + 1]>(smem_raw);
+    float (*sm_m)[16] = reinterpret_cast<float (*)[16]>(smem_raw + sizeof(float) * DW * 16 * (VD + 1));
     float (*sm_l)[16] = sm_m + DW;
     __shared__ float sm_w[16][MAX_SPLITS];       // weights of the slices when this block merges them
     __shared__ float sm_inv[16];
@@ -107,7 +110,7 @@ attn_decode_kernel(const __nv_bfloat16* __restrict__ q, int q_stride, const __nv
         seg_end = work[blockIdx.y + 1];
         segments = work + gridDim.y + 1;
     }
-    const size_t head_off = (size_t)kvh * page_size * hd;
+    const size_t head_off = (size_t)kvh * page_size;
     __nv_bfloat16* my_ring = ring + (size_t)warp * RING * STAGE;
     // No pdl_launch_dependents() here: released early, the blocks of the product that follows moved
     // onto the SMs this kernel leaves free and fetched weights against it (measured: the step ran
@@ -157,7 +160,8 @@ attn_decode_kernel(const __nv_bfloat16* __restrict__ q, int q_stride, const __nv
         if (v < tile_hi) {
             const int kb = tile_of(v) * TILE;
             const int page = pt[kb / page_size];
-            const size_t off = (size_t)page * Hkv * page_size * hd + head_off + (size_t)(kb % page_size) * hd;
+            const size_t first_row = (size_t)page * Hkv * page_size + head_off + kb % page_size;
+            const size_t off = first_row * hd, voff = first_row * vd;
             __nv_bfloat16* ks = my_ring + (size_t)(n % RING) * STAGE;
             __nv_bfloat16* vs = ks + TILE * LD;
             for (int i = lane; i < TILE * (HD / 8); i += 32) {
@@ -165,7 +169,16 @@ attn_decode_kernel(const __nv_bfloat16* __restrict__ q, int q_stride, const __nv
                 const bool ok = kb + r < len && c < hd;
                 const size_t src = off + (size_t)(ok ? r : 0) * hd + (ok ? c : 0);
                 cp_async16((uint32_t)__cvta_generic_to_shared(ks + r * LD + c), k_pages + src, ok);
-                cp_async16((uint32_t)__cvta_generic_to_shared(vs + r * LD + c), v_pages + src, ok);
+                if constexpr (HD == VD) {
+                    if (vd == hd) cp_async16((uint32_t)__cvta_generic_to_shared(vs + r * LV + c), v_pages + (src - off) + voff, ok);
+                }
+            }
+            if (HD != VD || vd != hd) {
+                for (int i = lane; i < TILE * (VD / 8); i += 32) {
+                    const int r = i / (VD / 8), c = (i % (VD / 8)) * 8;
+                    const bool ok = kb + r < len && c < vd;
+                    cp_async16((uint32_t)__cvta_generic_to_shared(vs + r * LV + c), v_pages + voff + (size_t)(ok ? r : 0) * vd + (ok ? c : 0), ok);
+                }
             }
         }
         cp_async_commit();          // an empty group when there is no tile: the count of groups stays in step
@@ -203,9 +216,9 @@ attn_decode_kernel(const __nv_bfloat16* __restrict__ q, int q_stride, const __nv
         qf[kk][3] = (r1ok && d1 < hd) ? *reinterpret_cast<const uint32_t*>(q1p + d1) : 0u;
     }
 
-    float o[HD / 8][4];
+    float o[VD / 8][4];
 #pragma unroll
-    for (int j = 0; j < HD / 8; ++j)
+    for (int j = 0; j < VD / 8; ++j)
 #pragma unroll
         for (int i = 0; i < 4; ++i) o[j][i] = 0.f;
     float m0 = -CUDART_INF_F, m1 = -CUDART_INF_F, l0 = 0.f, l1 = 0.f;
@@ -277,11 +290,11 @@ attn_decode_kernel(const __nv_bfloat16* __restrict__ q, int q_stride, const __nv
         l0 = l0 * c0 + ps0;
         l1 = l1 * c1 + ps1;
 #pragma unroll
-        for (int dp = 0; dp < HD / 16; ++dp) {
+        for (int dp = 0; dp < VD / 16; ++dp) {
             // V transposed on load: matrices (keys 0-7, d 0-7), (keys 8-15, d 0-7), (keys 0-7, d 8-15), (keys 8-15, d 8-15)
             const int r = (lane & 7) + ((lane >> 3) & 1) * 8, c = dp * 16 + (lane >> 4) * 8;
             uint32_t b0, b1, b2, b3;
-            ldsm_x4_t((uint32_t)__cvta_generic_to_shared(vs + r * LD + c), b0, b1, b2, b3);
+            ldsm_x4_t((uint32_t)__cvta_generic_to_shared(vs + r * LV + c), b0, b1, b2, b3);
             float (&oa)[4] = o[2 * dp];
             float (&ob)[4] = o[2 * dp + 1];
             oa[0] *= c0; oa[1] *= c0; oa[2] *= c1; oa[3] *= c1;
@@ -305,7 +318,7 @@ attn_decode_kernel(const __nv_bfloat16* __restrict__ q, int q_stride, const __nv
     l1 += __shfl_xor_sync(0xffffffffu, l1, 2);
     __syncthreads();        // all rings are idle: their memory now holds the warps' states
 #pragma unroll
-    for (int j = 0; j < HD / 8; ++j) {
+    for (int j = 0; j < VD / 8; ++j) {
         const int d = j * 8 + 2 * t;
         sm_o[warp][g][d] = o[j][0];
         sm_o[warp][g][d + 1] = o[j][1];
@@ -318,8 +331,8 @@ attn_decode_kernel(const __nv_bfloat16* __restrict__ q, int q_stride, const __nv
     }
     __syncthreads();
     const int rows = min(16, G - gt * 16);
-    for (int i = threadIdx.x; i < rows * hd; i += DW * 32) {
-        int r = i / hd, d = i % hd;
+    for (int i = threadIdx.x; i < rows * vd; i += DW * 32) {
+        int r = i / vd, d = i % vd;
         float mx = -CUDART_INF_F;
 #pragma unroll
         for (int w = 0; w < DW; ++w) mx = fmaxf(mx, sm_m[w][r]);
@@ -336,10 +349,10 @@ attn_decode_kernel(const __nv_bfloat16* __restrict__ q, int q_stride, const __nv
         if (parts == 1) {
             // sink (optional): one more term exp(sink[h]) in the head's denominator, with no key and no value
             if (sink) l += expf(sink[h] - mx);
-            out[((size_t)tok * H + h) * hd + d] = __float2bfloat16_rn(acc / l);
+            out[((size_t)tok * H + h) * vd + d] = __float2bfloat16_rn(acc / l);
         } else {
             size_t base = ((size_t)tok * H + h) * part_stride + split;
-            part_o[base * hd + d] = acc;
+            part_o[base * vd + d] = acc;
             if (d == 0) { part_ml[base * 2] = mx; part_ml[base * 2 + 1] = l; }
         }
     }
@@ -370,14 +383,14 @@ attn_decode_kernel(const __nv_bfloat16* __restrict__ q, int q_stride, const __nv
         if (lane == 0) sm_inv[r] = 1.0f / l;
     }
     __syncthreads();
-    for (int i = threadIdx.x; i < rows * hd; i += DW * 32) {
-        const int r = i / hd, d = i % hd;
+    for (int i = threadIdx.x; i < rows * vd; i += DW * 32) {
+        const int r = i / vd, d = i % vd;
         const int h = kvh * G + gt * 16 + r;
-        const float* po = part_o + ((size_t)tok * H + h) * part_stride * hd + d;
+        const float* po = part_o + ((size_t)tok * H + h) * part_stride * vd + d;
         float acc = 0.f;
 #pragma unroll 8
-        for (int s2 = 0; s2 < parts; ++s2) acc += __ldcg(po + (size_t)s2 * hd) * sm_w[r][s2];
-        out[((size_t)tok * H + h) * hd + d] = __float2bfloat16_rn(acc * sm_inv[r]);
+        for (int s2 = 0; s2 < parts; ++s2) acc += __ldcg(po + (size_t)s2 * vd) * sm_w[r][s2];
+        out[((size_t)tok * H + h) * vd + d] = __float2bfloat16_rn(acc * sm_inv[r]);
     }
     }   // segments
 }
@@ -412,12 +425,12 @@ __global__ void attn_merge_kernel(const float* __restrict__ part_o, const float*
     }
 }
 
-template <int HD>
+template <int HD, int VD>
 int launch(const void* q, int q_stride, const void* k_pages, const void* v_pages, const int* page_table, int pt_stride,
            const int* tok_pos, const int* tok_seq, const int* slots, float* part_o, float* part_ml, int* counters,
            void* out, int T, int H, int Hkv, int hd, int page_size, float scale, int window, int n_splits,
            const int* work, int teams, const void* next_w, long next_bytes, int early_loads, const float* sink,
-           float softcap, int keep_first, cudaStream_t stream) {
+           float softcap, int keep_first, int vd, cudaStream_t stream) {
     int G = H / Hkv, gtiles = (G + 15) / 16;
     dim3 grid(n_splits, Hkv * gtiles, T);
     if (work) grid = dim3(Hkv * gtiles, teams, 1);      // n_splits is then the room for parts per token in the scratch
@@ -425,22 +438,22 @@ int launch(const void* q, int q_stride, const void* k_pages, const void* v_pages
     long piece = (next_w && !((uintptr_t)next_w & 15)) ? next_bytes / n_blocks / 16 * 16 : 0;
     if (piece > (1 << 20)) piece = 1 << 20;
     if (piece <= 0) next_w = nullptr;
-    constexpr size_t ring = (size_t)DW * RING * 2 * TILE * (HD + PAD) * 2;
-    constexpr size_t merge = sizeof(float) * DW * 16 * (HD + 1) + sizeof(float) * 2 * DW * 16;
+    constexpr size_t ring = (size_t)DW * ring_tiles(VD) * TILE * (HD + VD + 2 * PAD) * 2;
+    constexpr size_t merge = sizeof(float) * DW * 16 * (VD + 1) + sizeof(float) * 2 * DW * 16;
     constexpr size_t smem = ring > merge ? ring : merge;
     static bool configured = false;
     if (!configured) {
-        if (cudaFuncSetAttribute(attn_decode_kernel<HD>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem) != cudaSuccess)
+        if (cudaFuncSetAttribute(attn_decode_kernel<HD, VD>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem) != cudaSuccess)
             return lq_launch_status();
         configured = true;
     }
-    int rc = launch_pdl(attn_decode_kernel<HD>, grid, dim3(DW * 32), smem, stream, (const __nv_bfloat16*)q, q_stride,
+    int rc = launch_pdl(attn_decode_kernel<HD, VD>, grid, dim3(DW * 32), smem, stream, (const __nv_bfloat16*)q, q_stride,
         (const __nv_bfloat16*)k_pages, (const __nv_bfloat16*)v_pages, page_table, pt_stride, tok_pos, tok_seq, slots,
         part_o, part_ml, counters, (__nv_bfloat16*)out, H, Hkv, hd, page_size, scale, window, n_splits, n_splits, work,
-        (const char*)next_w, (unsigned)piece, early_loads, sink, softcap, keep_first);
+        (const char*)next_w, (unsigned)piece, early_loads, sink, softcap, keep_first, vd);
     if (rc != LQ_OK || n_splits == 1 || counters != nullptr) return rc;
     return launch_pdl(attn_merge_kernel, dim3(T * H), dim3(128), 0, stream, (const float*)part_o, (const float*)part_ml,
-                      (__nv_bfloat16*)out, hd, n_splits, H, sink);
+                      (__nv_bfloat16*)out, vd, n_splits, H, sink);
 }
 
 }  // namespace
@@ -475,24 +488,40 @@ bool sizes_ok(int H, int Hkv, int hd, int page_size, int q_stride, int n_splits)
 // softcap c (0: none): score <- c tanh(score / c) after the scale.  keep_first n (0: none; with a window): a
 // token's first n keys stay visible when its window has moved past them; the tiles of a token are then counted
 // through the kept tiles ahead of the window and then the window's (a work list's tile ranges are such counts).
+//
+// vd: the size of a value head (a multiple of 8, at most 256), where it is another than hd; out is [T, H*vd] and the
+// scratch holds rows of vd.
+LQ_EXPORT int lq_attn_decode_vd(const void* q, int q_stride, const void* k_pages, const void* v_pages,
+                                const int* page_table, int pt_stride, const int* tok_pos, const int* tok_seq,
+                                const int* slots, float* part_o, float* part_ml, int* counters, void* out, int T,
+                                int H, int Hkv, int hd, int vd, int page_size, float scale, int window, int n_splits,
+                                const int* work, int teams, const void* next_w, long next_bytes, int early_loads,
+                                const float* sink, float softcap, int keep_first, cudaStream_t stream) {
+    if (T <= 0) return LQ_OK;
+    if (!sizes_ok(H, Hkv, hd, page_size, q_stride, n_splits) || vd <= 0 || vd % 8 || vd > 256) return LQ_BAD_SIZE;
+    if (n_splits > 1 && (!part_o || !part_ml)) return LQ_BAD_SIZE;
+    if (work && (teams < 1 || teams > 65535 || (n_splits > 1 && !counters))) return LQ_BAD_SIZE;
+    if (softcap < 0.f || keep_first < 0) return LQ_BAD_SIZE;
+#define LQ_GO(HD, VD) return launch<HD, VD>(q, q_stride, k_pages, v_pages, page_table, pt_stride, tok_pos, tok_seq, slots, \
+                                            part_o, part_ml, counters, out, T, H, Hkv, hd, page_size, scale, window, n_splits, \
+                                            work, teams, next_w, next_bytes, early_loads, sink, softcap, keep_first, vd, stream)
+    if (vd > 128) LQ_GO(128, 256);
+    if (hd <= 32 && vd <= 32) LQ_GO(32, 32);
+    if (hd <= 64 && vd <= 64) LQ_GO(64, 64);
+    if (hd <= 64) LQ_GO(64, 128);
+    LQ_GO(128, 128);
+#undef LQ_GO
+}
+
 LQ_EXPORT int lq_attn_decode_capped(const void* q, int q_stride, const void* k_pages, const void* v_pages,
                                     const int* page_table, int pt_stride, const int* tok_pos, const int* tok_seq,
                                     const int* slots, float* part_o, float* part_ml, int* counters, void* out, int T,
                                     int H, int Hkv, int hd, int page_size, float scale, int window, int n_splits,
                                     const int* work, int teams, const void* next_w, long next_bytes, int early_loads,
                                     const float* sink, float softcap, int keep_first, cudaStream_t stream) {
-    if (T <= 0) return LQ_OK;
-    if (!sizes_ok(H, Hkv, hd, page_size, q_stride, n_splits)) return LQ_BAD_SIZE;
-    if (n_splits > 1 && (!part_o || !part_ml)) return LQ_BAD_SIZE;
-    if (work && (teams < 1 || teams > 65535 || (n_splits > 1 && !counters))) return LQ_BAD_SIZE;
-    if (softcap < 0.f || keep_first < 0) return LQ_BAD_SIZE;
-#define LQ_GO(HD) return launch<HD>(q, q_stride, k_pages, v_pages, page_table, pt_stride, tok_pos, tok_seq, slots, \
-                                    part_o, part_ml, counters, out, T, H, Hkv, hd, page_size, scale, window, n_splits, \
-                                    work, teams, next_w, next_bytes, early_loads, sink, softcap, keep_first, stream)
-    if (hd <= 32) LQ_GO(32);
-    if (hd <= 64) LQ_GO(64);
-    LQ_GO(128);
-#undef LQ_GO
+    return lq_attn_decode_vd(q, q_stride, k_pages, v_pages, page_table, pt_stride, tok_pos, tok_seq, slots, part_o, part_ml, counters,
+                             out, T, H, Hkv, hd, hd, page_size, scale, window, n_splits, work, teams, next_w, next_bytes, early_loads,
+                             sink, softcap, keep_first, stream);
 }
 
 LQ_EXPORT int lq_attn_decode_sink(const void* q, int q_stride, const void* k_pages, const void* v_pages,

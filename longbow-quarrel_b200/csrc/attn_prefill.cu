@@ -57,21 +57,22 @@ __device__ __forceinline__ uint32_t pack_bf16(float lo, float hi) {
     return *reinterpret_cast<uint32_t*>(&v);
 }
 
-// HD: head_dim rounded up to 32, 64 or 128; the real head_dim hd is a multiple of 8.
-template <int HD>
+// HD: head_dim rounded up to 32, 64 or 128; the real head_dim hd is a multiple of 8.  VD: the same for a value head (its size
+// vd may be another than hd, up to 256).
+template <int HD, int VD>
 __global__ void __launch_bounds__(NT)
 attn_prefill_kernel(const __nv_bfloat16* __restrict__ q, int q_stride, const __nv_bfloat16* __restrict__ k_pages,
                     const __nv_bfloat16* __restrict__ v_pages, const int* __restrict__ page_table, int pt_stride,
                     const int* __restrict__ slots, const int* __restrict__ kv_len, const int* __restrict__ qb_seq,
                     const int* __restrict__ qb_row, const int* __restrict__ qb_rows, const int* __restrict__ qb_pos,
                     __nv_bfloat16* __restrict__ out, int H, int Hkv, int hd, float scale_log2, int window, const float* __restrict__ sink,
-                    float cap_pre, int keep_first) {
-    constexpr int LD = HD + PAD;                       // shared-memory row length in elements
+                    float cap_pre, int keep_first, int vd) {
+    constexpr int LD = HD + PAD, LV = VD + PAD;        // shared-memory row lengths in elements: queries and keys, values
     constexpr int KD = HD / 16;                        // k16 steps over the head dimension
     extern __shared__ __align__(16) uint8_t smem_raw[];
     __nv_bfloat16* sq = reinterpret_cast<__nv_bfloat16*>(smem_raw);              // [64][LD]
     __nv_bfloat16* sk = sq + BLOCK_M * LD;                                        // [2][64][LD]
-    __nv_bfloat16* sv = sk + 2 * BLOCK_N * LD;                                    // [2][64][LD]
+    __nv_bfloat16* sv = sk + 2 * BLOCK_N * LD;                                    // [2][64][LV]
 
     const int tid = threadIdx.x, warp = tid >> 5, lane = tid & 31, g = lane >> 2, t = lane & 3;
     // Heads vary fastest: the work list has the blocks with the most keys first, so the launch order is
@@ -103,23 +104,28 @@ attn_prefill_kernel(const __nv_bfloat16* __restrict__ q, int q_stride, const __n
     };
     auto load_kv = [&](int tile, int stage) {
         const int page = pt[tile];
-        const size_t base = ((size_t)page * Hkv + kvh) * BLOCK_N * hd;
+        const size_t base = ((size_t)page * Hkv + kvh) * BLOCK_N * hd, vbase = ((size_t)page * Hkv + kvh) * BLOCK_N * vd;
         const int kb = tile * BLOCK_N;
         for (int i = tid; i < BLOCK_N * (HD / 8); i += NT) {
             int r = i / (HD / 8), c = (i % (HD / 8)) * 8;
             bool ok = kb + r < len && c < hd;
             size_t off = base + (size_t)(ok ? r : 0) * hd + (ok ? c : 0);
             cp_async16((uint32_t)__cvta_generic_to_shared(sk + (stage * BLOCK_N + r) * LD + c), k_pages + off, ok);
-            cp_async16((uint32_t)__cvta_generic_to_shared(sv + (stage * BLOCK_N + r) * LD + c), v_pages + off, ok);
+        }
+        for (int i = tid; i < BLOCK_N * (VD / 8); i += NT) {
+            int r = i / (VD / 8), c = (i % (VD / 8)) * 8;
+            bool ok = kb + r < len && c < vd;
+            size_t off = vbase + (size_t)(ok ? r : 0) * vd + (ok ? c : 0);
+            cp_async16((uint32_t)__cvta_generic_to_shared(sv + (stage * BLOCK_N + r) * LV + c), v_pages + off, ok);
         }
     };
     load_q();
     load_kv(tile_at(0), 0);
     cp_async_commit();
 
-    float o[HD / 8][4];
+    float o[VD / 8][4];
 #pragma unroll
-    for (int j = 0; j < HD / 8; ++j)
+    for (int j = 0; j < VD / 8; ++j)
 #pragma unroll
         for (int i = 0; i < 4; ++i) o[j][i] = 0.f;
     float m0 = -CUDART_INF_F, m1 = -CUDART_INF_F, l0 = 0.f, l1 = 0.f;
@@ -150,7 +156,7 @@ attn_prefill_kernel(const __nv_bfloat16* __restrict__ q, int q_stride, const __n
         // (the block's first window tile may still hold some for a warp whose own window starts later).
         if (kb <= warp_pos_hi && (kb + BLOCK_N > warp_key_lo || kb < keep_first)) {
             const __nv_bfloat16* ks = sk + stage * BLOCK_N * LD;
-            const __nv_bfloat16* vs = sv + stage * BLOCK_N * LD;
+            const __nv_bfloat16* vs = sv + stage * BLOCK_N * LV;
             float s[8][4];
 #pragma unroll
             for (int j = 0; j < 8; ++j)
@@ -213,16 +219,16 @@ attn_prefill_kernel(const __nv_bfloat16* __restrict__ q, int q_stride, const __n
             l0 = l0 * c0 + ps0;
             l1 = l1 * c1 + ps1;
 #pragma unroll
-            for (int j = 0; j < HD / 8; ++j) { o[j][0] *= c0; o[j][1] *= c0; o[j][2] *= c1; o[j][3] *= c1; }
+            for (int j = 0; j < VD / 8; ++j) { o[j][0] *= c0; o[j][1] *= c0; o[j][2] *= c1; o[j][3] *= c1; }
 #pragma unroll
             for (int kk = 0; kk < 4; ++kk) {          // 16 keys per step
 #pragma unroll
-                for (int dp = 0; dp < HD / 16; ++dp) {
+                for (int dp = 0; dp < VD / 16; ++dp) {
                     // B fragments of V, transposed on load: matrices (keys 0-7, d 0-7), (keys 8-15, d 0-7),
                     // (keys 0-7, d 8-15), (keys 8-15, d 8-15)
                     int r = kk * 16 + (lane & 7) + ((lane >> 3) & 1) * 8, c = dp * 16 + (lane >> 4) * 8;
                     uint32_t b0, b1, b2, b3;
-                    ldsm_x4_t((uint32_t)__cvta_generic_to_shared(vs + r * LD + c), b0, b1, b2, b3);
+                    ldsm_x4_t((uint32_t)__cvta_generic_to_shared(vs + r * LV + c), b0, b1, b2, b3);
                     mma_bf16(o[2 * dp], pa[kk][0], pa[kk][1], pa[kk][2], pa[kk][3], b0, b1);
                     mma_bf16(o[2 * dp + 1], pa[kk][0], pa[kk][1], pa[kk][2], pa[kk][3], b2, b3);
                 }
@@ -242,61 +248,75 @@ attn_prefill_kernel(const __nv_bfloat16* __restrict__ q, int q_stride, const __n
     }
     const float i0 = 1.0f / l0, i1 = 1.0f / l1;
 #pragma unroll
-    for (int j = 0; j < HD / 8; ++j) {
+    for (int j = 0; j < VD / 8; ++j) {
         int d = j * 8 + 2 * t;
-        if (d >= hd) continue;
+        if (d >= vd) continue;
         if (row0ok) {
-            size_t off = ((size_t)(row0 + warp * 16 + g) * H + h) * hd + d;
+            size_t off = ((size_t)(row0 + warp * 16 + g) * H + h) * vd + d;
             *reinterpret_cast<uint32_t*>(out + off) = pack_bf16(o[j][0] * i0, o[j][1] * i0);
         }
         if (row1ok) {
-            size_t off = ((size_t)(row0 + warp * 16 + g + 8) * H + h) * hd + d;
+            size_t off = ((size_t)(row0 + warp * 16 + g + 8) * H + h) * vd + d;
             *reinterpret_cast<uint32_t*>(out + off) = pack_bf16(o[j][2] * i1, o[j][3] * i1);
         }
     }
 }
 
-template <int HD>
+template <int HD, int VD>
 int launch(const void* q, int q_stride, const void* k_pages, const void* v_pages, const int* page_table, int pt_stride,
            const int* slots, const int* kv_len, const int* qb_seq, const int* qb_row, const int* qb_rows,
            const int* qb_pos, void* out, int n_blocks, int H, int Hkv, int hd, float scale, int window,
-           const float* sink, float softcap, int keep_first, cudaStream_t stream) {
-    constexpr size_t smem = (size_t)(BLOCK_M + 4 * BLOCK_N) * (HD + PAD) * 2;
+           const float* sink, float softcap, int keep_first, int vd, cudaStream_t stream) {
+    constexpr size_t smem = ((size_t)(BLOCK_M + 2 * BLOCK_N) * (HD + PAD) + (size_t)2 * BLOCK_N * (VD + PAD)) * 2;
     static bool configured = false;
     if (!configured) {
-        if (cudaFuncSetAttribute(attn_prefill_kernel<HD>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem) != cudaSuccess)
+        if (cudaFuncSetAttribute(attn_prefill_kernel<HD, VD>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem) != cudaSuccess)
             return lq_launch_status();
         configured = true;
     }
     dim3 grid(n_blocks * H);
-    return launch_pdl(attn_prefill_kernel<HD>, grid, dim3(NT), smem, stream, (const __nv_bfloat16*)q, q_stride,
+    return launch_pdl(attn_prefill_kernel<HD, VD>, grid, dim3(NT), smem, stream, (const __nv_bfloat16*)q, q_stride,
         (const __nv_bfloat16*)k_pages, (const __nv_bfloat16*)v_pages, page_table, pt_stride, slots, kv_len, qb_seq, qb_row,
         qb_rows, qb_pos, (__nv_bfloat16*)out, H, Hkv, hd, (softcap > 0.f ? softcap : scale) * 1.4426950408889634f, window, sink,
-        softcap > 0.f ? scale / softcap : 0.f, keep_first);
+        softcap > 0.f ? scale / softcap : 0.f, keep_first, vd);
 }
 
 }  // namespace
 
-// q: rows of q_stride elements whose first H*hd hold the query heads; out [T, H*hd].
+// q: rows of q_stride elements whose first H*hd hold the query heads; out [T, H*vd].
 // qb_*: the work list, n_blocks entries: sequence, first packed row, rows (<= 64), position of the first row.
-// head_dim a multiple of 8 and at most 128; the cache's page size must be 64.
+// head_dim a multiple of 8 and at most 128, a value head's size vd one at most 256; the cache's page size must be 64.
 // sink (or null): float32 [H]; each head's softmax denominator gets one more term exp(sink[h]).
 // softcap c (0: none): score <- c tanh(score / c) after the scale.  keep_first n (0: none; with a window): a row's
 // first n keys stay visible when its window has moved past them.
+LQ_EXPORT int lq_attn_prefill_vd(const void* q, int q_stride, const void* k_pages, const void* v_pages,
+                                 const int* page_table, int pt_stride, const int* slots, const int* kv_len,
+                                 const int* qb_seq, const int* qb_row, const int* qb_rows, const int* qb_pos, void* out,
+                                 int n_blocks, int H, int Hkv, int hd, int vd, int page_size, float scale, int window,
+                                 const float* sink, float softcap, int keep_first, cudaStream_t stream) {
+    if (n_blocks <= 0) return LQ_OK;
+    if (softcap < 0.f || keep_first < 0) return LQ_BAD_SIZE;
+    if (hd % 8 || hd > 128 || hd <= 0 || vd % 8 || vd > 256 || vd <= 0 || H % Hkv || page_size != BLOCK_N || q_stride % 8)
+        return LQ_BAD_SIZE;
+#define LQ_GO(HD, VD) return launch<HD, VD>(q, q_stride, k_pages, v_pages, page_table, pt_stride, slots, kv_len, qb_seq, qb_row, \
+                                            qb_rows, qb_pos, out, n_blocks, H, Hkv, hd, scale, window, sink, softcap, keep_first, \
+                                            vd, stream)
+    if (vd > 128) LQ_GO(128, 256);
+    if (hd <= 32 && vd <= 32) LQ_GO(32, 32);
+    if (hd <= 64 && vd <= 64) LQ_GO(64, 64);
+    if (hd <= 64) LQ_GO(64, 128);
+    LQ_GO(128, 128);
+#undef LQ_GO
+}
+
+// The same with values as wide as keys.
 LQ_EXPORT int lq_attn_prefill_capped(const void* q, int q_stride, const void* k_pages, const void* v_pages,
                                      const int* page_table, int pt_stride, const int* slots, const int* kv_len,
                                      const int* qb_seq, const int* qb_row, const int* qb_rows, const int* qb_pos, void* out,
                                      int n_blocks, int H, int Hkv, int hd, int page_size, float scale, int window,
                                      const float* sink, float softcap, int keep_first, cudaStream_t stream) {
-    if (n_blocks <= 0) return LQ_OK;
-    if (softcap < 0.f || keep_first < 0) return LQ_BAD_SIZE;
-    if (hd % 8 || hd > 128 || hd <= 0 || H % Hkv || page_size != BLOCK_N || q_stride % 8) return LQ_BAD_SIZE;
-#define LQ_GO(HD) return launch<HD>(q, q_stride, k_pages, v_pages, page_table, pt_stride, slots, kv_len, qb_seq, qb_row, \
-                                    qb_rows, qb_pos, out, n_blocks, H, Hkv, hd, scale, window, sink, softcap, keep_first, stream)
-    if (hd <= 32) LQ_GO(32);
-    if (hd <= 64) LQ_GO(64);
-    LQ_GO(128);
-#undef LQ_GO
+    return lq_attn_prefill_vd(q, q_stride, k_pages, v_pages, page_table, pt_stride, slots, kv_len, qb_seq, qb_row, qb_rows, qb_pos,
+                              out, n_blocks, H, Hkv, hd, hd, page_size, scale, window, sink, softcap, keep_first, stream);
 }
 
 LQ_EXPORT int lq_attn_prefill(const void* q, int q_stride, const void* k_pages, const void* v_pages,

@@ -45,6 +45,19 @@ __device__ __forceinline__ float warp_max(float v) {
     return v;
 }
 
+// What a gated feed-forward makes of a gate and an up value: u g / (1 + e^(-g)) (limit 0), or with a limit m > 0 both are
+// clamped first and the up value is shifted: (u + 1) g / (1 + e^(-1.702 g)), g = min(gate, m), u = clamp(up, -m, m).
+struct Glu {
+    float lim, slope, shift;
+    __device__ __forceinline__ explicit Glu(float m)
+        : lim(m > 0.f ? m : __builtin_huge_valf()), slope(m > 0.f ? 1.702f : 1.f), shift(m > 0.f ? 1.f : 0.f) {}
+    template <bool FAST> __device__ __forceinline__ float of(float g, float u) const {
+        g = fminf(g, lim);
+        u = fminf(fmaxf(u, -lim), lim) + shift;
+        return u * (g / (1.f + (FAST ? __expf(-slope * g) : expf(-slope * g))));
+    }
+};
+
 // ------------------------------------------------------------------ programmatic dependent launch
 // Kernels of a step follow one another on one stream.  Launched with launch_pdl, a kernel's
 // blocks may be scheduled while the kernel before it is still draining; they run up to

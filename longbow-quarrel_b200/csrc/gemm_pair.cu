@@ -182,7 +182,7 @@ gemm_pair_kernel(const __grid_constant__ CUtensorMap map_a, const __grid_constan
                 // BN holds whole heads; q leaves by TMA, rows of k and v go to their cache pages.
                 qkv_epilogue_staged(taddr, BN, qkv, &map_c, sm.stage[quarter], which, m0 + quarter * 32, M, n0, N, lane);
             } else if (m0 + quarter * 32 < M) {
-                staged_epilogue<EPI>(taddr, BN, sm.stage[quarter], which, &map_c, m0 + quarter * 32, n0, N, lane);
+                staged_epilogue<EPI>(taddr, BN, sm.stage[quarter], which, &map_c, m0 + quarter * 32, n0, N, lane, qkv.glu_limit);
             }
             fence_before();
             __syncwarp();
@@ -265,9 +265,9 @@ LQ_EXPORT int lq_gemm_pair_takes(int M, int N, int K) {
 
 // A [M, K] and W [N, K] bfloat16, row-major, 16-byte aligned, K % 8 == 0; epi: EPI_BF16, EPI_F32, EPI_RESID
 // (C == residual, float32 [M, N], added in place) or EPI_SWIGLU (N counts the interleaved gate and up rows,
-// C is [M, N / 2]).  LQ_BAD_SIZE when the output cannot leave by TMA (rows not 16-byte aligned).
+// C is [M, N / 2]; glu_limit: 0 or the clamped form's limit, see Glu).  LQ_BAD_SIZE when the output cannot leave by TMA (rows not 16-byte aligned).
 LQ_EXPORT int lq_gemm_pair(const void* A, const void* W, void* C, const float* residual, int M, int N, int K, int epi,
-                           cudaStream_t stream) {
+                           float glu_limit, cudaStream_t stream) {
     if (M <= 0 || N <= 0) return LQ_OK;
     if (K <= 0 || K % 8 != 0) return LQ_BAD_SIZE;
     if (((uintptr_t)A & 15) || ((uintptr_t)W & 15)) return LQ_BAD_SIZE;
@@ -276,7 +276,11 @@ LQ_EXPORT int lq_gemm_pair(const void* A, const void* W, void* C, const float* r
         case EPI_BF16: return launch<EPI_BF16>(A, W, C, residual, M, N, K, stream);
         case EPI_F32: return launch<EPI_F32>(A, W, C, residual, M, N, K, stream);
         case EPI_RESID: return residual ? launch<EPI_RESID>(A, W, C, residual, M, N, K, stream) : LQ_BAD_SIZE;
-        case EPI_SWIGLU: return launch<EPI_SWIGLU>(A, W, C, residual, M, N, K, stream);
+        case EPI_SWIGLU: {
+            QkvArgs args{};
+            args.glu_limit = glu_limit;
+            return launch<EPI_SWIGLU>(A, W, C, residual, M, N, K, stream, args);
+        }
     }
     return LQ_BAD_DTYPE;
 }

@@ -87,12 +87,13 @@ int launch_mt(const void* X, const void* W, void* C, const float* residual, int 
 // in_sums [M, in_blocks] holds the rows' sums of squares, in_inv_width = 1 / width, in_eps the norm's eps.
 // next_w, next_bytes (or null): weights that are read next on this stream; their first next_bytes
 // are asked into L2 while this product runs out.
+// glu_limit: for EPI_SWIGLU, 0 or the clamped form's limit (see Glu).
 // out_gain, out_x, out_sums (EPI_RESID only, or null): also write (new residual * out_gain) as
 // bfloat16 [M, N] and the sums of squares [M, lq_gemm_skinny_blocks(N)] for the product that follows.
 LQ_EXPORT int lq_gemm_skinny(const void* X, const void* W, void* C, const float* residual, int M, int N, int K,
                              int epi, const float* in_sums, int in_blocks, float in_inv_width, float in_eps,
                              const float* out_gain, void* out_x, float* out_sums, const void* next_w, long next_bytes,
-                             cudaStream_t stream) {
+                             float glu_limit, cudaStream_t stream) {
     if (M <= 0 || N <= 0) return LQ_OK;
     if (M > 64 || K % 8 != 0 || K <= 0) return LQ_BAD_SIZE;
     if (epi == EPI_SWIGLU && N % 16 != 0) return LQ_BAD_SIZE;
@@ -101,12 +102,14 @@ LQ_EXPORT int lq_gemm_skinny(const void* X, const void* W, void* C, const float*
     if (out_x && (epi != EPI_RESID || !out_gain || !out_sums)) return LQ_BAD_SIZE;
     const NormArgs norm{in_sums, in_blocks, in_inv_width, in_eps, out_x ? out_gain : nullptr,
                         (__nv_bfloat16*)out_x, out_x ? out_sums : nullptr};
+    QkvArgs args{};
+    args.glu_limit = glu_limit;
     int mt = (M + 7) / 8;
     switch (mt) {
-        case 1: return launch_mt<1>(X, W, C, residual, M, N, K, epi, stream, norm, next_w, next_bytes);
-        case 2: return launch_mt<2>(X, W, C, residual, M, N, K, epi, stream, norm, next_w, next_bytes);
-        case 3: case 4: return launch_mt<4>(X, W, C, residual, M, N, K, epi, stream, norm, next_w, next_bytes);
-        default: return launch_mt<8>(X, W, C, residual, M, N, K, epi, stream, norm, next_w, next_bytes);
+        case 1: return launch_mt<1>(X, W, C, residual, M, N, K, epi, stream, norm, next_w, next_bytes, args);
+        case 2: return launch_mt<2>(X, W, C, residual, M, N, K, epi, stream, norm, next_w, next_bytes, args);
+        case 3: case 4: return launch_mt<4>(X, W, C, residual, M, N, K, epi, stream, norm, next_w, next_bytes, args);
+        default: return launch_mt<8>(X, W, C, residual, M, N, K, epi, stream, norm, next_w, next_bytes, args);
     }
 }
 

@@ -52,7 +52,7 @@ __device__ __forceinline__ void mma_bf16(float (&c)[4], uint32_t a0, uint32_t a1
 }
 
 // What the q/k/v epilogue needs beside the product: where each token stands and where its cache
-// page is.  W holds H query heads, then Hkv key heads, then Hkv value heads, hd rows each.
+// page is (and what the gated one needs, its halves' limit).  W holds H query heads, then Hkv key heads, then Hkv value heads, hd rows each.
 struct QkvArgs {
     const float* cos_t;       // [positions, hd / 2] or null (no rotation)
     const float* sin_t;
@@ -63,6 +63,7 @@ struct QkvArgs {
     __nv_bfloat16* k_pages;
     __nv_bfloat16* v_pages;
     int pt_stride, H, Hkv, hd, page_size;
+    float glu_limit;          // EPI_SWIGLU: see Glu
 };
 
 // RMS norm folded into the products on either side of it (null pointers: not used).
@@ -310,7 +311,7 @@ struct Unit {
                 float u = total(r + 8, m) * sc;
                 int f = (n0 >> 1) + r;
                 if (f < (N >> 1))
-                    ((__nv_bfloat16*)Cout)[(size_t)m * (N >> 1) + f] = __float2bfloat16_rn(u * (s / (1.0f + expf(-s))));
+                    ((__nv_bfloat16*)Cout)[(size_t)m * (N >> 1) + f] = __float2bfloat16_rn(Glu(qkv.glu_limit).of<false>(s, u));
             } else {
                 int n = n0 + r;
                 if (n >= N) continue;

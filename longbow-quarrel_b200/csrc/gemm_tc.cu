@@ -59,19 +59,20 @@ struct Smem {
 // of a matrix whose rows are 16-byte aligned, the case in which this function would load float4s itself).
 template <int EPI>
 __device__ __forceinline__ void store_chunk(const uint32_t (&r)[32], void* Cout,
-                                            const float* residual, int m, int n, int M, int N, int n_lim,
+                                            const float* residual, int m, int n, int M, int N, int n_lim, float glu_limit,
                                             const float4* pre = nullptr) {
     if (m >= M || n >= n_lim) return;
     if (EPI == EPI_SWIGLU) {
         // 32 columns = [8 gate, 8 up, 8 gate, 8 up] -> 16 outputs at column n / 2 of [M, N / 2].
         const int NO = N >> 1, no = n >> 1, no_lim = n_lim >> 1;
+        const Glu glu(glu_limit);
         float o[16];
 #pragma unroll
         for (int h = 0; h < 2; ++h)
 #pragma unroll
             for (int i = 0; i < 8; ++i) {
                 float g = __uint_as_float(r[h * 16 + i]), u = __uint_as_float(r[h * 16 + 8 + i]);
-                o[h * 8 + i] = u * (g / (1.0f + __expf(-g)));
+                o[h * 8 + i] = glu.of<true>(g, u);
             }
         __nv_bfloat16* dst = (__nv_bfloat16*)Cout + (size_t)m * NO + no;
         if (no + 16 <= no_lim && (NO & 7) == 0) {
@@ -267,7 +268,7 @@ gemm_tc_kernel(const __grid_constant__ CUtensorMap map_a, const __grid_constant_
                 if constexpr (STAGED) {
                     if (m0 + quarter * 32 < M)          // (with 64-row stages only the first two warps hold rows of x)
                         staged_epilogue<EPI>(taddr, BN, sm.stage[quarter], stage_buf, &map_c,
-                                             (splits > 1 ? range * plane_rows : 0) + m0 + quarter * 32, n0, N, lane);
+                                             (splits > 1 ? range * plane_rows : 0) + m0 + quarter * 32, n0, N, lane, qkv.glu_limit);
                 }
             } else {
 #pragma unroll 1
@@ -281,9 +282,9 @@ gemm_tc_kernel(const __grid_constant__ CUtensorMap map_a, const __grid_constant_
 #pragma unroll
                         for (int i = 0; i < 8; ++i) now[i] = pre[i];
                         fetched = c + 1 < (BN + 31) / 32 && fetch(c + 1);
-                        store_chunk<EPI>(r, dst, residual, m, n0 + c * 32, M, N, n_lim, have ? now : nullptr);
+                        store_chunk<EPI>(r, dst, residual, m, n0 + c * 32, M, N, n_lim, 0.f, have ? now : nullptr);
                     } else {
-                        store_chunk<EPI>(r, dst, residual, m, n0 + c * 32, M, N, n_lim);
+                        store_chunk<EPI>(r, dst, residual, m, n0 + c * 32, M, N, n_lim, qkv.glu_limit);
                     }
                 }
             }
@@ -363,9 +364,10 @@ __global__ void __launch_bounds__(256) splitk_reduce_kernel(const float* __restr
         sum4(gcol, v);
         sum4(gcol + 8, u);
         __nv_bfloat16* dst = (__nv_bfloat16*)Cout + (size_t)m * NO + c;
+        const Glu glu(qkv.glu_limit);
 #pragma unroll
         for (int i = 0; i < 4; ++i)
-            if (c + i < NO) dst[i] = __float2bfloat16_rn(u[i] * (v[i] / (1.0f + __expf(-v[i]))));
+            if (c + i < NO) dst[i] = __float2bfloat16_rn(glu.of<true>(v[i], u[i]));
         return;
     }
     sum4(c, v);
@@ -525,10 +527,13 @@ int gemm_tc_dispatch(const void* A, const void* W, void* C, const float* residua
 // A [M, K] and W [N, K] bfloat16, row-major, 16-byte aligned, K % 8 == 0.
 // For EPI_SWIGLU, N counts the interleaved gate and up rows (N % 16 == 0) and C is [M, N / 2].
 // scratch: lq_gemm_tc_scratch_floats(M, N, K) floats (0: unused): a plane of M rounded up to 32 rows for each range of K.
+// glu_limit: for EPI_SWIGLU, 0 or the clamped form's limit (see Glu).
 LQ_EXPORT int lq_gemm_tc(const void* A, const void* W, void* C, const float* residual, int M, int N, int K, int epi,
-                         float* scratch, cudaStream_t stream) {
+                         float* scratch, float glu_limit, cudaStream_t stream) {
     if (epi < EPI_BF16 || epi > EPI_SWIGLU) return LQ_BAD_DTYPE;
-    return gemm_tc_dispatch(A, W, C, residual, M, N, K, epi, scratch, QkvArgs{}, stream);
+    QkvArgs args{};
+    args.glu_limit = glu_limit;
+    return gemm_tc_dispatch(A, W, C, residual, M, N, K, epi, scratch, args, stream);
 }
 
 // The q/k/v projection with its epilogue fused: X [M, K] . W^T for W [(H + 2 Hkv) hd, K]; q and k are rotated

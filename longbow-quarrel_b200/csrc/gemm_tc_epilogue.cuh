@@ -39,7 +39,8 @@ template <int EPI> struct StagedCols {
 // next and is kept across calls, as are the stores in flight (wait for them with bulk_wait<0> at the end).
 template <int EPI>
 __device__ __forceinline__ void staged_epilogue(uint32_t taddr, int bn, uint8_t* bufs, int& which, const CUtensorMap* map_c,
-                                                int y, int n0, int N, int lane) {
+                                                int y, int n0, int N, int lane, float glu_limit) {
+    const Glu glu(glu_limit);
     constexpr int COLS = StagedCols<EPI>::value;
 #pragma unroll 1
     for (int c0 = 0; c0 < bn && n0 + c0 < N; c0 += COLS) {
@@ -71,7 +72,7 @@ __device__ __forceinline__ void staged_epilogue(uint32_t taddr, int bn, uint8_t*
 #pragma unroll
                     for (int i = 0; i < 8; ++i) {
                         const float gt = __uint_as_float(r[h * 16 + i]), up = __uint_as_float(r[h * 16 + 8 + i]);
-                        o[h * 8 + i] = up * (gt / (1.0f + __expf(-gt)));
+                        o[h * 8 + i] = glu.of<true>(gt, up);
                     }
                 *staged_at(buf, lane, sub * 2) = make_uint4(pack2(o[0], o[1]), pack2(o[2], o[3]), pack2(o[4], o[5]), pack2(o[6], o[7]));
                 *staged_at(buf, lane, sub * 2 + 1) = make_uint4(pack2(o[8], o[9]), pack2(o[10], o[11]), pack2(o[12], o[13]), pack2(o[14], o[15]));
@@ -89,7 +90,8 @@ __device__ __forceinline__ void staged_epilogue(uint32_t taddr, int bn, uint8_t*
     }
 }
 
-// What the q/k/v epilogue needs beside the product: where each row stands and where its cache page is.
+// What the q/k/v epilogue needs beside the product: where each row stands and where its cache page is (and what the gated
+// one needs, its halves' limit).
 // W holds H query heads, then Hkv key heads, then Hkv value heads, hd rows each.
 struct QkvArgs {
     const float* cos_t;       // [positions, hd / 2] or null (no rotation)
@@ -101,6 +103,7 @@ struct QkvArgs {
     __nv_bfloat16* k_pages;
     __nv_bfloat16* v_pages;
     int pt_stride, H, Hkv, hd, page_size;
+    float glu_limit;          // EPI_SWIGLU: see Glu
 };
 
 // Where elements j .. of head `head` of row m go: q_out, or the row's place in a cache page.

@@ -1160,12 +1160,9 @@ LQ_EXPORT int lq_activation(const void* x, void* out, int dtype, long long total
 
 // out[t, f] = act(gu[t, f] + b[f]) * (gu[t, F + f] + b[F + f]): a gated feed-forward's two halves (gate columns, then up
 // columns) with their biases (float32 [2F], or none), the activation in float32.
-// act 5 clamps both halves: g sigmoid(1.702 g) (u + 1) with g = min(gate, limit), u = clamp(up, -limit, limit).
+// act 5: the clamped form of Glu.
 __device__ __forceinline__ float gated(float g, float u, int act, float limit) {
-    if (act != 5) return activation(g, act) * u;
-    g = fminf(g, limit);
-    u = fminf(fmaxf(u, -limit), limit);
-    return g / (1.f + expf(-1.702f * g)) * (u + 1.f);
+    return act == 5 ? Glu(limit).of<false>(g, u) : activation(g, act) * u;
 }
 
 template <typename TI, typename TO>
@@ -1413,9 +1410,9 @@ LQ_EXPORT int lq_attention_plain(const void* q, int q_stride, int dtype, const v
 
 // ------------------------------------------------------------------ swiglu
 // out = up * gate / (1 + e^-gate) from gu [T, 2F].  block == 0: gate in columns
-// [0, F), up in [F, 2F).  block == b > 0: columns alternate b gate, b up, b gate, ...
+// [0, F), up in [F, 2F).  block == b > 0: columns alternate b gate, b up, b gate, ...  limit > 0: the clamped form (see Glu).
 template <typename T>
-__global__ void swiglu_kernel(const T* __restrict__ gu, T* __restrict__ out, int F, size_t total, int block) {
+__global__ void swiglu_kernel(const T* __restrict__ gu, T* __restrict__ out, int F, size_t total, int block, float limit) {
     pdl_launch_dependents();
     pdl_wait();
     size_t i = (size_t)blockIdx.x * blockDim.x + threadIdx.x;
@@ -1426,18 +1423,18 @@ __global__ void swiglu_kernel(const T* __restrict__ gu, T* __restrict__ out, int
     int ui = block ? gi + block : F + f;
     float g = to_f32(gu[t * 2 * F + gi]);
     float u = to_f32(gu[t * 2 * F + ui]);
-    out[i] = from_f32<T>(u * (g / (1.0f + expf(-g))));
+    out[i] = from_f32<T>(Glu(limit).of<false>(g, u));
 }
 
-LQ_EXPORT int lq_swiglu(const void* gu, void* out, int dtype, int T, int F, int block, cudaStream_t stream) {
+LQ_EXPORT int lq_swiglu(const void* gu, void* out, int dtype, int T, int F, int block, float limit, cudaStream_t stream) {
     size_t total = (size_t)T * F;
     if (total == 0) return LQ_OK;
     if (block < 0 || (block && F % block)) return LQ_BAD_SIZE;
     unsigned blocks = (unsigned)((total + 255) / 256);
     if (dtype == LQ_F32)
-        return launch_pdl(swiglu_kernel<float>, dim3(blocks), dim3(256), 0, stream, (const float*)gu, (float*)out, F, total, block);
+        return launch_pdl(swiglu_kernel<float>, dim3(blocks), dim3(256), 0, stream, (const float*)gu, (float*)out, F, total, block, limit);
     else if (dtype == LQ_BF16)
-        return launch_pdl(swiglu_kernel<__nv_bfloat16>, dim3(blocks), dim3(256), 0, stream, (const __nv_bfloat16*)gu, (__nv_bfloat16*)out, F, total, block);
+        return launch_pdl(swiglu_kernel<__nv_bfloat16>, dim3(blocks), dim3(256), 0, stream, (const __nv_bfloat16*)gu, (__nv_bfloat16*)out, F, total, block, limit);
     else
         return LQ_BAD_DTYPE;
     return lq_launch_status();

@@ -13,7 +13,7 @@ KEYS_PER_SPLIT = 128         # a slice shorter than this is not worth a block of
 
 def resident_blocks(device, hd: int = 128) -> int:
     """Blocks of the decode kernel that run at a time: one (8 warps, ~200 KB of key/value rings) per SM,
-    two where the rings are half as large (head_dim up to 64)."""
+    two where the rings are half as large (hd, the larger of a head's key and value sizes, up to 64)."""
     return ops.sm_count(device) * (2 if hd <= 64 else 1)
 
 
@@ -120,32 +120,35 @@ def decode_work_name(H: int, Hkv: int, window: int | None, keep_first: int = 0, 
 PREFILL_LISTS = {"query_blocks64": query_blocks(64), "query_blocks128": query_blocks(128)}
 
 
-def prefill_kernel(dtype: torch.dtype, hd: int, page_size: int = 64) -> str | None:
-    """Which prompt kernel takes queries of this dtype and head size: "tc" (tcgen05), "mma" (mma.sync),
-    or None (the plain kernel)."""
+def _mma_sizes(hd: int, vd: int | None) -> bool:
+    """Head sizes that the mma.sync kernels take: keys of whole sixteens up to 128, values of whole eights up to 256."""
+    return hd % 16 == 0 and hd <= 128 and (vd is None or (vd % 8 == 0 and vd <= 256))
+
+
+def prefill_kernel(dtype: torch.dtype, hd: int, page_size: int = 64, vd: int | None = None) -> str | None:
+    """Which prompt kernel takes queries of this dtype, head size and value size (None: the head's): "tc" (tcgen05),
+    "mma" (mma.sync), or None (the plain kernel)."""
     if dtype != torch.bfloat16 or page_size != 64:
         return None
-    if USE_TC_PREFILL and hd in (64, 128):
+    if USE_TC_PREFILL and hd in (64, 128) and vd in (None, hd):
         return "tc"
-    if hd % 16 == 0 and hd <= 128:
-        return "mma"
-    return None
+    return "mma" if _mma_sizes(hd, vd) else None
 
 
-def decode_kernel(dtype: torch.dtype, hd: int) -> bool:
-    """Whether single tokens of this dtype and head size go to the split decode kernel."""
-    return dtype == torch.bfloat16 and hd % 16 == 0 and hd <= 128
+def decode_kernel(dtype: torch.dtype, hd: int, vd: int | None = None) -> bool:
+    """Whether single tokens of this dtype, head size and value size go to the split decode kernel."""
+    return dtype == torch.bfloat16 and _mma_sizes(hd, vd)
 
 
 def step_needs(dtype: torch.dtype, hd: int, H: int | None = None, Hkv: int | None = None, window: int | None = None,
-               device=None, keep_first: int = 0, chunk: int | None = None) -> dict:
+               device=None, keep_first: int = 0, chunk: int | None = None, vd: int | None = None) -> dict:
     """The work lists that attention of this dtype and head size reads: the query blocks of steps with
     prompts, and (when the head counts are given) the balanced segments of steps of single tokens."""
-    kind = prefill_kernel(dtype, hd)
+    kind = prefill_kernel(dtype, hd, vd=vd)
     name = {"tc": "query_blocks128", "mma": "query_blocks64"}.get(kind)
     needs = {name: PREFILL_LISTS[name]} if name else {}
-    if H is not None and Hkv and BALANCED_DECODE and decode_kernel(dtype, hd):
-        needs[decode_work_name(H, Hkv, window, keep_first, chunk)] = decode_work(H, Hkv, window, device, hd, keep_first, chunk)
+    if H is not None and Hkv and BALANCED_DECODE and decode_kernel(dtype, hd, vd):
+        needs[decode_work_name(H, Hkv, window, keep_first, chunk)] = decode_work(H, Hkv, window, device, max(hd, vd or hd), keep_first, chunk)
     return needs
 
 
@@ -166,10 +169,7 @@ def attention(qkv, cache_view, ctx, H, Hkv, hd, scale, window, next_w=None, vd=N
     sees only its own block of n positions.  gate_per_head: the gate is [T, H], one number for a head's values."""
     vd = vd or hd
     keep_first = int(keep_first or 0) if window else 0
-    if vd != hd:
-        return general_attention(qkv, cache_view, ctx, H, Hkv, hd, vd, scale, window, sink, gate, softcap, keep_first, chunk,
-                                 gate_per_head)
-    out = _attention(qkv, cache_view, ctx, H, Hkv, hd, scale, window, next_w, sink, gate, softcap, keep_first, chunk)
+    out = _attention(qkv, cache_view, ctx, H, Hkv, hd, scale, window, next_w, sink, gate, softcap, keep_first, chunk, vd)
     if gate is not None and out is not None:
         # The tensor-core kernels leave the gate to a kernel of its own.
         return ops.gate_mul(out, gate, "sigmoid", group=vd if gate_per_head else 1)
@@ -177,14 +177,14 @@ def attention(qkv, cache_view, ctx, H, Hkv, hd, scale, window, next_w=None, vd=N
                                                          softcap, keep_first, chunk, gate_per_head)
 
 
-def _attention(qkv, cache_view, ctx, H, Hkv, hd, scale, window, next_w, sink, gate, softcap=None, keep_first=0, chunk=None):
+def _attention(qkv, cache_view, ctx, H, Hkv, hd, scale, window, next_w, sink, gate, softcap, keep_first, chunk, vd):
     """The tensor-core kernels where they take the sizes; None where only the plain kernel does and a gate
-    is to be applied (the plain kernel applies it itself)."""
+    is to be applied or values have a size of their own (the plain kernel does both itself)."""
     aligned = qkv.stride(0) % 8 == 0 and qkv.data_ptr() % 16 == 0
     more = dict(sink=sink, softcap=softcap, keep_first=keep_first)
     mask = ops.span(window, chunk)          # the kernels take a window as w and blocks of n positions as -n
     if not ctx.decode and aligned:
-        kind = prefill_kernel(qkv.dtype, hd, cache_view.page_size)
+        kind = prefill_kernel(qkv.dtype, hd, cache_view.page_size, vd)
         if kind == "tc":
             blocks = _blocks(ctx, "query_blocks128")
             if blocks is not None:
@@ -195,21 +195,21 @@ def _attention(qkv, cache_view, ctx, H, Hkv, hd, scale, window, next_w, sink, ga
             blocks = _blocks(ctx, "query_blocks64")
             if blocks is not None:
                 return ops.attn_prefill(qkv, cache_view.k_pages, cache_view.v_pages, cache_view.page_table, ctx.slots,
-                                        ctx.kv_len, blocks, H, Hkv, hd, cache_view.page_size, scale, mask, **more)
-    if ctx.decode and aligned and decode_kernel(qkv.dtype, hd) and cache_view.page_size % 16 == 0:
+                                        ctx.kv_len, blocks, H, Hkv, hd, cache_view.page_size, scale, mask, vd=vd, **more)
+    if ctx.decode and aligned and decode_kernel(qkv.dtype, hd, vd) and cache_view.page_size % 16 == 0:
         work = ctx.extra.get(decode_work_name(H, Hkv, window, keep_first, chunk))
         if work is not None and work.numel():
-            teams = decode_teams(ctx.T, Hkv, -(-(H // Hkv) // 16), resident_blocks(qkv.device, hd))
+            teams = decode_teams(ctx.T, Hkv, -(-(H // Hkv) // 16), resident_blocks(qkv.device, max(hd, vd)))
             if work.numel() == decode_work_size(ctx.T, teams):
                 return ops.attn_decode(qkv, cache_view.k_pages, cache_view.v_pages, cache_view.page_table, ctx.tok_pos,
                                        ctx.tok_seq, ctx.slots, H, Hkv, hd, cache_view.page_size, scale, mask,
                                        min(MAX_SPLITS, teams), next_w=next_w, early_loads=True, work=work, teams=teams,
-                                       **more)
-        n_splits = decode_splits(ctx.T, Hkv, -(-(H // Hkv) // 16), ctx.max_kv, resident_blocks(qkv.device, hd))
+                                       vd=vd, **more)
+        n_splits = decode_splits(ctx.T, Hkv, -(-(H // Hkv) // 16), ctx.max_kv, resident_blocks(qkv.device, max(hd, vd)))
         return ops.attn_decode(qkv, cache_view.k_pages, cache_view.v_pages, cache_view.page_table, ctx.tok_pos,
                                ctx.tok_seq, ctx.slots, H, Hkv, hd, cache_view.page_size, scale, mask, n_splits,
-                               next_w=next_w, early_loads=True, **more)      # a decode step: one new token per sequence
-    if gate is not None:
+                               next_w=next_w, early_loads=True, vd=vd, **more)      # a decode step: one new token per sequence
+    if gate is not None or vd != hd:
         return None
     return ops.attention_plain(qkv, cache_view.k_pages, cache_view.v_pages, cache_view.page_table, ctx.tok_pos,
                                ctx.tok_seq, ctx.slots, H, Hkv, hd, cache_view.page_size, scale, window, sink=sink,

@@ -104,17 +104,17 @@ def interleave_gate_up(gate: torch.Tensor, up: torch.Tensor) -> torch.Tensor:
     return torch.stack([gate.reshape(F // b, b, K), up.reshape(F // b, b, K)], dim=1).reshape(2 * F, K).contiguous()
 
 
-def linear_swiglu(a: torch.Tensor, weight: LinearWeight, block: int) -> torch.Tensor:
-    """act(a . Wg^T) * (a . Wu^T) for the stacked weight [2F, K]; block 0 = gate rows
-    then up rows, block 8 = interleaved."""
+def linear_swiglu(a: torch.Tensor, weight: LinearWeight, block: int, limit: float = 0.0) -> torch.Tensor:
+    """silu(a . Wg^T) * (a . Wu^T) for the stacked weight [2F, K]; block 0 = gate rows
+    then up rows, block 8 = interleaved.  limit > 0: the clamped form of ops.swiglu."""
     if block == GATE_UP_BLOCK and a.dtype == torch.bfloat16 and weight.tensor.dtype == torch.bfloat16:
         from . import tensorcore
-        out = tensorcore.linear_swiglu_bf16(a, weight)
+        out = tensorcore.linear_swiglu_bf16(a, weight, limit)
         if out is not None:
             note(weight)
             return out
     gu = linear(a, weight, a.dtype)
-    return ops.swiglu(gu, block)
+    return ops.swiglu(gu, block, limit=limit)
 
 
 def linear_act(a: torch.Tensor, weight: LinearWeight, activation: str, out_dtype: torch.dtype) -> torch.Tensor:

@@ -374,15 +374,16 @@ def span(window: int | None, chunk: int | None = None) -> int:
     return int(window or 0)
 
 
-def swiglu(gu: torch.Tensor, block: int = 0, out: torch.Tensor | None = None) -> torch.Tensor:
+def swiglu(gu: torch.Tensor, block: int = 0, out: torch.Tensor | None = None, limit: float = 0.0) -> torch.Tensor:
     """gu [T, 2F] -> up * silu(gate) [T, F].  block 0: gate columns, then up columns;
-    block b: b gate columns, b up columns, alternating."""
+    block b: b gate columns, b up columns, alternating.  limit m > 0: (u + 1) g sigmoid(1.702 g) instead, with
+    g = min(gate, m) and u = clamp(up, -m, m)."""
     T, F2 = gu.shape
     F = F2 // 2
     if out is None:
         out = torch.empty((T, F), dtype=gu.dtype, device=gu.device)
-    fn = _fn("plain_kernels", "lq_swiglu", [c_void_p, c_void_p, c_int, c_int, c_int, c_int, c_void_p])
-    _check(fn(_p(_contig(gu, "gu")), _p(out), dtype_code(gu), T, F, block, _stream()), "swiglu")
+    fn = _fn("plain_kernels", "lq_swiglu", [c_void_p, c_void_p, c_int, c_int, c_int, c_int, c_float, c_void_p])
+    _check(fn(_p(_contig(gu, "gu")), _p(out), dtype_code(gu), T, F, block, float(limit), _stream()), "swiglu")
     return out
 
 
@@ -1129,11 +1130,11 @@ def _next(next_w, limit=None):
 
 
 def gemm_skinny(a, w: torch.Tensor, epi: int, residual: torch.Tensor | None = None,
-                out: torch.Tensor | None = None, emit: tuple | None = None, next_w: torch.Tensor | None = None):
+                out: torch.Tensor | None = None, emit: tuple | None = None, next_w: torch.Tensor | None = None, limit: float = 0.0):
     """a [M <= 64, K] . w [N, K]^T, both bfloat16, streaming w once from memory.
     epi: EPI_BF16 / EPI_F32 store; EPI_RESID adds into the float32 `residual` in place;
     EPI_SWIGLU reads w as alternating blocks of 8 gate and 8 up rows and stores
-    up * silu(gate) [M, N / 2].
+    up * silu(gate) [M, N / 2], or with limit > 0 the clamped form (see swiglu).
     `a` may be NormedRows.  emit = (gain [N] float32, eps), with EPI_RESID only: also returns what the
     RMS norm with that gain makes of the new residual, as NormedRows: (residual, rows).
     next_w: the weights that the stream reads after these; their first bytes are asked into L2."""
@@ -1163,11 +1164,11 @@ def gemm_skinny(a, w: torch.Tensor, epi: int, residual: torch.Tensor | None = No
                           torch.empty((M, -(-N // 16)), dtype=torch.float32, device=a.device), eps)
     fn = _fn("gemm_skinny", "lq_gemm_skinny", [c_void_p, c_void_p, c_void_p, c_void_p, c_int, c_int, c_int, c_int,
                                                c_void_p, c_int, c_float, c_float, c_void_p, c_void_p, c_void_p, c_void_p,
-                                               c_long, c_void_p])
+                                               c_long, c_float, c_void_p])
     next_p, next_n = _next(next_w)
     _check(fn(_p(_contig(a, "a")), _p(_contig(w, "w")), _p(out), _p(residual), M, N, K, epi, in_sums, in_blocks, in_inv,
               in_eps, _p(gain), _p(rows.data) if rows else None, _p(rows.sums) if rows else None, next_p, next_n,
-              _stream()), "gemm_skinny", 1, f"gemm_skinny:rows{-(-M // 8) * 8}" + (":norm_in" if in_blocks else "")
+              float(limit), _stream()), "gemm_skinny", 1, f"gemm_skinny:rows{-(-M // 8) * 8}" + (":norm_in" if in_blocks else "")
            + (":norm_out" if rows else ""))
     return (out, rows) if emit is not None else out
 
@@ -1222,7 +1223,7 @@ def _gemm_tc_scratch_floats(M: int, N: int, K: int) -> int:
 
 
 def gemm_tc(a: torch.Tensor, w: torch.Tensor, epi: int, residual: torch.Tensor | None = None,
-            out: torch.Tensor | None = None) -> torch.Tensor:
+            out: torch.Tensor | None = None, limit: float = 0.0) -> torch.Tensor:
     """a [M, K] . w [N, K]^T on the tcgen05 tensor cores (TMA-fed, float32 accumulation in
     tensor memory), with the epilogues of gemm_skinny.  For many rows; with few tiles (few rows
     and a narrow weight) the contraction is cut into ranges that a second kernel adds."""
@@ -1245,15 +1246,15 @@ def gemm_tc(a: torch.Tensor, w: torch.Tensor, epi: int, residual: torch.Tensor |
     if (gemm_pair_takes(M, N, K) and out.is_contiguous() and out.data_ptr() % 16 == 0
             and (out_cols * out.element_size()) % 16 == 0 and a.is_contiguous() and w.is_contiguous()):
         # Many rows: tiles of 256 x 256 on pairs of SMs, the output leaving by TMA.
-        fn = _fn("gemm_pair", "lq_gemm_pair", [c_void_p, c_void_p, c_void_p, c_void_p, c_int, c_int, c_int, c_int, c_void_p])
-        _check(fn(_p(a), _p(w), _p(out), _p(residual), M, N, K, epi, _stream()), "gemm_pair")
+        fn = _fn("gemm_pair", "lq_gemm_pair", [c_void_p, c_void_p, c_void_p, c_void_p, c_int, c_int, c_int, c_int, c_float, c_void_p])
+        _check(fn(_p(a), _p(w), _p(out), _p(residual), M, N, K, epi, float(limit), _stream()), "gemm_pair")
         return out
     # Few tiles (few rows, narrow weight): the kernel cuts the contraction into ranges and adds them afterwards.
     splits = int(_fn("gemm_tc", "lq_gemm_tc_splits", [c_int, c_int, c_int])(M, N, K))
     scratch = torch.empty(_gemm_tc_scratch_floats(M, N, K), dtype=torch.float32, device=a.device) if splits > 1 else None
     fn = _fn("gemm_tc", "lq_gemm_tc", [c_void_p, c_void_p, c_void_p, c_void_p, c_int, c_int, c_int, c_int, c_void_p,
-                                       c_void_p])
-    _check(fn(_p(_contig(a, "a")), _p(_contig(w, "w")), _p(out), _p(residual), M, N, K, epi, _p(scratch), _stream()),
+                                       c_float, c_void_p])
+    _check(fn(_p(_contig(a, "a")), _p(_contig(w, "w")), _p(out), _p(residual), M, N, K, epi, _p(scratch), float(limit), _stream()),
            "gemm_tc", 2 if splits > 1 else 1, "gemm_tc:split_k" if splits > 1 else ("gemm_tc:few_rows" if M <= 64 else None))
     return out
 
@@ -1307,28 +1308,33 @@ def _check_sink(sink, H: int):
 
 def attn_prefill(q: torch.Tensor, k_pages, v_pages, page_table, slots, kv_len, query_blocks, H: int, Hkv: int, hd: int,
                  page_size: int, scale: float, window: int | None, out: torch.Tensor | None = None,
-                 sink: torch.Tensor | None = None, softcap: float | None = None, keep_first: int = 0) -> torch.Tensor:
+                 sink: torch.Tensor | None = None, softcap: float | None = None, keep_first: int = 0,
+                 vd: int | None = None) -> torch.Tensor:
     """Causal attention of blocks of query rows over the paged bfloat16 cache (flash style:
     tensor-core products, online softmax in float32).  query_blocks = (sequence, first row,
     rows, first position) int32 tensors, one entry for each block of at most 64 rows.  softcap c: score <-
     c tanh(score / c) after the scale; keep_first n (with a window): a row's first n keys stay visible.  window: as `span`
-    makes it (w positions; -n for blocks of n positions; 0 or None for all)."""
+    makes it (w positions; -n for blocks of n positions; 0 or None for all).  vd: size of a value head (default hd)."""
     T = q.shape[0]
+    vd = vd or hd
     if q.dtype != torch.bfloat16 or k_pages.dtype != torch.bfloat16:
         raise KernelError("attn_prefill takes bfloat16 queries and cache")
-    if hd % 16 or hd > 128 or page_size != 64:
-        raise KernelError(f"attn_prefill: head_dim {hd} (multiple of 16, at most 128), page size {page_size} (64)")
+    if hd % 16 or hd > 128 or vd % 8 or vd > 256 or page_size != 64:
+        raise KernelError(f"attn_prefill: head_dim {hd} (multiple of 16, at most 128), value size {vd} (multiple of 8, at most 256), "
+                          f"page size {page_size} (64)")
+    if k_pages.shape[-1] != hd or v_pages.shape[-1] != vd:
+        raise KernelError(f"attn_prefill: the cache's heads are {k_pages.shape[-1]} and {v_pages.shape[-1]} wide, not {hd} and {vd}")
     if out is None:
-        out = torch.empty((T, H * hd), dtype=torch.bfloat16, device=q.device)
+        out = torch.empty((T, H * vd), dtype=torch.bfloat16, device=q.device)
     qb_seq, qb_row, qb_rows, qb_pos = query_blocks
-    fn = _fn("attn_prefill", "lq_attn_prefill_capped", [c_void_p, c_int, c_void_p, c_void_p, c_void_p, c_int, c_void_p, c_void_p,
-                                                        c_void_p, c_void_p, c_void_p, c_void_p, c_void_p, c_int, c_int, c_int,
-                                                        c_int, c_int, c_float, c_int, c_void_p, c_float, c_int, c_void_p])
+    fn = _fn("attn_prefill", "lq_attn_prefill_vd", [c_void_p, c_int, c_void_p, c_void_p, c_void_p, c_int, c_void_p, c_void_p,
+                                                    c_void_p, c_void_p, c_void_p, c_void_p, c_void_p, c_int, c_int, c_int, c_int,
+                                                    c_int, c_int, c_float, c_int, c_void_p, c_float, c_int, c_void_p])
     _check_sink(sink, H)
     _check(fn(_p(q), q.stride(0), _p(k_pages), _p(v_pages), _p(page_table), page_table.stride(0), _p(slots), _p(kv_len),
-              _p(qb_seq), _p(qb_row), _p(qb_rows), _p(qb_pos), _p(out), qb_seq.numel(), H, Hkv, hd, page_size,
+              _p(qb_seq), _p(qb_row), _p(qb_rows), _p(qb_pos), _p(out), qb_seq.numel(), H, Hkv, hd, vd, page_size,
               float(scale), int(window or 0), _p(sink), float(softcap or 0.0), int(keep_first if window else 0), _stream()),
-           "attn_prefill")
+           "attn_prefill", 1, "attn_prefill:vd" if vd != hd else None)
     return out
 
 
@@ -1369,7 +1375,7 @@ def attn_decode(q: torch.Tensor, k_pages, v_pages, page_table, tok_pos, tok_seq,
                 out: torch.Tensor | None = None, scratch: tuple | None = None,
                 next_w: torch.Tensor | None = None, early_loads: bool = False,
                 work: torch.Tensor | None = None, teams: int = 0, sink: torch.Tensor | None = None,
-                softcap: float | None = None, keep_first: int = 0) -> torch.Tensor:
+                softcap: float | None = None, keep_first: int = 0, vd: int | None = None) -> torch.Tensor:
     """Attention of single query rows over the paged bfloat16 cache, the keys of each
     sequence cut into n_splits slices that are merged afterwards.  With `work` (int32: teams + 1 offsets,
     then (token, first tile, last tile + 1, part, parts) per segment) the grid is `teams` blocks per kv
@@ -1382,21 +1388,24 @@ def attn_decode(q: torch.Tensor, k_pages, v_pages, page_table, tok_pos, tok_seq,
     scale.  keep_first n (with a window): a token's first n keys stay visible once its window has moved past them;
     the tiles that a work list counts are then the kept tiles ahead of the window and after them the window's.
     window: as `span` makes it (w positions; -n for blocks of n positions, whose tiles a work list counts from the
-    block's first; 0 or None for all)."""
+    block's first; 0 or None for all).  vd: size of a value head (default hd)."""
     T = q.shape[0]
+    vd = vd or hd
     if q.dtype != torch.bfloat16 or k_pages.dtype != torch.bfloat16:
         raise KernelError("attn_decode takes bfloat16 queries and cache")
-    if hd % 16 or hd > 128:
-        raise KernelError(f"attn_decode: head_dim {hd} must be a multiple of 16 and at most 128")
+    if hd % 16 or hd > 128 or vd % 8 or vd > 256:
+        raise KernelError(f"attn_decode: head_dim {hd} must be a multiple of 16 and at most 128, a value's size {vd} one of 8 and at most 256")
+    if k_pages.shape[-1] != hd or v_pages.shape[-1] != vd:
+        raise KernelError(f"attn_decode: the cache's heads are {k_pages.shape[-1]} and {v_pages.shape[-1]} wide, not {hd} and {vd}")
     if out is None:
-        out = torch.empty((T, H * hd), dtype=torch.bfloat16, device=q.device)
+        out = torch.empty((T, H * vd), dtype=torch.bfloat16, device=q.device)
     part_o = part_ml = None
     if n_splits > 1:
         if scratch is None:
-            scratch = (torch.empty(T * H * n_splits * hd, dtype=torch.float32, device=q.device),
+            scratch = (torch.empty(T * H * n_splits * vd, dtype=torch.float32, device=q.device),
                        torch.empty(T * H * n_splits * 2, dtype=torch.float32, device=q.device))
         part_o, part_ml = scratch
-        if part_o.numel() < T * H * n_splits * hd or part_ml.numel() < T * H * n_splits * 2:
+        if part_o.numel() < T * H * n_splits * vd or part_ml.numel() < T * H * n_splits * 2:
             raise KernelError("attn_decode: scratch too small")
     counters = None
     if n_splits > 1:
@@ -1410,13 +1419,13 @@ def attn_decode(q: torch.Tensor, k_pages, v_pages, page_table, tok_pos, tok_seq,
                              or work.numel() < teams + 1 + 5 * T):
         raise KernelError("attn_decode: the work list must be int32 with teams + 1 offsets and at least a segment per token")
     _check_sink(sink, H)
-    fn = _fn("attn_decode", "lq_attn_decode_capped", [c_void_p, c_int, c_void_p, c_void_p, c_void_p, c_int, c_void_p,
-                                                      c_void_p, c_void_p, c_void_p, c_void_p, c_void_p, c_void_p, c_int,
-                                                      c_int, c_int, c_int, c_int, c_float, c_int, c_int, c_void_p, c_int,
-                                                      c_void_p, c_long, c_int, c_void_p, c_float, c_int, c_void_p])
+    fn = _fn("attn_decode", "lq_attn_decode_vd", [c_void_p, c_int, c_void_p, c_void_p, c_void_p, c_int, c_void_p,
+                                                  c_void_p, c_void_p, c_void_p, c_void_p, c_void_p, c_void_p, c_int,
+                                                  c_int, c_int, c_int, c_int, c_int, c_float, c_int, c_int, c_void_p, c_int,
+                                                  c_void_p, c_long, c_int, c_void_p, c_float, c_int, c_void_p])
     next_p, next_n = _next(next_w, PREFETCH_BYTES_ATTN)
     _check(fn(_p(q), q.stride(0), _p(k_pages), _p(v_pages), _p(page_table), page_table.stride(0), _p(tok_pos),
-              _p(tok_seq), _p(slots), _p(part_o), _p(part_ml), _p(counters), _p(out), T, H, Hkv, hd, page_size,
+              _p(tok_seq), _p(slots), _p(part_o), _p(part_ml), _p(counters), _p(out), T, H, Hkv, hd, vd, page_size,
               float(scale), int(window or 0), n_splits, _p(work), int(teams), next_p, next_n, int(early_loads), _p(sink),
               float(softcap or 0.0), int(keep_first if window else 0), _stream()),
            "attn_decode", 2 if n_splits > 1 and counters is None else 1,

@@ -42,11 +42,11 @@ def linear_bf16(a, weight, out_dtype, residual, emit=None):
     return fn(a, weight.tensor, ops.EPI_F32 if out_dtype == torch.float32 else ops.EPI_BF16, **more)
 
 
-def linear_swiglu_bf16(a, weight):
-    """a . W^T over rows interleaved in blocks of 8 (gate, up), then up * silu(gate)."""
+def linear_swiglu_bf16(a, weight, limit: float = 0.0):
+    """a . W^T over rows interleaved in blocks of 8 (gate, up), then up * silu(gate) (limit: the clamped form of ops.swiglu)."""
     M, K = a.shape
     if K % 8:
         return None
     fn = _decode_kernel(M, weight.N, K)
     more = {"next_w": weight.next_tensor} if fn is ops.gemm_skinny else {}
-    return fn(_rows_for(fn, a), weight.tensor, ops.EPI_SWIGLU, **more)
+    return fn(_rows_for(fn, a), weight.tensor, ops.EPI_SWIGLU, limit=limit, **more)

@@ -127,7 +127,8 @@ class Attention(Mixer):
 
     def step_needs(self):
         return attention_kernels.step_needs(self.runtime.act_dtype, self.hd, self.H, self.Hkv, self.window,
-                                            self.runtime.device, keep_first=self.keep_first, chunk=self.chunk)
+                                            self.runtime.device, keep_first=self.keep_first, chunk=self.chunk,
+                                            vd=self.vd)
 
     def weights(self):
         n = self.names

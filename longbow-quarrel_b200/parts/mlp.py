@@ -5,8 +5,8 @@ Gate and up are one matrix product over the stacked weight [2F, D].
 Options that other designs use: `activation` "gelu_tanh" or "gelu" (the erf form) instead of "silu", or "sigmoid_clamped" with
 a `limit` m (y = W_down (g sigmoid(1.702 g) (u + 1)), g = min(W_gate h, m), u = clamp(W_up h, -m, m)), and
 `bias` (each of the three projections with a bias: y = W_down (act(W_gate h + b_g) * (W_up h + b_u)) + b_d).
-With either the activation is a kernel of its own behind the product (whose sums it reads in 32-bit where
-biases are added); the fused SwiGLU epilogues serve the plain form."""
+With gelu or biases the activation is a kernel of its own behind the product (whose sums it reads in 32-bit where
+biases are added); the products' epilogues serve "silu" and "sigmoid_clamped" without biases."""
 from __future__ import annotations
 
 import torch
@@ -32,7 +32,7 @@ class GatedMLP(FeedForward):
         self.limit = float(limit or 0.0)
         self.runtime, self.D, self.F = runtime, hidden_size, intermediate_size
         self.activation, self.bias = activation, bool(bias)
-        self.plain = activation == "silu" and not self.bias
+        self.plain = activation in ("silu", "sigmoid_clamped") and not self.bias        # what the products' epilogues know
         self.folds_norm = self.plain        # the products of the plain form can take and leave unfinished rows of a norm
         self.names = {**DEFAULT_NAMES, **(names or {})}
         for key in ("gate", "up", "down"):
@@ -71,7 +71,7 @@ class GatedMLP(FeedForward):
         """With `residual` None the output comes back as float32 [T, D] instead of being added."""
         if residual is None:
             if self.plain:
-                return linear.linear(linear.linear_swiglu(h, self.w_gu, self.block), self.w_down, torch.float32)
+                return linear.linear(linear.linear_swiglu(h, self.w_gu, self.block, self.limit), self.w_down, torch.float32)
             gu = linear.linear(h, self.w_gu, torch.float32 if self.bias else self.runtime.act_dtype)
             out = linear.linear(ops.gated_act(gu, self.b_gu, self.activation, self.runtime.act_dtype, self.limit), self.w_down, torch.float32)
             return ops.add_bias(out, self.b_down) if self.bias else out
@@ -83,7 +83,7 @@ class GatedMLP(FeedForward):
             if self.bias:
                 ops.add_bias(residual, self.b_down)
             return None
-        act = linear.linear_swiglu(h, self.w_gu, self.block)
+        act = linear.linear_swiglu(h, self.w_gu, self.block, self.limit)
         if emit is None:
             linear.linear(act, self.w_down, self.runtime.act_dtype, residual=residual)
             return None
