@@ -13,7 +13,9 @@
 //   M_ts = sum_r k_t[r] k_s[r] a_(s+1)[r] ... a_t[r]   and   N_ts (q_t in place of k_t)   what a token of the record adds to that,
 //   u_t = b_t (v_t - S_0^T (A_t k_t) - sum_(s<t) M_ts u_s)          o_t = S_0^T (A_t q_t) + sum_(s<=t) N_ts u_s
 //   S_DC = diag(A_DC) S_0 + sum_s (a_(s+1) ... a_DC k_s) u_s^T
-// Products of decays only, never a quotient, so a decay of zero is harmless.  delta_scan_kernel walks a sequence's
+// Products of decays only, never a quotient, so a decay of zero is harmless.  The state itself takes a decay as
+// S + (a - 1) S with a - 1 from expm1: a decay close to one, rounded and then applied for a thousand tokens, would leave a
+// trace of its rounding in what the first of them wrote.  delta_scan_kernel walks a sequence's
 // records with the state in registers: one round of sums over the key rows per record instead of one per token.
 //
 // Single tokens (one kernel, delta_single_kernel): convolution, unit vectors, the decays' and the output gate's second
@@ -21,21 +23,15 @@
 //
 // The convolution's last inputs are kept per slot as a ring of `taps` rows, the row of position p at p % taps: a step
 // of one token writes a row that it does not read.
-#include "common.cuh"
+#include "tcgen05.cuh"
 
 constexpr int DC = 4;                 // tokens of a record
-constexpr int LPC = 8;                // lanes that share a value column: lane l holds key rows 4 l .. 4 l + 3 of every 32
 constexpr int DSCAL = 4 + 16 + 16;    // scalars of a record: b [4], M [4][4] (t, s), N [4][4]
 
 typedef unsigned long long f2;        // two float32 side by side
 __device__ __forceinline__ f2 fma2(f2 a, f2 b, f2 c) {
     f2 d;
     asm("fma.rn.f32x2 %0, %1, %2, %3;" : "=l"(d) : "l"(a), "l"(b), "l"(c));
-    return d;
-}
-__device__ __forceinline__ f2 mul2(f2 a, f2 b) {
-    f2 d;
-    asm("mul.rn.f32x2 %0, %1, %2;" : "=l"(d) : "l"(a), "l"(b));
     return d;
 }
 __device__ __forceinline__ f2 pack2(float lo, float hi) {
@@ -48,13 +44,13 @@ __device__ __forceinline__ float2 unpack2(f2 v) {
     asm("mov.b64 {%0, %1}, %2;" : "=f"(r.x), "=f"(r.y) : "l"(v));
     return r;
 }
-__device__ __forceinline__ void cp_async16(uint32_t dst, const void* src) {
-    asm volatile("cp.async.cg.shared.global [%0], [%1], 16;" ::"r"(dst), "l"(src) : "memory");
+// An untiled bulk copy into this block's shared memory; both addresses and the size in whole sixteens.
+__device__ __forceinline__ void bulk_load(uint32_t dst, const void* src, uint32_t bytes, uint32_t bar) {
+    asm volatile("cp.async.bulk.shared::cluster.global.mbarrier::complete_tx::bytes [%0], [%1], %2, [%3];"
+                 ::"r"(dst), "l"(src), "r"(bytes), "r"(bar) : "memory");
 }
-__device__ __forceinline__ void cp_async_commit() { asm volatile("cp.async.commit_group;" ::: "memory"); }
-template <int N> __device__ __forceinline__ void cp_async_wait() { asm volatile("cp.async.wait_group %0;" ::"n"(N) : "memory"); }
-__device__ __forceinline__ float sigmoid_f(float x) { return 1.f / (1.f + expf(-x)); }
-__device__ __forceinline__ float silu_f(float x) { return x / (1.f + expf(-x)); }
+__device__ __forceinline__ float sigmoid_f(float x) { return __frcp_rn(1.f + expf(-x)); }
+__device__ __forceinline__ float silu_f(float x) { return x * sigmoid_f(x); }
 __device__ __forceinline__ float softplus_f(float x) { return fmaxf(x, 0.f) + log1pf(expf(-fabsf(x))); }
 
 struct DeltaArgs {
@@ -79,128 +75,154 @@ struct DeltaArgs {
 // A record's rows of key channels are padded with zeros to whole 32s.
 __host__ __device__ __forceinline__ int pad_rows(int dk) { return (dk + 31) / 32 * 32; }
 __host__ __device__ __forceinline__ int pad4(int n) { return (n + 3) / 4 * 4; }
-// Per (record, head): A_t k_t [DC][DKP], A_t q_t [DC][DKP], decayed k_s [DC][DKP], A_DC [DKP], v [DC][pad4(dv)], scalars.
+// Per (record, head): scalars, A_t k_t [DC][DKP], A_t q_t [DC][DKP], decayed k_s [DC][DKP], A_DC - 1 [DKP], v [DC][pad4(dv)].
 __host__ __device__ __forceinline__ int record_floats(int dk, int dv) { return (3 * DC + 1) * pad_rows(dk) + DC * pad4(dv) + DSCAL; }
 // Where the records of sequence b start: unique and never overlapping, whatever the sequences' lengths are.
 __device__ __forceinline__ int first_record(const int* cu_rows, int b) { return cu_rows[b] / DC + b; }
 
-// One block per (record, sequence, value head).
-constexpr int DP_THREADS = 128;
-__global__ void __launch_bounds__(DP_THREADS) delta_prepare_kernel(DeltaArgs a) {
+// A warp per (record, value head), four heads a block; lane l holds the key channels l, l + 32, ... of its head (CPL of them),
+// so every sum over them stays inside the warp.
+constexpr int DP_WARPS = 4;
+template <int CPL>
+__global__ void __launch_bounds__(DP_WARPS * 32) delta_prepare_kernel(DeltaArgs a) {
     pdl_launch_dependents();
-    extern __shared__ float sm[];
-    const int dk = a.dk, dv = a.dv, tid = threadIdx.x, warp = tid >> 5, lane = tid & 31;
-    float* sq = sm;                              // [DC][dk]
-    float* sk = sq + DC * dk;                    // [DC][dk]
-    __shared__ float inv_q[DC], inv_k[DC], red[DP_THREADS / 32][32];
+    const int dk = a.dk, dv = a.dv, lane = threadIdx.x & 31, h = blockIdx.z * DP_WARPS + (threadIdx.x >> 5), b = blockIdx.y;
     pdl_wait();
-    const int b = blockIdx.y, h = blockIdx.z, g = h / (a.H / a.G);
-    const int row0 = a.cu_rows[b], n_rows = a.cu_rows[b + 1] - row0, t0 = blockIdx.x * DC;
+    if (h >= a.H) return;
+    const int g = h / (a.H / a.G), t0 = blockIdx.x * DC, row0 = a.cu_rows[b], n_rows = a.cu_rows[b + 1] - row0;
     if (t0 >= n_rows) return;
     const int n = min(DC, n_rows - t0), taps = a.taps, keep = taps - 1;
     const int pos0 = a.tok_pos[row0];            // the step's first position of this sequence
     const float* ring = a.ring + (size_t)a.slots[b] * taps * a.C;
     const int dkp = pad_rows(dk), dvp = pad4(dv);
     float* rec = a.records + ((size_t)(first_record(a.cu_rows, b) + blockIdx.x) * a.H + h) * record_floats(dk, dv);
-    float* rec_v = rec + (3 * DC + 1) * dkp;
-    float* rec_s = rec_v + DC * dvp;
+    float* vec = rec + DSCAL;
+    float* rec_v = vec + (3 * DC + 1) * dkp;
     // The raw input of channel c at the step's row i (below 0: a row of an earlier step, zero ahead of the sequence).
     auto input = [&](int i, int c) -> float {
         if (i >= 0) return a.rows[(size_t)(row0 + i) * a.stride + c];
         const int p = pos0 + i;
         return p >= 0 ? ring[(size_t)(p % taps) * a.C + c] : 0.f;
     };
-    // Convolution and silu: q and k of the head to shared memory, v straight into the record.
-    for (int e = tid; e < 2 * dk + dvp; e += DP_THREADS) {
-        const int c = e < dk ? g * dk + e : (e < 2 * dk ? a.G * dk + g * dk + (e - dk) : 2 * a.G * dk + h * dv + (e - 2 * dk));
-        float acc[DC] = {};
-        if (e < 2 * dk + dv) {
-            if (taps <= 5) {
-                float w[5], x[DC + 4];
+    // Convolution and silu of channel c for the record's tokens; zero behind the last one.
+    auto conv = [&](int c, float (&y)[DC]) {
 #pragma unroll
-                for (int j = 0; j < 5; ++j) w[j] = j < taps ? a.taps_w[(size_t)j * a.C + c] : 0.f;
+        for (int t = 0; t < DC; ++t) y[t] = 0.f;
+        if (taps == 4 && t0 >= 3 && n == DC) {   // the usual case: four taps, every row the step's own
+            const float* p = a.rows + (size_t)(row0 + t0 - 3) * a.stride + c;
+            float x[DC + 3];
 #pragma unroll
-                for (int i = 0; i < DC + 4; ++i) x[i] = (i < n + keep) ? input(t0 + i - keep, c) : 0.f;
+            for (int i = 0; i < DC + 3; ++i, p += a.stride) x[i] = *p;
+#pragma unroll
+            for (int j = 0; j < 4; ++j) {
+                const float w = a.taps_w[(size_t)j * a.C + c];
+#pragma unroll
+                for (int t = 0; t < DC; ++t) y[t] = fmaf(w, x[t + j], y[t]);
+            }
+#pragma unroll
+            for (int t = 0; t < DC; ++t) y[t] = silu_f(y[t]);
+            return;
+        }
+        if (taps <= 5) {
+            float x[DC + 4];
+#pragma unroll
+            for (int i = 0; i < DC + 4; ++i) x[i] = (i < n + keep) ? input(t0 + i - keep, c) : 0.f;
+#pragma unroll
+            for (int j = 0; j < 5; ++j)
+                if (j < taps) {
+                    const float w = a.taps_w[(size_t)j * a.C + c];
+#pragma unroll
+                    for (int t = 0; t < DC; ++t) y[t] = fmaf(w, x[t + j], y[t]);
+                }
+        } else {
+            for (int j = 0; j < taps; ++j) {
+                const float w = a.taps_w[(size_t)j * a.C + c];
 #pragma unroll
                 for (int t = 0; t < DC; ++t)
-#pragma unroll
-                    for (int j = 0; j < 5; ++j)
-                        if (j < taps) acc[t] = fmaf(w[j], x[t + j], acc[t]);
-            } else {
-                for (int t = 0; t < n; ++t)
-                    for (int j = 0; j < taps; ++j) acc[t] = fmaf(a.taps_w[(size_t)j * a.C + c], input(t0 + t - keep + j, c), acc[t]);
+                    if (t < n) y[t] = fmaf(w, input(t0 + t - keep + j, c), y[t]);
             }
         }
 #pragma unroll
+        for (int t = 0; t < DC; ++t) y[t] = t < n ? silu_f(y[t]) : 0.f;
+    };
+    float q[CPL][DC], k[CPL][DC], z[CPL][DC];
+#pragma unroll
+    for (int i = 0; i < CPL; ++i) {
+        const int r = i * 32 + lane;
+#pragma unroll
         for (int t = 0; t < DC; ++t) {
-            const float y = (t < n && e < 2 * dk + dv) ? silu_f(acc[t]) : 0.f;
-            if (e < dk) sq[t * dk + e] = y;
-            else if (e < 2 * dk) sk[t * dk + e - dk] = y;
-            else rec_v[t * dvp + e - 2 * dk] = y;
+            q[i][t] = k[i][t] = 0.f;
+            z[i][t] = (r < dk && t < n) ? a.z[(size_t)(row0 + t0 + t) * a.H * dk + h * dk + r] + a.z_bias[h * dk + r] : 0.f;
+        }
+        if (r < dk) {
+            conv(g * dk + r, q[i]);
+            conv(a.G * dk + g * dk + r, k[i]);
         }
     }
-    __syncthreads();
-    // Unit vectors: a warp per token.
-    for (int t = warp; t < DC; t += DP_THREADS / 32) {
+    // Unit vectors.
+#pragma unroll
+    for (int t = 0; t < DC; ++t) {
         float s0 = 0.f, s1 = 0.f;
-        for (int r = lane; r < dk; r += 32) {
-            s0 = fmaf(sq[t * dk + r], sq[t * dk + r], s0);
-            s1 = fmaf(sk[t * dk + r], sk[t * dk + r], s1);
+#pragma unroll
+        for (int i = 0; i < CPL; ++i) {
+            s0 = fmaf(q[i][t], q[i][t], s0);
+            s1 = fmaf(k[i][t], k[i][t], s1);
         }
-        s0 = warp_sum(s0);
-        s1 = warp_sum(s1);
-        if (lane == 0) {
-            inv_q[t] = a.q_scale / sqrtf(s0 + a.unit_eps);
-            inv_k[t] = 1.f / sqrtf(s1 + a.unit_eps);
+        s0 = a.q_scale / sqrtf(warp_sum(s0) + a.unit_eps);
+        s1 = 1.f / sqrtf(warp_sum(s1) + a.unit_eps);
+#pragma unroll
+        for (int i = 0; i < CPL; ++i) {
+            q[i][t] *= s0;
+            k[i][t] *= s1;
         }
     }
-    __syncthreads();
-    // Decays, the decayed vectors, and every thread's share of the sixteen sums over the key channels:
+    // Decays, the decayed vectors, and the lane's share of the sixteen sums over the key channels:
     // M_10, M_20, M_21, M_30, M_31, M_32, then N_00, N_10, N_11, N_20, ... N_33.
     float part[16];
 #pragma unroll
     for (int i = 0; i < 16; ++i) part[i] = 0.f;
     const float rate = a.rate[h];
-    for (int r = tid; r < dkp; r += DP_THREADS) {
-        float d[DC], k[DC], q[DC];
 #pragma unroll
-        for (int t = 0; t < DC; ++t) {
-            const bool in = r < dk && t < n;
-            d[t] = 1.f;
-            k[t] = q[t] = 0.f;
-            if (in) {
-                const float z = a.z[(size_t)(row0 + t0 + t) * a.H * dk + h * dk + r] + a.z_bias[h * dk + r];
-                d[t] = expf(-rate * softplus_f(z));
-                k[t] = sk[t * dk + r] * inv_k[t];
-                q[t] = sq[t * dk + r] * inv_q[t];
-            }
-        }
-        float A = 1.f;
+    for (int i = 0; i < CPL; ++i) {
+        const int r = i * 32 + lane;
+        float A = 1.f, log_a = 0.f;
         float kd[DC];                            // k_s times the decays after s, up to the token being walked
         int m = 0, nn = 6;
 #pragma unroll
         for (int t = 0; t < DC; ++t) {
-            A *= d[t];
+            float d = 1.f;
+            if (r < dk && t < n) {
+                const float log_d = -rate * softplus_f(z[i][t]);
+                d = expf(log_d);
+                log_a += log_d;
+            }
+            A *= d;
 #pragma unroll
             for (int s = 0; s < t; ++s) {
-                kd[s] *= d[t];
-                part[m] = fmaf(kd[s], k[t], part[m]);
+                kd[s] *= d;
+                part[m] = fmaf(kd[s], k[i][t], part[m]);
                 ++m;
             }
-            kd[t] = k[t];
+            kd[t] = k[i][t];
 #pragma unroll
             for (int s = 0; s <= t; ++s) {
-                part[nn] = fmaf(kd[s], q[t], part[nn]);
+                part[nn] = fmaf(kd[s], q[i][t], part[nn]);
                 ++nn;
             }
-            rec[t * dkp + r] = A * k[t];
-            rec[(DC + t) * dkp + r] = A * q[t];
+            vec[t * dkp + r] = A * k[i][t];
+            vec[(DC + t) * dkp + r] = A * q[i][t];
         }
 #pragma unroll
-        for (int s = 0; s < DC; ++s) rec[(2 * DC + s) * dkp + r] = kd[s];
-        rec[3 * DC * dkp + r] = r < dk ? A : 0.f;
+        for (int s = 0; s < DC; ++s) vec[(2 * DC + s) * dkp + r] = kd[s];
+        vec[3 * DC * dkp + r] = expm1f(log_a);
     }
-    // Sixteen sums over a warp at once (a lane hands half of its values across and keeps the other half), then the warps.
+    for (int e = lane; e < dvp; e += 32) {
+        float y[DC] = {};
+        if (e < dv) conv(2 * a.G * dk + h * dv + e, y);
+#pragma unroll
+        for (int t = 0; t < DC; ++t) rec_v[t * dvp + e] = y[t];
+    }
+    // Sixteen sums over a warp at once (a lane hands half of its values across and keeps the other half): lane l gets sum l & 15.
 #pragma unroll
     for (int w = 8; w >= 1; w >>= 1) {
         const bool upper = lane & w;
@@ -211,56 +233,63 @@ __global__ void __launch_bounds__(DP_THREADS) delta_prepare_kernel(DeltaArgs a) 
             part[t] = mine + __shfl_xor_sync(0xffffffffu, give, w);
         }
     }
-    red[warp][lane] = part[0] + __shfl_xor_sync(0xffffffffu, part[0], 16);
-    __syncthreads();
-    if (tid < DSCAL) {
-        float v = 0.f;
-        if (tid < 4) {
-            v = tid < n ? sigmoid_f(a.rows[(size_t)(row0 + t0 + tid) * a.stride + a.b_off + h]) : 0.f;
-        } else {
-            const bool is_n = tid >= 20;
-            const int t = (tid - (is_n ? 20 : 4)) >> 2, s = tid & 3;
-            const int at = is_n ? (s <= t ? 6 + t * (t + 1) / 2 + s : -1) : (s < t ? t * (t - 1) / 2 + s : -1);
-            if (at >= 0)
-#pragma unroll
-                for (int w = 0; w < DP_THREADS / 32; ++w) v += red[w][at];
-        }
-        rec_s[tid] = v;
-    }
+    const float sum = part[0] + __shfl_xor_sync(0xffffffffu, part[0], 16);
+    // Lane l writes entry l & 15 of M (l < 16) or N: row t, column s.
+    const int t = (lane >> 2) & 3, s = lane & 3;
+    const int at = lane >= 16 ? (s <= t ? 6 + t * (t + 1) / 2 + s : -1) : (s < t ? t * (t - 1) / 2 + s : -1);
+    const float entry = __shfl_sync(0xffffffffu, sum, at < 0 ? 0 : at);
+    rec[4 + lane] = at < 0 ? 0.f : entry;
+    if (lane < DC) rec[lane] = lane < n ? sigmoid_f(a.rows[(size_t)(row0 + t0 + lane) * a.stride + a.b_off + h]) : 0.f;
 }
 
-// One block per (sequence, value head, some value columns): a warp takes 4 * NC neighbouring columns, eight lanes each
-// with KR of the key rows and NC columns.  A record is brought into shared memory while the ones before it are worked on.
-constexpr int DS_STAGES = 4;
-template <int KR, int NC>
-__global__ void __launch_bounds__(256, 1) delta_scan_kernel(DeltaArgs a, int cols) {
+// One block per (sequence, value head, some value columns): a warp takes 32 / LPC groups of NC neighbouring columns, LPC lanes
+// share a group, each with KR of the key rows.  The last warp brings the records into a ring in shared memory by bulk
+// copies; the others take them from there at their own pace.
+constexpr int DS_STAGES = 6;
+template <int KR, int LPC, int NC>
+__global__ void __launch_bounds__(288, 1) delta_scan_kernel(DeltaArgs a, int cols) {
+    using namespace tc;
     pdl_launch_dependents();
-    constexpr int DKP = KR * LPC, PIECES = KR / 4;
+    constexpr int DKP = KR * LPC, PIECES = KR / 4, SPAN = 4 * LPC;
+    static_assert(2 * DC * NC >= LPC && NC * DC >= 4 && (NC >= 2 * DC * NC / LPC), "every lane is left with sums of one token");
     extern __shared__ __align__(16) float sm[];
-    const int dv = a.dv, dvp = pad4(dv), H = a.H, tid = threadIdx.x, warp = tid >> 5, lane = tid & 31, l = lane & 7;
+    __shared__ __align__(8) uint64_t full[DS_STAGES], empty[DS_STAGES];
+    const int dv = a.dv, dvp = pad4(dv), H = a.H, tid = threadIdx.x, warp = tid >> 5, lane = tid & 31, l = lane & (LPC - 1);
+    const int consumers = (blockDim.x >> 5) - 1;
     const int b = blockIdx.x, h = blockIdx.y, col0 = blockIdx.z * cols;
-    const int vec_floats = (3 * DC + 1) * DKP, stage_floats = vec_floats + DC * cols + DSCAL;
+    constexpr int HEAD = DSCAL + (3 * DC + 1) * DKP;         // a record ahead of its values
+    const int stage_floats = HEAD + DC * cols;
     const int rf = record_floats(a.dk, dv);
-    const int c0 = warp * 4 * NC + (lane >> 3) * NC;         // this thread's first column inside the block's
+    if (tid == 0) {
+        for (int i = 0; i < DS_STAGES; ++i) {
+            mbar_init(smem_u32(&full[i]), 1);
+            mbar_init(smem_u32(&empty[i]), consumers);
+        }
+        mbar_fence_init();
+    }
+    __syncthreads();
     pdl_wait();
     const int row0 = a.cu_rows[b], row1 = a.cu_rows[b + 1], n_rec = (row1 - row0 + DC - 1) / DC;
-    const float* rec0 = a.records + ((size_t)first_record(a.cu_rows, b) * H + h) * rf;
-    const int vcols = min(cols, dvp - col0);                 // columns (whole fours) that the record has
-    auto fetch = [&](int i) {
-        if (i < n_rec) {
-            const float* src = rec0 + (size_t)i * H * rf;
-            const uint32_t dst = (uint32_t)__cvta_generic_to_shared(sm + (i % DS_STAGES) * stage_floats);
-            for (int e = tid; e < vec_floats / 4; e += blockDim.x) cp_async16(dst + e * 16, src + e * 4);
-            const int v4 = vcols / 4;
-            for (int e = tid; e < DC * v4; e += blockDim.x)
-                cp_async16(dst + (vec_floats + (e / v4) * cols + (e % v4) * 4) * 4, src + vec_floats + (e / v4) * dvp + col0 + (e % v4) * 4);
-            for (int e = tid; e < DSCAL / 4; e += blockDim.x)
-                cp_async16(dst + (vec_floats + DC * cols + e * 4) * 4, src + vec_floats + DC * dvp + e * 4);
-        }
-        cp_async_commit();
-    };
+    if (warp == consumers) {
+        if (lane == 0) {
+            const float* src = a.records + ((size_t)first_record(a.cu_rows, b) * H + h) * rf;
+            const uint32_t v_bytes = (uint32_t)min(cols, dvp - col0) * 4;            // whole fours
+            int i = 0;
+            for (; i < n_rec; ++i, src += (size_t)H * rf) {
+                const int s = i % DS_STAGES;
+                if (!mbar_wait(smem_u32(&empty[s]), ((i / DS_STAGES) & 1) ^ 1)) { give_up(1); break; }
+                const uint32_t bar = smem_u32(&full[s]), dst = smem_u32(sm + s * stage_floats);
+                mbar_expect_tx(bar, HEAD * 4 + DC * v_bytes);
+                bulk_load(dst, src, HEAD * 4, bar);
 #pragma unroll
-    for (int i = 0; i < DS_STAGES - 1; ++i) fetch(i);
+                for (int t = 0; t < DC; ++t) bulk_load(dst + (HEAD + t * cols) * 4, src + HEAD + t * dvp + col0, v_bytes, bar);
+            }
+            // After a wait that gave up, the copies that were started must land before the shared memory goes away.
+            if (i < n_rec)
+                for (int back = 1; back <= DS_STAGES && back <= i; ++back) mbar_wait(smem_u32(&full[(i - back) % DS_STAGES]), ((i - back) / DS_STAGES) & 1);
+        }
+        return;
+    }
     // The convolution's last inputs go to the ring; the blocks of a sequence share its channels.  (The records ahead
     // of this kernel were made from the ring as it was.)
     {
@@ -269,29 +298,30 @@ __global__ void __launch_bounds__(256, 1) delta_scan_kernel(DeltaArgs a, int col
         float* ring = a.ring + (size_t)a.slots[b] * taps * a.C;
         for (int i = max(0, n - taps); i < n; ++i) {
             const int p = a.tok_pos[row0 + i];
-            for (int c = lo + tid; c < hi; c += blockDim.x)
+            for (int c = lo + tid; c < hi; c += consumers * 32)
                 ring[(size_t)(p % taps) * a.C + c] = a.rows[(size_t)(row0 + i) * a.stride + c];
         }
     }
+    const int c0 = warp * (32 / LPC) * NC + (lane / LPC) * NC;       // this thread's first column inside the block's
     float* st = a.state + ((size_t)a.slots[b] * H + h) * a.dk * dv;
-    f2 S[KR / 2][NC];                            // rows 32 i + 4 l + {0, 1}, {2, 3} as pairs 2 i, 2 i + 1
+    f2 S[KR / 2][NC];                            // rows SPAN i + 4 l + {0, 1}, {2, 3} as pairs 2 i, 2 i + 1
 #pragma unroll
     for (int i = 0; i < PIECES; ++i)
 #pragma unroll
         for (int p = 0; p < 2; ++p)
 #pragma unroll
             for (int c = 0; c < NC; ++c) {
-                const int r = i * 32 + l * 4 + 2 * p, col = col0 + c0 + c;
+                const int r = i * SPAN + l * 4 + 2 * p, col = col0 + c0 + c;
                 const bool in = c0 + c < cols && col < dv;
                 S[2 * i + p][c] = pack2(in && r < a.dk ? st[(size_t)r * dv + col] : 0.f, in && r + 1 < a.dk ? st[(size_t)(r + 1) * dv + col] : 0.f);
             }
     for (int i = 0; i < n_rec; ++i) {
-        cp_async_wait<DS_STAGES - 2>();
-        __syncthreads();                         // record i is there, and everyone is done with the one before it
-        fetch(i + DS_STAGES - 1);
-        const float* rec = sm + (i % DS_STAGES) * stage_floats;
-        const float* vs = rec + vec_floats + c0;
-        const float4* sc = reinterpret_cast<const float4*>(rec + vec_floats + DC * cols);
+        const int stage = i % DS_STAGES;
+        if (!mbar_wait(smem_u32(&full[stage]), (i / DS_STAGES) & 1)) { give_up(2); break; }
+        const float* rec = sm + stage * stage_floats;
+        const float* vec = rec + DSCAL + l * 4;
+        const float* vs = rec + HEAD + c0;
+        const float4* sc = reinterpret_cast<const float4*>(rec);
         f2 acc2[2 * DC][NC];
 #pragma unroll
         for (int t = 0; t < 2 * DC; ++t)
@@ -301,87 +331,97 @@ __global__ void __launch_bounds__(256, 1) delta_scan_kernel(DeltaArgs a, int col
         for (int j = 0; j < PIECES; ++j)
 #pragma unroll
             for (int t = 0; t < 2 * DC; ++t) {
-                const ulonglong2 x = *reinterpret_cast<const ulonglong2*>(rec + t * DKP + j * 32 + l * 4);
+                const ulonglong2 x = *reinterpret_cast<const ulonglong2*>(vec + t * DKP + j * SPAN);
 #pragma unroll
                 for (int c = 0; c < NC; ++c) {
                     acc2[t][c] = fma2(S[2 * j][c], x.x, acc2[t][c]);
                     acc2[t][c] = fma2(S[2 * j + 1][c], x.y, acc2[t][c]);
                 }
             }
-        float mine[NC], u[DC][NC];
+        // What token t reads from the state with k (sum t * NC + c of column c) and with q (sum (DC + t) * NC + c) is added up
+        // over the LPC lanes of the columns: in each step a lane hands half of its sums across and keeps the other half, so
+        // lane l is left with the sums PER l .. PER l + PER - 1.
+        constexpr int PER = 2 * DC * NC / LPC;
+        float acc[2 * DC * NC];
 #pragma unroll
-        for (int c = 0; c < NC; ++c) {
-            float acc[2 * DC];
+        for (int t = 0; t < 2 * DC; ++t)
 #pragma unroll
-            for (int t = 0; t < 2 * DC; ++t) {
+            for (int c = 0; c < NC; ++c) {
                 const float2 f = unpack2(acc2[t][c]);
-                acc[t] = f.x + f.y;
+                acc[t * NC + c] = f.x + f.y;
             }
-            // Eight sums over the column's eight lanes: lane l is left with sum number l.
 #pragma unroll
-            for (int w = 4; w >= 1; w >>= 1) {
-                const bool upper = l & w;
+        for (int w = LPC / 2; w >= 1; w >>= 1) {
+            const bool upper = l & w;
+            const int half = PER * w;
 #pragma unroll
-                for (int t = 0; t < w; ++t) {
-                    const float give = upper ? acc[t] : acc[t + w];
-                    const float keep = upper ? acc[t + w] : acc[t];
-                    acc[t] = keep + __shfl_xor_sync(0xffffffffu, give, w);
-                }
+            for (int v = 0; v < half; ++v) {
+                const float give = upper ? acc[v] : acc[v + half];
+                const float keep = upper ? acc[v + half] : acc[v];
+                acc[v] = keep + __shfl_xor_sync(0xffffffffu, give, w);
             }
-            mine[c] = acc[0];
         }
         const float4 beta = sc[0], m1 = sc[2], m2 = sc[3], m3 = sc[4];
+        float u[DC][NC];
 #pragma unroll
         for (int c = 0; c < NC; ++c) {
             float r[DC];
 #pragma unroll
-            for (int t = 0; t < DC; ++t) r[t] = vs[t * cols + c] - __shfl_sync(0xffffffffu, mine[c], (lane & 24) + t);
+            for (int t = 0; t < DC; ++t)
+                r[t] = vs[t * cols + c] - __shfl_sync(0xffffffffu, acc[(t * NC + c) % PER], (lane & ~(LPC - 1)) + (t * NC + c) / PER);
             u[0][c] = beta.x * r[0];
             u[1][c] = beta.y * (r[1] - m1.x * u[0][c]);
             u[2][c] = beta.z * (r[2] - m2.x * u[0][c] - m2.y * u[1][c]);
             u[3][c] = beta.w * (r[3] - m3.x * u[0][c] - m3.y * u[1][c] - m3.z * u[2][c]);
         }
-        if (l >= DC) {
-            const int t = l - DC, row = row0 + i * DC + t;
+        if (l >= LPC / 2) {                      // the lanes that hold sums with q
+            const int t = (l * PER) / NC - DC, cc = (l * PER) % NC, row = row0 + i * DC + t;
             const float4 nt = sc[5 + t];
 #pragma unroll
-            for (int c = 0; c < NC; ++c)
-                if (row < row1 && c0 + c < cols && col0 + c0 + c < dv)
-                    a.raw[((size_t)row * H + h) * dv + col0 + c0 + c] = mine[c] + nt.x * u[0][c] + nt.y * u[1][c] + nt.z * u[2][c] + nt.w * u[3][c];
-        }
+            for (int v = 0; v < PER; ++v) {
+                const int col = c0 + cc + v;
+                // u of column cc + v: picked without indexing registers by a number that is not known when compiling
+                float u0 = u[0][v], u1 = u[1][v], u2 = u[2][v], u3 = u[3][v];
 #pragma unroll
-        for (int j = 0; j < PIECES; ++j) {
-            const ulonglong2 A = *reinterpret_cast<const ulonglong2*>(rec + 3 * DC * DKP + j * 32 + l * 4);
-#pragma unroll
-            for (int c = 0; c < NC; ++c) {
-                S[2 * j][c] = mul2(S[2 * j][c], A.x);
-                S[2 * j + 1][c] = mul2(S[2 * j + 1][c], A.y);
+                for (int c = v + PER; c < NC; c += PER)
+                    if (cc + v == c) { u0 = u[0][c]; u1 = u[1][c]; u2 = u[2][c]; u3 = u[3][c]; }
+                if (row < row1 && col < cols && col0 + col < dv)
+                    a.raw[((size_t)row * H + h) * dv + col0 + col] = acc[v] + nt.x * u0 + nt.y * u1 + nt.z * u2 + nt.w * u3;
             }
         }
+        f2 uu[DC][NC];
 #pragma unroll
-        for (int s = 0; s < DC; ++s) {
-            f2 uu[NC];
+        for (int s = 0; s < DC; ++s)
 #pragma unroll
-            for (int c = 0; c < NC; ++c) uu[c] = pack2(u[s][c], u[s][c]);
+            for (int c = 0; c < NC; ++c) uu[s][c] = pack2(u[s][c], u[s][c]);
 #pragma unroll
-            for (int j = 0; j < PIECES; ++j) {
-                const ulonglong2 x = *reinterpret_cast<const ulonglong2*>(rec + (2 * DC + s) * DKP + j * 32 + l * 4);
+        for (int j = 0; j < PIECES; ++j) {
+            const ulonglong2 E = *reinterpret_cast<const ulonglong2*>(vec + 3 * DC * DKP + j * SPAN);
+#pragma unroll
+            for (int c = 0; c < NC; ++c) {
+                S[2 * j][c] = fma2(S[2 * j][c], E.x, S[2 * j][c]);
+                S[2 * j + 1][c] = fma2(S[2 * j + 1][c], E.y, S[2 * j + 1][c]);
+            }
+#pragma unroll
+            for (int s = 0; s < DC; ++s) {
+                const ulonglong2 x = *reinterpret_cast<const ulonglong2*>(vec + (2 * DC + s) * DKP + j * SPAN);
 #pragma unroll
                 for (int c = 0; c < NC; ++c) {
-                    S[2 * j][c] = fma2(x.x, uu[c], S[2 * j][c]);
-                    S[2 * j + 1][c] = fma2(x.y, uu[c], S[2 * j + 1][c]);
+                    S[2 * j][c] = fma2(x.x, uu[s][c], S[2 * j][c]);
+                    S[2 * j + 1][c] = fma2(x.y, uu[s][c], S[2 * j + 1][c]);
                 }
             }
         }
+        __syncwarp();
+        if (lane == 0) mbar_arrive(smem_u32(&empty[stage]));
     }
-    cp_async_wait<0>();
 #pragma unroll
     for (int i = 0; i < PIECES; ++i)
 #pragma unroll
         for (int p = 0; p < 2; ++p)
 #pragma unroll
             for (int c = 0; c < NC; ++c) {
-                const int r = i * 32 + l * 4 + 2 * p, col = col0 + c0 + c;
+                const int r = i * SPAN + l * 4 + 2 * p, col = col0 + c0 + c;
                 if (c0 + c < cols && col < dv) {
                     const float2 f = unpack2(S[2 * i + p][c]);
                     if (r < a.dk) st[(size_t)r * dv + col] = f.x;
@@ -390,21 +430,30 @@ __global__ void __launch_bounds__(256, 1) delta_scan_kernel(DeltaArgs a, int col
             }
 }
 
-static int scan_columns(int B, int H, int dv) {
-    // Columns of a block: 32, or fewer where that leaves multiprocessors without a block.
-    int cols = 32;
-    while (cols > 8 && (long)B * H * ((dv + cols - 1) / cols) < 100) cols >>= 1;
+static int scan_columns(int B, int H, int dv, int least, int most) {
+    // Columns of a block: as many as it has warps for, or fewer where that leaves multiprocessors without a block.
+    int cols = most;
+    while (cols / 2 >= least && cols % 8 == 0 && (long)B * H * ((dv + cols - 1) / cols) < 100) cols >>= 1;
     return cols;
 }
 
-template <int KR, int NC>
+template <int KR, int LPC, int NC>
 static int scan_launch(const DeltaArgs& a, int B, cudaStream_t stream) {
-    const int cols = scan_columns(B, a.H, a.dv), threads = cols / (4 * NC) * 32;
-    const size_t smem = (size_t)DS_STAGES * ((3 * DC + 1) * KR * LPC + DC * cols + DSCAL) * sizeof(float);
+    constexpr int PER_WARP = 32 / LPC * NC;
+    const int cols = scan_columns(B, a.H, a.dv, PER_WARP, 32 < 8 * PER_WARP ? 32 : 8 * PER_WARP), threads = (cols / PER_WARP + 1) * 32;
+    const size_t smem = (size_t)DS_STAGES * (DSCAL + (3 * DC + 1) * KR * LPC + DC * cols) * sizeof(float);
     if (smem > 48 * 1024 &&
-        cudaFuncSetAttribute(delta_scan_kernel<KR, NC>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem) != cudaSuccess)
+        cudaFuncSetAttribute(delta_scan_kernel<KR, LPC, NC>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem) != cudaSuccess)
         return lq_launch_status();
-    return launch_pdl(delta_scan_kernel<KR, NC>, dim3(B, a.H, (a.dv + cols - 1) / cols), dim3(threads), smem, stream, a, cols);
+    // Not ahead of its time: blocks that start while the records are still being made take what room they find, several on
+    // one multiprocessor, and stay there; started afterwards they spread out (measured: half the time).
+    return launch_after(delta_scan_kernel<KR, LPC, NC>, dim3(B, a.H, (a.dv + cols - 1) / cols), dim3(threads), smem, stream, a, cols);
+}
+
+template <int CPL>
+static int prepare_launch(const DeltaArgs& a, int B, int max_new, cudaStream_t stream) {
+    return launch_pdl(delta_prepare_kernel<CPL>, dim3((max_new + DC - 1) / DC, B, (a.H + DP_WARPS - 1) / DP_WARPS), dim3(DP_WARPS * 32), 0,
+                      stream, a);
 }
 
 // Floats of scratch that a step with prompts needs for its records.
@@ -421,19 +470,27 @@ LQ_EXPORT int lq_delta_prompt(const float* rows, int stride, int b_off, const fl
     if (dk < 1 || dk > 256 || dv < 1 || G < 1 || H % G || taps < 1) return LQ_BAD_SIZE;
     DeltaArgs a{rows, stride, b_off, taps_w, taps, 2 * G * dk + H * dv, ring, z, z_bias, rate, state, cu_rows, slots, tok_pos,
                 records, raw, H, G, dk, dv, q_scale, unit_eps};
-    const int rc = launch_pdl(delta_prepare_kernel, dim3((max_new + DC - 1) / DC, B, H), dim3(DP_THREADS), (size_t)2 * DC * dk * sizeof(float),
-                              stream, a);
-    if (rc != LQ_OK) return rc;
-    const int kr = pad_rows(dk) / LPC;
-    if (kr <= 4) return scan_launch<4, 2>(a, B, stream);
-    if (kr <= 8) return scan_launch<8, 2>(a, B, stream);
-    if (kr <= 12) return scan_launch<12, 2>(a, B, stream);
-    if (kr <= 16) return scan_launch<16, 2>(a, B, stream);
-    if (kr <= 20) return scan_launch<20, 1>(a, B, stream);
-    if (kr <= 24) return scan_launch<24, 1>(a, B, stream);
-    if (kr <= 28) return scan_launch<28, 1>(a, B, stream);
-    return scan_launch<32, 1>(a, B, stream);
+    int rc = LQ_BAD_SIZE;
+    const int cpl = pad_rows(dk) / 32;
+#define LQ_GO(CPL, ...) case CPL: \
+        rc = prepare_launch<CPL>(a, B, max_new, stream); \
+        return rc != LQ_OK ? rc : scan_launch<__VA_ARGS__>(a, B, stream)
+    switch (cpl) {
+        LQ_GO(1, 4, 8, 2);
+        LQ_GO(2, 8, 8, 2);
+        LQ_GO(3, 12, 8, 2);
+        LQ_GO(4, 16, 8, 2);
+        LQ_GO(5, 20, 8, 2);
+        LQ_GO(6, 24, 8, 2);
+        LQ_GO(7, 28, 8, 2);
+        LQ_GO(8, 32, 8, 2);
+    }
+#undef LQ_GO
+    return rc;
 }
+
+LQ_EXPORT int lq_delta_status() { return tc::status_read(); }
+LQ_EXPORT int* lq_delta_status_word() { return tc::status_word(); }
 
 // ------------------------------------------------------------------ one token per sequence
 struct DeltaSingleArgs {
@@ -444,7 +501,8 @@ struct DeltaSingleArgs {
     int ra_ld, rg_ld;            // row lengths (whole eights; what lies beyond ra, rg is zero)
     const float* norm_w;         // [dv]
     float norm_eps;
-    void* out;                   // [B, H * dv]
+    void* out;                   // [B, H * dv], float32 or bfloat16
+    int out_bf16;
     int cg;                      // threads side by side along a row of the state
 };
 
@@ -477,7 +535,7 @@ template <> __device__ __forceinline__ float dot_row<__nv_bfloat16>(const __nv_b
 // neighbouring columns of up to KR rows in registers between the read and the write.  Columns beyond cg * VW take
 // another turn.
 constexpr int DT_THREADS = 256;
-template <typename T, typename TW, int KR, int VW>
+template <typename TW, int KR, int VW>
 __global__ void __launch_bounds__(DT_THREADS) delta_single_kernel(DeltaSingleArgs s) {
     pdl_launch_dependents();
     extern __shared__ __align__(16) float sm[];
@@ -487,7 +545,7 @@ __global__ void __launch_bounds__(DT_THREADS) delta_single_kernel(DeltaSingleArg
     const int cg = s.cg, rg = DT_THREADS / cg, group = tid / cg, cl = tid % cg;
     float* sq = sm;                              // [dk]
     float* sk = sq + dk;                         // [dk]
-    float* sa = sk + dk;                         // [dk] decays
+    float* sa = sk + dk;                         // [dk] decays, less one
     float* sv = sa + dk;                         // [dv]
     float* so = sv + dv;                         // [dv]
     float* sgate = so + dv;                      // [dv]
@@ -552,7 +610,7 @@ __global__ void __launch_bounds__(DT_THREADS) delta_single_kernel(DeltaSingleArg
     for (int e = tid; e < dk + dv; e += DT_THREADS) {
         if (e < dk) {
             const float z = dot_row<TW>((const TW*)s.a2 + (size_t)(h * dk + e) * s.ra_ld, xa, s.ra_ld) + a.z_bias[h * dk + e];
-            sa[e] = expf(-a.rate[h] * softplus_f(z));
+            sa[e] = expm1f(-a.rate[h] * softplus_f(z));
         } else {
             sgate[e - dk] = sigmoid_f(dot_row<TW>((const TW*)s.g2 + (size_t)(h * dv + e - dk) * s.rg_ld, xg, s.rg_ld));
         }
@@ -577,7 +635,7 @@ __global__ void __launch_bounds__(DT_THREADS) delta_single_kernel(DeltaSingleArg
                 const float d = sa[r], k = sk[r], q = sq[r];
 #pragma unroll
                 for (int v = 0; v < VW; ++v) {
-                    S[i][v] *= d;
+                    S[i][v] = fmaf(S[i][v], d, S[i][v]);
                     rk[v] = fmaf(S[i][v], k, rk[v]);
                     rq[v] = fmaf(S[i][v], q, rq[v]);
                 }
@@ -633,11 +691,15 @@ __global__ void __launch_bounds__(DT_THREADS) delta_single_kernel(DeltaSingleArg
 #pragma unroll
     for (int w = 0; w < DT_THREADS / 32; ++w) total += part[w];
     const float inv = 1.f / sqrtf(total / (float)dv + s.norm_eps);
-    T* out = (T*)s.out + ((size_t)row * H + h) * dv;
-    for (int d = tid; d < dv; d += DT_THREADS) out[d] = from_f32<T>(so[d] * inv * s.norm_w[d] * sgate[d]);
+    const size_t at = ((size_t)row * H + h) * dv;
+    for (int d = tid; d < dv; d += DT_THREADS) {
+        const float y = so[d] * inv * s.norm_w[d] * sgate[d];
+        if (s.out_bf16) ((__nv_bfloat16*)s.out)[at + d] = __float2bfloat16_rn(y);
+        else ((float*)s.out)[at + d] = y;
+    }
 }
 
-template <typename T, typename TW>
+template <typename TW>
 static int single_launch(DeltaSingleArgs& s, int B, cudaStream_t stream) {
     const int dk = s.d.dk, dv = s.d.dv, vw = dv % 4 == 0 ? 4 : 1;
     // As many threads along a row as there are columns, unless that leaves a thread too many rows.
@@ -654,11 +716,11 @@ static int single_launch(DeltaSingleArgs& s, int B, cudaStream_t stream) {
         return launch_pdl(kernel, dim3(B, s.d.H), dim3(DT_THREADS), smem, stream, s);
     };
     if (vw == 4) {
-        if (kr <= 4) return go(delta_single_kernel<T, TW, 4, 4>);
-        if (kr <= 8) return go(delta_single_kernel<T, TW, 8, 4>);
-        return go(delta_single_kernel<T, TW, 16, 4>);
+        if (kr <= 4) return go(delta_single_kernel<TW, 4, 4>);
+        if (kr <= 8) return go(delta_single_kernel<TW, 8, 4>);
+        return go(delta_single_kernel<TW, 16, 4>);
     }
-    return go(delta_single_kernel<T, TW, 16, 1>);
+    return go(delta_single_kernel<TW, 16, 1>);
 }
 
 // One token per sequence (row cu_rows[b] of rows): out [B, H dv], normed and gated.
@@ -672,11 +734,9 @@ LQ_EXPORT int lq_delta_single(const float* rows, int stride, int b_off, const fl
         return LQ_BAD_SIZE;
     DeltaSingleArgs s{{rows, stride, b_off, taps_w, taps, 2 * G * dk + H * dv, ring, nullptr, z_bias, rate, state, cu_rows, slots, tok_pos,
                        nullptr, nullptr, H, G, dk, dv, q_scale, unit_eps},
-                      a_off, ra, g_off, rg, a2, g2, ra_ld, rg_ld, norm_w, norm_eps, out, 1};
-    typedef __nv_bfloat16 bf;
-    if (out_dtype == LQ_F32 && w_dtype == LQ_F32) return single_launch<float, float>(s, B, stream);
-    if (out_dtype == LQ_F32 && w_dtype == LQ_BF16) return single_launch<float, bf>(s, B, stream);
-    if (out_dtype == LQ_BF16 && w_dtype == LQ_F32) return single_launch<bf, float>(s, B, stream);
-    if (out_dtype == LQ_BF16 && w_dtype == LQ_BF16) return single_launch<bf, bf>(s, B, stream);
+                      a_off, ra, g_off, rg, a2, g2, ra_ld, rg_ld, norm_w, norm_eps, out, out_dtype == LQ_BF16, 1};
+    if (out_dtype != LQ_F32 && out_dtype != LQ_BF16) return LQ_BAD_DTYPE;
+    if (w_dtype == LQ_F32) return single_launch<float>(s, B, stream);
+    if (w_dtype == LQ_BF16) return single_launch<__nv_bfloat16>(s, B, stream);
     return LQ_BAD_DTYPE;
 }

@@ -90,7 +90,7 @@ _WATCHED = {"gemm_tc": {1: "the TMA producer waited for a free stage", 2: "the p
                         3: "the product issuer waited for a stage's copies", 4: "the epilogue waited for an accumulator"},
             "gemm_pair": {1: "a TMA producer waited for a free stage", 2: "the product issuer waited for a free accumulator",
                           3: "the product issuer waited for a stage's copies", 4: "an epilogue waited for an accumulator"},
-            "attn_prefill_tc": {}}
+            "attn_prefill_tc": {}, "delta": {1: "the copying warp waited for a free stage", 2: "a warp waited for a record"}}
 _status_words: dict[str, object] = {}
 
 

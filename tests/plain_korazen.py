@@ -59,10 +59,15 @@ def load_folder(folder):
 # --------------------------------------------------------------------------- small pieces
 
 _STORAGE = None        # set by forward(storage=...): the dtype in which activations are kept between operations
+_NOISE = None          # set by forward(noise=...): (relative size, generator)
+_MARGINS = None        # set by forward(margins=...): receives how firmly every position of a delta-rule layer reads its state
 
 
 def _st(x: torch.Tensor) -> torch.Tensor:
-    """What a tensor looks like after it was stored in the storage dtype between two operations."""
+    """What a tensor looks like after it was stored in the storage dtype between two operations, or moved as much by chance."""
+    if _NOISE is not None:
+        size, gen = _NOISE
+        x = x * (1.0 + size * (2.0 * torch.rand(x.shape, generator=gen, dtype=x.dtype) - 1.0))
     return x if _STORAGE is None else x.to(_STORAGE).to(x.dtype)
 
 
@@ -129,11 +134,17 @@ def delta_rule(q, k, v, b, a, state: list | None = None) -> torch.Tensor:
     T, H, dim = q.shape
     S = torch.zeros(H, dim, v.shape[2], dtype=q.dtype)
     o = torch.zeros_like(v)
+    margins = torch.zeros(T, dtype=torch.float64)
     for t in range(T):
         S = a[t][:, :, None] * S
         u = b[t][:, None] * (v[t] - torch.einsum("hdv,hd->hv", S, k[t]))
         S = S + k[t][:, :, None] * u[:, None, :]
         o[t] = torch.einsum("hdv,hd->hv", S, q[t])
+        if _MARGINS is not None:
+            whole = torch.einsum("hdv,hd->hv", S.abs(), q[t].abs())
+            margins[t] = float((o[t].norm(dim=1) / whole.norm(dim=1).clamp_min(1e-30)).min())
+    if _MARGINS is not None:
+        _MARGINS.append(margins)
     if state is not None:
         state.append(S)
     return o
@@ -210,11 +221,15 @@ def _sub(weights: dict, prefix: str) -> dict:
     return {n[len(prefix):]: t for n, t in weights.items() if n.startswith(prefix)}
 
 
-def forward(cfg: dict, weights: dict, tokens, dtype=torch.float64, storage=None, layers_out: list | None = None) -> torch.Tensor:
+def forward(cfg: dict, weights: dict, tokens, dtype=torch.float64, storage=None, layers_out: list | None = None,
+            noise: tuple | None = None, margins: list | None = None) -> torch.Tensor:
     """Logits [T, vocab] of one sequence.  storage: the dtype activations are kept in between operations (None: dtype).
-    layers_out: receives the residual stream after every layer."""
-    global _STORAGE
-    _STORAGE = storage
+    layers_out: receives the residual stream after every layer.  noise = (size, seed): what is stored between operations is
+    moved by a relative amount drawn from +-size.  margins: receives for every delta-rule layer how far each position's
+    weakest read-out is from cancelling, |S^T q| over |S|^T |q|."""
+    global _STORAGE, _NOISE, _MARGINS
+    _STORAGE, _MARGINS = storage, margins
+    _NOISE = (noise[0], torch.Generator().manual_seed(noise[1])) if noise is not None else None
     try:
         eps = cfg["norm"]["eps"]
         W = {n: t.to(dtype) for n, t in weights.items()}
@@ -229,7 +244,7 @@ def forward(cfg: dict, weights: dict, tokens, dtype=torch.float64, storage=None,
                 layers_out.append(x.clone())
         return _st(unit_rms(x, eps) * W["final.norm"]) @ W["head"].T * cfg["logit_scale"]
     finally:
-        _STORAGE = None
+        _STORAGE = _NOISE = _MARGINS = None
 
 
 def greedy(cfg: dict, weights: dict, prompt, n_new: int) -> list[int]:
