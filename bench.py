@@ -400,6 +400,8 @@ def design_bench(args) -> int:
         return raritar_bench(args)
     if args.design == "lavutar":
         return lavutar_bench(args)
+    if args.design == "korazen":
+        return korazen_bench(args)
     return fetorax_bench(args)
 
 
@@ -797,6 +799,117 @@ def lavutar_bench(args) -> int:
     return 0
 
 
+def korazen_config(size: str, block: int) -> dict:
+    """Four layers, each with a clamped gated feed-forward: the gated delta rule, two sides side by side (attention over
+    blocks of positions, linear attention with fixed decays), the delta rule, two sides whose attention has values twice
+    as wide as its keys."""
+    width, heads, kv, dim, ff = DESIGN_SIZES[size]
+    dense = {"kind": "dense", "ff": ff, "limit": 7.0}
+    delta = {"heads": heads, "kv_heads": heads, "dim": dim, "vdim": dim, "conv": 4, "rank": 64, "gate_rank": 64}
+
+    def two(vdim):
+        return {"left": {"heads": heads, "kv_heads": kv, "dim": dim, "vdim": vdim, "scale": dim ** -0.5, "mask": {"size": block},
+                         "rot": {"dims": dim, "base": 1e5}},
+                "right": {"heads": heads, "dim": dim, "vdim": dim, "decay": [1.0 - 2.0 ** -(4 + h % 8) for h in range(heads)]}}
+    layers = [{"type": kind, "mixer": m, "mlp": dense} for kind, m in (("channel_delta", delta), ("parallel", two(dim)), ("channel_delta", delta),
+                                                                       ("parallel", two(2 * dim)))]
+    return {"architecture": "Korazen", "vocab": DESIGN_VOCAB, "width": width, "norm": {"eps": 1e-5}, "logit_scale": 1.0, "layers": layers,
+            "max_positions": 8192}
+
+
+def lavutar_twin(size: str, block: int) -> dict:
+    """A Lavutar model of the same width, heads, depth and feed-forward width for `korazen_config`: two sides (softmax
+    attention over all positions, a decay for every key channel), attention over blocks, two sides, attention over
+    blocks with values twice as wide as keys, each with a gated feed-forward."""
+    width, heads, kv, dim, ff = DESIGN_SIZES[size]
+    cfg = lavutar_config(size, block, block)
+    blocks, two = cfg["layers"][0], cfg["layers"][3]
+    wide = {**blocks, "mixer": {**blocks["mixer"], "vdim": 2 * dim}}
+    return {**{k: v for k, v in cfg.items() if k != "loop"}, "layers": [two, blocks, two, wide]}
+
+
+def korazen_bench(args) -> int:
+    """Prefill and decode of a Korazen model of realistic layer sizes beside the closest model the library has, a Lavutar
+    model of the same sizes (random weights, vocabulary 32,000): tokens a second, what every kind of kernel adds to a
+    prompt step and to a decode step, and how many times their roofline the design's kernels take, beside the like
+    kernel of the other model."""
+    import numpy as np
+    import torch
+
+    from longbow_quarrel_b200.engine import Engine
+    peaks, peaks_from = load_peaks()
+    K, W = args.steps, max(3, args.warmup)
+    T, B, ctx, block = PREFILL_TOKENS, BATCH, 2048, 1280       # (blocks that decoded positions stand in the middle of)
+    hbm, tensor = peaks["hbm_gbs"] * 1e9, peaks["bf16_tflops"] * 1e12
+    rng = np.random.default_rng(0)
+    sampler = ClockSampler()
+    sampler.start()
+    out = {}
+    for size in args.sizes.split(","):
+        width, heads, kv, dim, ff = DESIGN_SIZES[size]
+        configs = {"korazen": korazen_config(size, block), "lavutar": lavutar_twin(size, block)}
+        res = {name: _design_run(torch, np, Engine, cfg, name, T, B, ctx, K, W, rng) for name, cfg in configs.items()}
+
+        def per_launch(kinds, *names):
+            n = sum(kinds[k][0] for k in names if k in kinds)
+            return sum(kinds[k][1] for k in names if k in kinds) / n if n else None
+
+        def roof(us, nbytes, flops=0.0):
+            """(us a launch, times its roofline)"""
+            return [round(us, 1), round(us / (max(nbytes / hbm, flops / tensor) * 1e6), 2)] if us else None
+        k, v = res["korazen"], res["lavutar"]
+        kp, kd, vp, vd = k["prefill_kernels_us"], k["decode_kernels_us"], v["prefill_kernels_us"], v["decode_kernels_us"]
+        full, seen = T * (T + 1) / 2, block * (block + 1) / 2 + (T - block) * (T - block + 1) / 2
+        per_head = T * heads * dim
+        state = B * heads * dim * dim * 4.0 * 2
+        # The delta rule's two prompt kernels together: q, k, v, decays and the raw outputs, 32-bit each; read-out, correction
+        # and write of a dim x dim state per head and token.
+        delta = sum(kp[n][1] for n in ("delta_prepare", "delta_scan") if n in kp) / 2 or None
+        linear = sum(kp[n][1] for n in ("linear_prepare", "linear_records") if n in kp) / 2 or None
+        kv_seen, kv_all = B * ((ctx + W + K // 2) % block + 1) * kv * dim * 2.0, B * ctx * kv * dim * 2.0
+        join_bytes = T * width * (4 + 8 + 2.0)
+        times = {
+            "prefill": {
+                "delta rule (records + scan)": roof(delta, per_head * 5 * 4.0, 6.0 * per_head * dim),
+                "lavutar scan with channel decays": roof(per_launch(vp, "linear_scan"), per_head * (3 * 2 + 4 + 4.0), 4.0 * per_head * dim),
+                "fixed-decay scan (records + scan)": roof(linear, per_head * (3 * 2 + 4.0), 4.0 * per_head * dim),
+                "attention, values as wide as keys (tcgen05)": roof(per_launch(kp, "attn_prefill_two", "attn_prefill_tc"), per_head * 6.0, 4.0 * heads * dim * seen),
+                "lavutar attention, values as wide as keys (blocks / all)": roof(per_launch(vp, "attn_prefill_two", "attn_prefill_tc"), per_head * 6.0,
+                                                                                 4.0 * heads * dim * (seen + 2 * full) / 3),
+                "attention, values twice as wide (mma.sync)": roof(per_launch(kp, "attn_prefill"), per_head * 10.0, 6.0 * heads * dim * seen),
+                "lavutar attention, values twice as wide (mma.sync)": roof(per_launch(vp, "attn_prefill"), per_head * 10.0, 6.0 * heads * dim * seen),
+                "branch norms + add + rows": roof(per_launch(kp, "join"), (6 * join_bytes + 2 * (join_bytes + 4.0 * T * width)) / 8),
+                "lavutar layer norm": roof(per_launch(vp, "layernorm", "layernorm_vec"), T * width * (7 * 6.0 + 2 * 18.0) / 9),
+                "biases + unit norms + rotation + cache write": roof(per_launch(kp, "rope_partial"), T * (heads + 1.5 * kv) * dim * 6.0 + T * kv * dim * 3.0),
+                "lavutar unit norms + rotation + cache write": roof(per_launch(vp, "rope_partial"), T * (heads + 2 * kv) * dim * 6.0),
+            },
+            "decode": {
+                "delta rule (one kernel)": roof(per_launch(kd, "delta_single"), state + 2 * heads * dim * 64 * 2.0),
+                "lavutar scan with channel decays": roof(per_launch(vd, "linear_scan_single"), state),
+                "fixed-decay scan": roof(per_launch(kd, "linear_scan_single"), state),
+                "attention (both value sizes)": roof(per_launch(kd, "attn_decode"), kv_seen * 2.5),
+                "lavutar attention": roof(per_launch(vd, "attn_decode"), (2 * kv_all * 2 + kv_seen * 2 + kv_seen * 3) / 4),
+                "branch norms + add + rows": roof(per_launch(kd, "join"), B * width * 14.0),
+                "lavutar layer norm": roof(per_launch(vd, "layernorm", "layernorm_vec"), B * width * 8.0),
+            },
+        }
+
+        def small(kinds):
+            names = {"head_norm_gate", "head_norm_gate_wide", "gate_mul", "take_columns", "embedding_norm", "gemm_plain", "gated_act", "gated_act_vec", "rope_partial"}
+            return {n: round(kinds[n][1] / kinds[n][0], 1) for n in kinds if n in names}
+        out[size] = {"korazen": k, "lavutar": v, "us_and_times_the_roofline": times,
+                     "small_kernels_us_per_launch": {"prefill": small(kp), "decode": small(kd), "lavutar_prefill": small(vp), "lavutar_decode": small(vd)},
+                     "korazen_over_lavutar": {"prefill": round(k["prefill_tokens_per_s"] / v["prefill_tokens_per_s"], 3),
+                                              "decode": round(k["decode_tokens_per_s"] / v["decode_tokens_per_s"], 3)}}
+    clocks = sampler.stop()
+    print(json.dumps({"design": "korazen", "beside": "lavutar", "dtype": "bf16", "data": "synthetic", "layers": 4,
+                      "layer_order": "delta rule, two sides, delta rule, two sides with values twice as wide; beside two sides, attention over blocks, "
+                                     "two sides, attention over blocks with values twice as wide; each + gated ff",
+                      "vocab": DESIGN_VOCAB, "prefill_tokens": T, "decode_batch": B, "decode_context": ctx, "steps": K,
+                      "warmup": W, "peaks": peaks, "peaks_from": peaks_from, "clocks": clocks, "sizes": out}))
+    return 0
+
+
 def fetorax_bench(args) -> int:
     """Prefill and decode of a Fetorax model of the 1B and 8B layer sizes beside a Llama model of the same sizes
     (random weights, vocabulary cut to 32,000): tokens a second, the device time of every kind of kernel in one
@@ -906,9 +1019,9 @@ def fetorax_bench(args) -> int:
 
 def main() -> int:
     ap = argparse.ArgumentParser()
-    ap.add_argument("--design", default="", choices=["", "fetorax", "zoporax", "raritar", "lavutar"],
+    ap.add_argument("--design", default="", choices=["", "fetorax", "zoporax", "raritar", "lavutar", "korazen"],
                     help="instead of the default workload: this design beside the closest model the library has, at equal layer "
-                         "sizes (prefill, decode, kernel by kernel): fetorax beside Llama, zoporax beside Fetorax, raritar beside Llama, lavutar beside Fetorax")
+                         "sizes (prefill, decode, kernel by kernel): fetorax beside Llama, zoporax beside Fetorax, raritar beside Llama, lavutar beside Fetorax, korazen beside Lavutar")
     ap.add_argument("--sizes", default="1b,8b", help="--design: layer sizes to run, of " + ", ".join(DESIGN_SIZES))
     ap.add_argument("--gpus", type=int, default=1)
     ap.add_argument("--steps", type=int, default=128)

@@ -18,6 +18,10 @@
 // trace of its rounding in what the first of them wrote.  delta_scan_kernel walks a sequence's
 // records with the state in registers: one round of sums over the key rows per record instead of one per token.
 //
+// Linear attention with a fixed decay per head, S_t = d S_(t-1) + k_t v_t^T, o_t = S_t^T q_t (q, k and v through silu), takes
+// the same road for prompts: it is the rule with u_t = v_t, so its records hold A_t q_t, the decayed k_s, A_DC - 1, N and v
+// alone (linear_prepare_kernel), and the scan reads nothing out ahead of the write.
+//
 // Single tokens (one kernel, delta_single_kernel): convolution, unit vectors, the decays' and the output gate's second
 // products (over their small inner sizes), the recurrence, the head's norm and the gate; the state is read and written once.
 //
@@ -26,7 +30,10 @@
 #include "tcgen05.cuh"
 
 constexpr int DC = 4;                 // tokens of a record
-constexpr int DSCAL = 4 + 16 + 16;    // scalars of a record: b [4], M [4][4] (t, s), N [4][4]
+// Scalars of a record: b [4], M [4][4] (t, s), N [4][4]; or N alone.
+template <bool RULE> constexpr int scalars() { return RULE ? 4 + 16 + 16 : 16; }
+// Vectors of a record over the key channels: A_t k_t [DC], A_t q_t [DC], decayed k_s [DC], A_DC - 1; without the first DC.
+template <bool RULE> constexpr int vectors() { return RULE ? 3 * DC + 1 : 2 * DC + 1; }
 
 typedef unsigned long long f2;        // two float32 side by side
 __device__ __forceinline__ f2 fma2(f2 a, f2 b, f2 c) {
@@ -70,13 +77,19 @@ struct DeltaArgs {
     float* raw;                  // prompts: [T, H, dv] the heads' outputs, neither normed nor gated
     int H, G, dk, dv;
     float q_scale, unit_eps;
+    // Fixed decays: rows of either dtype, q, k and v where they lie, a decay per head.
+    const void* lin_rows;
+    int lin_stride, q_off, k_off, v_off;
+    const float* decay;
 };
 
 // A record's rows of key channels are padded with zeros to whole 32s.
 __host__ __device__ __forceinline__ int pad_rows(int dk) { return (dk + 31) / 32 * 32; }
 __host__ __device__ __forceinline__ int pad4(int n) { return (n + 3) / 4 * 4; }
-// Per (record, head): scalars, A_t k_t [DC][DKP], A_t q_t [DC][DKP], decayed k_s [DC][DKP], A_DC - 1 [DKP], v [DC][pad4(dv)].
-__host__ __device__ __forceinline__ int record_floats(int dk, int dv) { return (3 * DC + 1) * pad_rows(dk) + DC * pad4(dv) + DSCAL; }
+// Per (record, head): scalars, vectors [DKP] each, v [DC][pad4(dv)].
+template <bool RULE> __host__ __device__ __forceinline__ int record_floats(int dk, int dv) {
+    return scalars<RULE>() + vectors<RULE>() * pad_rows(dk) + DC * pad4(dv);
+}
 // Where the records of sequence b start: unique and never overlapping, whatever the sequences' lengths are.
 __device__ __forceinline__ int first_record(const int* cu_rows, int b) { return cu_rows[b] / DC + b; }
 
@@ -95,9 +108,9 @@ __global__ void __launch_bounds__(DP_WARPS * 32) delta_prepare_kernel(DeltaArgs 
     const int pos0 = a.tok_pos[row0];            // the step's first position of this sequence
     const float* ring = a.ring + (size_t)a.slots[b] * taps * a.C;
     const int dkp = pad_rows(dk), dvp = pad4(dv);
-    float* rec = a.records + ((size_t)(first_record(a.cu_rows, b) + blockIdx.x) * a.H + h) * record_floats(dk, dv);
-    float* vec = rec + DSCAL;
-    float* rec_v = vec + (3 * DC + 1) * dkp;
+    float* rec = a.records + ((size_t)(first_record(a.cu_rows, b) + blockIdx.x) * a.H + h) * record_floats<true>(dk, dv);
+    float* vec = rec + scalars<true>();
+    float* rec_v = vec + vectors<true>() * dkp;
     // The raw input of channel c at the step's row i (below 0: a row of an earlier step, zero ahead of the sequence).
     auto input = [&](int i, int c) -> float {
         if (i >= 0) return a.rows[(size_t)(row0 + i) * a.stride + c];
@@ -242,24 +255,107 @@ __global__ void __launch_bounds__(DP_WARPS * 32) delta_prepare_kernel(DeltaArgs 
     if (lane < DC) rec[lane] = lane < n ? sigmoid_f(a.rows[(size_t)(row0 + t0 + lane) * a.stride + a.b_off + h]) : 0.f;
 }
 
+// The records of linear attention with a fixed decay per head: a warp per (record, head) as above.
+template <typename T, int CPL>
+__global__ void __launch_bounds__(DP_WARPS * 32) linear_prepare_kernel(DeltaArgs a) {
+    pdl_launch_dependents();
+    const int dk = a.dk, dv = a.dv, lane = threadIdx.x & 31, h = blockIdx.z * DP_WARPS + (threadIdx.x >> 5), b = blockIdx.y;
+    pdl_wait();
+    if (h >= a.H) return;
+    const int t0 = blockIdx.x * DC, row0 = a.cu_rows[b], n_rows = a.cu_rows[b + 1] - row0;
+    if (t0 >= n_rows) return;
+    const int n = min(DC, n_rows - t0), dkp = pad_rows(dk), dvp = pad4(dv);
+    float* rec = a.records + ((size_t)(first_record(a.cu_rows, b) + blockIdx.x) * a.H + h) * record_floats<false>(dk, dv);
+    float* vec = rec + scalars<false>();
+    float* rec_v = vec + vectors<false>() * dkp;
+    const T* x = (const T*)a.lin_rows + (size_t)(row0 + t0) * a.lin_stride;
+    const float d = a.decay[h];
+    float part[16];                              // N_00, N_10, N_11, N_20, ... N_33, less the powers of d; six unused
+#pragma unroll
+    for (int i = 0; i < 16; ++i) part[i] = 0.f;
+    // What is left of the state's size behind each token, and behind the record (nothing decays where there is no token).
+    float A[DC], last = 1.f;
+#pragma unroll
+    for (int t = 0; t < DC; ++t) A[t] = last = t < n ? last * d : last;
+#pragma unroll
+    for (int i = 0; i < CPL; ++i) {
+        const int r = i * 32 + lane;
+        float q[DC], k[DC];
+#pragma unroll
+        for (int t = 0; t < DC; ++t) {
+            const bool in = r < dk && t < n;
+            q[t] = in ? silu_f(to_f32(x[(size_t)t * a.lin_stride + a.q_off + h * dk + r])) : 0.f;
+            k[t] = in ? silu_f(to_f32(x[(size_t)t * a.lin_stride + a.k_off + h * dk + r])) : 0.f;
+        }
+        int nn = 0;
+#pragma unroll
+        for (int t = 0; t < DC; ++t)
+#pragma unroll
+            for (int s = 0; s <= t; ++s) {
+                part[nn] = fmaf(k[s], q[t], part[nn]);
+                ++nn;
+            }
+#pragma unroll
+        for (int t = 0; t < DC; ++t) {
+            float left = k[t];                   // k_t behind the record's later tokens
+#pragma unroll
+            for (int s = t + 1; s < DC; ++s)
+                if (s < n) left *= d;
+            vec[t * dkp + r] = A[t] * q[t];
+            vec[(DC + t) * dkp + r] = left;
+        }
+        // d^n - 1 by the binomial of d - 1, so that a decay close to one keeps its digits.
+        const float e = d - 1.f;
+        float E = 0.f;
+#pragma unroll
+        for (int t = 0; t < DC; ++t)
+            if (t < n) E = fmaf(E, d, e);
+        vec[2 * DC * dkp + r] = E;
+    }
+    for (int c = lane; c < dvp; c += 32)
+#pragma unroll
+        for (int t = 0; t < DC; ++t)
+            rec_v[t * dvp + c] = (c < dv && t < n) ? silu_f(to_f32(x[(size_t)t * a.lin_stride + a.v_off + h * dv + c])) : 0.f;
+#pragma unroll
+    for (int w = 8; w >= 1; w >>= 1) {
+        const bool upper = lane & w;
+#pragma unroll
+        for (int t = 0; t < w; ++t) {
+            const float give = upper ? part[t] : part[t + w];
+            const float mine = upper ? part[t + w] : part[t];
+            part[t] = mine + __shfl_xor_sync(0xffffffffu, give, w);
+        }
+    }
+    const float sum = part[0] + __shfl_xor_sync(0xffffffffu, part[0], 16);
+    const int t = (lane >> 2) & 3, s = lane & 3;
+    const float entry = __shfl_sync(0xffffffffu, sum, s <= t ? t * (t + 1) / 2 + s : 0);
+    if (lane < 16) {
+        float p = 1.f;
+        for (int j = s; j < t; ++j) p *= d;
+        rec[lane] = s <= t ? p * entry : 0.f;
+    }
+}
+
 // One block per (sequence, value head, some value columns): a warp takes 32 / LPC groups of NC neighbouring columns, LPC lanes
 // share a group, each with KR of the key rows.  The last warp brings the records into a ring in shared memory by bulk
 // copies; the others take them from there at their own pace.
 constexpr int DS_STAGES = 6;
-template <int KR, int LPC, int NC>
-__global__ void __launch_bounds__(288, 1) delta_scan_kernel(DeltaArgs a, int cols) {
+template <int KR, int LPC, int NC, bool RULE>
+__device__ __forceinline__ void scan_records(const DeltaArgs& a, int cols) {
     using namespace tc;
     pdl_launch_dependents();
     constexpr int DKP = KR * LPC, PIECES = KR / 4, SPAN = 4 * LPC;
-    static_assert(2 * DC * NC >= LPC && NC * DC >= 4 && (NC >= 2 * DC * NC / LPC), "every lane is left with sums of one token");
+    // Vectors that the state is read out with: with the rule first those of k, then (QV on) those of q.
+    constexpr int READ = RULE ? 2 * DC : DC, QV = RULE ? DC : 0, PER = READ * NC / LPC, KD = READ;
+    static_assert(PER >= 1 && PER <= NC && NC % PER == 0, "every lane is left with sums of one token");
     extern __shared__ __align__(16) float sm[];
     __shared__ __align__(8) uint64_t full[DS_STAGES], empty[DS_STAGES];
     const int dv = a.dv, dvp = pad4(dv), H = a.H, tid = threadIdx.x, warp = tid >> 5, lane = tid & 31, l = lane & (LPC - 1);
     const int consumers = (blockDim.x >> 5) - 1;
     const int b = blockIdx.x, h = blockIdx.y, col0 = blockIdx.z * cols;
-    constexpr int HEAD = DSCAL + (3 * DC + 1) * DKP;         // a record ahead of its values
+    constexpr int HEAD = scalars<RULE>() + vectors<RULE>() * DKP;        // a record ahead of its values
     const int stage_floats = HEAD + DC * cols;
-    const int rf = record_floats(a.dk, dv);
+    const int rf = record_floats<RULE>(a.dk, dv);
     if (tid == 0) {
         for (int i = 0; i < DS_STAGES; ++i) {
             mbar_init(smem_u32(&full[i]), 1);
@@ -292,7 +388,7 @@ __global__ void __launch_bounds__(288, 1) delta_scan_kernel(DeltaArgs a, int col
     }
     // The convolution's last inputs go to the ring; the blocks of a sequence share its channels.  (The records ahead
     // of this kernel were made from the ring as it was.)
-    {
+    if constexpr (RULE) {
         const int share = gridDim.y * gridDim.z, mine = blockIdx.y * gridDim.z + blockIdx.z, taps = a.taps;
         const int per = (a.C + share - 1) / share, lo = mine * per, hi = min(a.C, lo + per), n = row1 - row0;
         float* ring = a.ring + (size_t)a.slots[b] * taps * a.C;
@@ -319,18 +415,18 @@ __global__ void __launch_bounds__(288, 1) delta_scan_kernel(DeltaArgs a, int col
         const int stage = i % DS_STAGES;
         if (!mbar_wait(smem_u32(&full[stage]), (i / DS_STAGES) & 1)) { give_up(2); break; }
         const float* rec = sm + stage * stage_floats;
-        const float* vec = rec + DSCAL + l * 4;
+        const float* vec = rec + scalars<RULE>() + l * 4;
         const float* vs = rec + HEAD + c0;
         const float4* sc = reinterpret_cast<const float4*>(rec);
-        f2 acc2[2 * DC][NC];
+        f2 acc2[READ][NC];
 #pragma unroll
-        for (int t = 0; t < 2 * DC; ++t)
+        for (int t = 0; t < READ; ++t)
 #pragma unroll
             for (int c = 0; c < NC; ++c) acc2[t][c] = 0ull;
 #pragma unroll
         for (int j = 0; j < PIECES; ++j)
 #pragma unroll
-            for (int t = 0; t < 2 * DC; ++t) {
+            for (int t = 0; t < READ; ++t) {
                 const ulonglong2 x = *reinterpret_cast<const ulonglong2*>(vec + t * DKP + j * SPAN);
 #pragma unroll
                 for (int c = 0; c < NC; ++c) {
@@ -338,13 +434,12 @@ __global__ void __launch_bounds__(288, 1) delta_scan_kernel(DeltaArgs a, int col
                     acc2[t][c] = fma2(S[2 * j + 1][c], x.y, acc2[t][c]);
                 }
             }
-        // What token t reads from the state with k (sum t * NC + c of column c) and with q (sum (DC + t) * NC + c) is added up
+        // What token t reads from the state with k (sum t * NC + c of column c) and with q (sum (QV + t) * NC + c) is added up
         // over the LPC lanes of the columns: in each step a lane hands half of its sums across and keeps the other half, so
         // lane l is left with the sums PER l .. PER l + PER - 1.
-        constexpr int PER = 2 * DC * NC / LPC;
-        float acc[2 * DC * NC];
+        float acc[READ * NC];
 #pragma unroll
-        for (int t = 0; t < 2 * DC; ++t)
+        for (int t = 0; t < READ; ++t)
 #pragma unroll
             for (int c = 0; c < NC; ++c) {
                 const float2 f = unpack2(acc2[t][c]);
@@ -361,22 +456,29 @@ __global__ void __launch_bounds__(288, 1) delta_scan_kernel(DeltaArgs a, int col
                 acc[v] = keep + __shfl_xor_sync(0xffffffffu, give, w);
             }
         }
-        const float4 beta = sc[0], m1 = sc[2], m2 = sc[3], m3 = sc[4];
         float u[DC][NC];
+        if constexpr (RULE) {
+            const float4 beta = sc[0], m1 = sc[2], m2 = sc[3], m3 = sc[4];
 #pragma unroll
-        for (int c = 0; c < NC; ++c) {
-            float r[DC];
+            for (int c = 0; c < NC; ++c) {
+                float r[DC];
+#pragma unroll
+                for (int t = 0; t < DC; ++t)
+                    r[t] = vs[t * cols + c] - __shfl_sync(0xffffffffu, acc[(t * NC + c) % PER], (lane & ~(LPC - 1)) + (t * NC + c) / PER);
+                u[0][c] = beta.x * r[0];
+                u[1][c] = beta.y * (r[1] - m1.x * u[0][c]);
+                u[2][c] = beta.z * (r[2] - m2.x * u[0][c] - m2.y * u[1][c]);
+                u[3][c] = beta.w * (r[3] - m3.x * u[0][c] - m3.y * u[1][c] - m3.z * u[2][c]);
+            }
+        } else {
 #pragma unroll
             for (int t = 0; t < DC; ++t)
-                r[t] = vs[t * cols + c] - __shfl_sync(0xffffffffu, acc[(t * NC + c) % PER], (lane & ~(LPC - 1)) + (t * NC + c) / PER);
-            u[0][c] = beta.x * r[0];
-            u[1][c] = beta.y * (r[1] - m1.x * u[0][c]);
-            u[2][c] = beta.z * (r[2] - m2.x * u[0][c] - m2.y * u[1][c]);
-            u[3][c] = beta.w * (r[3] - m3.x * u[0][c] - m3.y * u[1][c] - m3.z * u[2][c]);
+#pragma unroll
+                for (int c = 0; c < NC; ++c) u[t][c] = vs[t * cols + c];
         }
-        if (l >= LPC / 2) {                      // the lanes that hold sums with q
-            const int t = (l * PER) / NC - DC, cc = (l * PER) % NC, row = row0 + i * DC + t;
-            const float4 nt = sc[5 + t];
+        if (l * PER >= QV * NC) {                // the lanes that hold sums with q
+            const int t = (l * PER) / NC - QV, cc = (l * PER) % NC, row = row0 + i * DC + t;
+            const float4 nt = sc[(RULE ? 5 : 0) + t];
 #pragma unroll
             for (int v = 0; v < PER; ++v) {
                 const int col = c0 + cc + v;
@@ -396,7 +498,7 @@ __global__ void __launch_bounds__(288, 1) delta_scan_kernel(DeltaArgs a, int col
             for (int c = 0; c < NC; ++c) uu[s][c] = pack2(u[s][c], u[s][c]);
 #pragma unroll
         for (int j = 0; j < PIECES; ++j) {
-            const ulonglong2 E = *reinterpret_cast<const ulonglong2*>(vec + 3 * DC * DKP + j * SPAN);
+            const ulonglong2 E = *reinterpret_cast<const ulonglong2*>(vec + (KD + DC) * DKP + j * SPAN);
 #pragma unroll
             for (int c = 0; c < NC; ++c) {
                 S[2 * j][c] = fma2(S[2 * j][c], E.x, S[2 * j][c]);
@@ -404,7 +506,7 @@ __global__ void __launch_bounds__(288, 1) delta_scan_kernel(DeltaArgs a, int col
             }
 #pragma unroll
             for (int s = 0; s < DC; ++s) {
-                const ulonglong2 x = *reinterpret_cast<const ulonglong2*>(vec + (2 * DC + s) * DKP + j * SPAN);
+                const ulonglong2 x = *reinterpret_cast<const ulonglong2*>(vec + (KD + s) * DKP + j * SPAN);
 #pragma unroll
                 for (int c = 0; c < NC; ++c) {
                     S[2 * j][c] = fma2(x.x, uu[s][c], S[2 * j][c]);
@@ -430,6 +532,11 @@ __global__ void __launch_bounds__(288, 1) delta_scan_kernel(DeltaArgs a, int col
             }
 }
 
+template <int KR, int LPC, int NC>
+__global__ void __launch_bounds__(288, 1) delta_scan_kernel(const __grid_constant__ DeltaArgs a, int cols) { scan_records<KR, LPC, NC, true>(a, cols); }
+template <int KR, int LPC, int NC>
+__global__ void __launch_bounds__(288, 1) linear_records_kernel(const __grid_constant__ DeltaArgs a, int cols) { scan_records<KR, LPC, NC, false>(a, cols); }
+
 static int scan_columns(int B, int H, int dv, int least, int most) {
     // Columns of a block: as many as it has warps for, or fewer where that leaves multiprocessors without a block.
     int cols = most;
@@ -437,17 +544,21 @@ static int scan_columns(int B, int H, int dv, int least, int most) {
     return cols;
 }
 
-template <int KR, int LPC, int NC>
+template <bool RULE, int KR, int LPC, int NC>
 static int scan_launch(const DeltaArgs& a, int B, cudaStream_t stream) {
     constexpr int PER_WARP = 32 / LPC * NC;
     const int cols = scan_columns(B, a.H, a.dv, PER_WARP, 32 < 8 * PER_WARP ? 32 : 8 * PER_WARP), threads = (cols / PER_WARP + 1) * 32;
-    const size_t smem = (size_t)DS_STAGES * (DSCAL + (3 * DC + 1) * KR * LPC + DC * cols) * sizeof(float);
-    if (smem > 48 * 1024 &&
-        cudaFuncSetAttribute(delta_scan_kernel<KR, LPC, NC>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem) != cudaSuccess)
-        return lq_launch_status();
-    // Not ahead of its time: blocks that start while the records are still being made take what room they find, several on
-    // one multiprocessor, and stay there; started afterwards they spread out (measured: half the time).
-    return launch_after(delta_scan_kernel<KR, LPC, NC>, dim3(B, a.H, (a.dv + cols - 1) / cols), dim3(threads), smem, stream, a, cols);
+    const size_t smem = (size_t)DS_STAGES * (scalars<RULE>() + vectors<RULE>() * KR * LPC + DC * cols) * sizeof(float);
+    auto go = [&](auto kernel) {
+        if (smem > 48 * 1024 &&
+            cudaFuncSetAttribute(kernel, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem) != cudaSuccess)
+            return lq_launch_status();
+        // Not ahead of its time: blocks that start while the records are still being made take what room they find, several
+        // on one multiprocessor, and stay there; started afterwards they spread out (measured: half the time).
+        return launch_after(kernel, dim3(B, a.H, (a.dv + cols - 1) / cols), dim3(threads), smem, stream, a, cols);
+    };
+    if constexpr (RULE) return go(delta_scan_kernel<KR, LPC, NC>);
+    else return go(linear_records_kernel<KR, LPC, NC>);
 }
 
 template <int CPL>
@@ -458,7 +569,10 @@ static int prepare_launch(const DeltaArgs& a, int B, int max_new, cudaStream_t s
 
 // Floats of scratch that a step with prompts needs for its records.
 LQ_EXPORT long long lq_delta_record_floats(int T, int B, int H, int dk, int dv) {
-    return (long long)(T / DC + B) * H * record_floats(dk, dv);
+    return (long long)(T / DC + B) * H * record_floats<true>(dk, dv);
+}
+LQ_EXPORT long long lq_linear_record_floats(int T, int B, int H, int dk, int dv) {
+    return (long long)(T / DC + B) * H * record_floats<false>(dk, dv);
 }
 
 // Prompts and portions: rows [T, stride] float32 (q, k, v, b side by side), z [T, H dk] float32 -> raw [T, H, dv].
@@ -470,23 +584,38 @@ LQ_EXPORT int lq_delta_prompt(const float* rows, int stride, int b_off, const fl
     if (dk < 1 || dk > 256 || dv < 1 || G < 1 || H % G || taps < 1) return LQ_BAD_SIZE;
     DeltaArgs a{rows, stride, b_off, taps_w, taps, 2 * G * dk + H * dv, ring, z, z_bias, rate, state, cu_rows, slots, tok_pos,
                 records, raw, H, G, dk, dv, q_scale, unit_eps};
-    int rc = LQ_BAD_SIZE;
-    const int cpl = pad_rows(dk) / 32;
-#define LQ_GO(CPL, ...) case CPL: \
-        rc = prepare_launch<CPL>(a, B, max_new, stream); \
-        return rc != LQ_OK ? rc : scan_launch<__VA_ARGS__>(a, B, stream)
-    switch (cpl) {
-        LQ_GO(1, 4, 8, 2);
-        LQ_GO(2, 8, 8, 2);
-        LQ_GO(3, 12, 8, 2);
-        LQ_GO(4, 16, 8, 2);
-        LQ_GO(5, 20, 8, 2);
-        LQ_GO(6, 24, 8, 2);
-        LQ_GO(7, 28, 8, 2);
-        LQ_GO(8, 32, 8, 2);
-    }
+    switch (pad_rows(dk) / 32) {
+#define LQ_GO(CPL) case CPL: { \
+        const int rc = prepare_launch<CPL>(a, B, max_new, stream); \
+        return rc != LQ_OK ? rc : scan_launch<true, 4 * CPL, 8, 2>(a, B, stream); }
+        LQ_GO(1) LQ_GO(2) LQ_GO(3) LQ_GO(4) LQ_GO(5) LQ_GO(6) LQ_GO(7) LQ_GO(8)
 #undef LQ_GO
-    return rc;
+    }
+    return LQ_BAD_SIZE;
+}
+
+// The same for linear attention with a fixed decay per head: rows [T, stride] of either dtype, H heads of q at q_off, of k at
+// k_off (dk each) and of v at v_off (dv each), all through silu -> raw [T, H, dv].
+LQ_EXPORT int lq_linear_prompt(const void* rows, int dtype, int stride, int q_off, int k_off, int v_off, const float* decay, float* state,
+                               const int* cu_rows, const int* slots, float* records, float* raw, int B, int max_new, int H, int dk, int dv,
+                               cudaStream_t stream) {
+    if (B <= 0 || max_new <= 0) return LQ_OK;
+    if (dk < 1 || dk > 256 || dv < 1) return LQ_BAD_SIZE;
+    if (dtype != LQ_F32 && dtype != LQ_BF16) return LQ_BAD_DTYPE;
+    DeltaArgs a{};
+    a.state = state; a.cu_rows = cu_rows; a.slots = slots; a.records = records; a.raw = raw;
+    a.H = a.G = H; a.dk = dk; a.dv = dv;
+    a.lin_rows = rows; a.lin_stride = stride; a.q_off = q_off; a.k_off = k_off; a.v_off = v_off; a.decay = decay;
+    const dim3 grid((max_new + DC - 1) / DC, B, (H + DP_WARPS - 1) / DP_WARPS), block(DP_WARPS * 32);
+    switch (pad_rows(dk) / 32) {
+#define LQ_GO(CPL) case CPL: { \
+        const int rc = dtype == LQ_F32 ? launch_pdl(linear_prepare_kernel<float, CPL>, grid, block, 0, stream, a) \
+                                       : launch_pdl(linear_prepare_kernel<__nv_bfloat16, CPL>, grid, block, 0, stream, a); \
+        return rc != LQ_OK ? rc : scan_launch<false, 4 * CPL, 8, 2>(a, B, stream); }
+        LQ_GO(1) LQ_GO(2) LQ_GO(3) LQ_GO(4) LQ_GO(5) LQ_GO(6) LQ_GO(7) LQ_GO(8)
+#undef LQ_GO
+    }
+    return LQ_BAD_SIZE;
 }
 
 LQ_EXPORT int lq_delta_status() { return tc::status_read(); }
@@ -553,7 +682,8 @@ __global__ void __launch_bounds__(DT_THREADS) delta_single_kernel(DeltaSingleArg
     float* xg = xa + s.ra_ld;                    // [rg_ld]
     float* red = xg + s.rg_ld;                   // [rg][2][cg * VW]
     __shared__ float sums[3], part[DT_THREADS / 32];
-    pdl_wait();
+    // Row, position and slot are written before the step starts, the state and the ring by the step before: they are read,
+    // and the second products' weights asked for, before the kernel ahead is known to have finished.
     const int row = a.cu_rows[b], pos = a.tok_pos[row], slot = a.slots[b];
     const float* x = a.rows + (size_t)row * a.stride;
     float* ring = a.ring + (size_t)slot * taps * a.C;
@@ -575,18 +705,30 @@ __global__ void __launch_bounds__(DT_THREADS) delta_single_kernel(DeltaSingleArg
         }
     };
     load_state(cl * VW);
+    for (int e = tid; e < dk + dv; e += DT_THREADS) {
+        const TW* w = e < dk ? (const TW*)s.a2 + (size_t)(h * dk + e) * s.ra_ld : (const TW*)s.g2 + (size_t)(h * dv + e - dk) * s.rg_ld;
+        asm volatile("prefetch.global.L2 [%0];" ::"l"(w));
+    }
+    // Channel e of q, k (key head g) and v (head h), side by side as below; its sum over the taps on earlier inputs.
+    auto channel = [&](int e) { return e < dk ? g * dk + e : (e < 2 * dk ? G * dk + g * dk + (e - dk) : 2 * G * dk + h * dv + (e - 2 * dk)); };
+    for (int e = tid; e < 2 * dk + dv; e += DT_THREADS) {
+        const int c = channel(e);
+        float acc = 0.f;
+#pragma unroll 4
+        for (int j = 0; j < keep; ++j) {
+            const int p = pos - keep + j;
+            if (p >= 0) acc = fmaf(a.taps_w[(size_t)j * a.C + c], ring[(size_t)(p % taps) * a.C + c], acc);
+        }
+        sq[e < 2 * dk ? e : dk + e] = acc;                           // sq, sk, (sa), sv lie one after another
+    }
+    pdl_wait();
     for (int i = tid; i < s.ra_ld + s.rg_ld; i += DT_THREADS)
         xa[i] = i < s.ra_ld ? (i < s.ra ? x[s.a_off + i] : 0.f) : (i - s.ra_ld < s.rg ? x[s.g_off + i - s.ra_ld] : 0.f);
     for (int e = tid; e < 2 * dk + dv; e += DT_THREADS) {
-        const int c = e < dk ? g * dk + e : (e < 2 * dk ? G * dk + g * dk + (e - dk) : 2 * G * dk + h * dv + (e - 2 * dk));
+        const int c = channel(e);
         const float own = x[c];
-        float acc = 0.f;
-        for (int j = 0; j < taps; ++j) {
-            const int p = pos - keep + j;
-            const float v = j == keep ? own : (p >= 0 ? ring[(size_t)(p % taps) * a.C + c] : 0.f);
-            acc = fmaf(a.taps_w[(size_t)j * a.C + c], v, acc);
-        }
-        sq[e < 2 * dk ? e : dk + e] = silu_f(acc);                   // sq, sk, (sa), sv lie one after another
+        float& y = sq[e < 2 * dk ? e : dk + e];                      // (the thread's own sum)
+        y = silu_f(fmaf(a.taps_w[(size_t)keep * a.C + c], own, y));
         // Of the value heads that share a key head, the first one's block moves its channels' ring on.
         if (e >= 2 * dk || h % (H / G) == 0) ring[(size_t)(pos % taps) * a.C + c] = own;
     }

@@ -1252,6 +1252,38 @@ __global__ void gate_mul_kernel(T* __restrict__ x, const TG* __restrict__ gate, 
     x[i] = from_f32<T>(to_f32(x[i]) * (act == 1 ? sg : g * sg));
 }
 
+// bfloat16 rows behind a gate per value, eight numbers a thread: the same arithmetic.
+template <typename TG>
+__global__ void gate_mul_vec_kernel(uint4* __restrict__ x, const TG* __restrict__ gate, int gate_stride, int cols8, size_t total8, int act) {
+    pdl_launch_dependents();
+    pdl_wait();
+    const size_t i = (size_t)blockIdx.x * blockDim.x + threadIdx.x;
+    if (i >= total8) return;
+    const TG* gp = gate + (i / cols8) * gate_stride + (i % cols8) * 8;
+    float g[8];
+    if constexpr (sizeof(TG) == 4) {
+        const float4 a = reinterpret_cast<const float4*>(gp)[0], b = reinterpret_cast<const float4*>(gp)[1];
+        g[0] = a.x; g[1] = a.y; g[2] = a.z; g[3] = a.w; g[4] = b.x; g[5] = b.y; g[6] = b.z; g[7] = b.w;
+    } else {
+        const uint4 raw = *reinterpret_cast<const uint4*>(gp);
+        const __nv_bfloat162* p = reinterpret_cast<const __nv_bfloat162*>(&raw);
+#pragma unroll
+        for (int j = 0; j < 4; ++j) {
+            const float2 f = __bfloat1622float2(p[j]);
+            g[2 * j] = f.x; g[2 * j + 1] = f.y;
+        }
+    }
+    uint4 v = x[i];
+    __nv_bfloat162* p = reinterpret_cast<__nv_bfloat162*>(&v);
+#pragma unroll
+    for (int j = 0; j < 4; ++j) {
+        const float2 f = __bfloat1622float2(p[j]);
+        const float s0 = 1.f / (1.f + expf(-g[2 * j])), s1 = 1.f / (1.f + expf(-g[2 * j + 1]));
+        p[j] = __floats2bfloat162_rn(f.x * (act == 1 ? s0 : g[2 * j] * s0), f.y * (act == 1 ? s1 : g[2 * j + 1] * s1));
+    }
+    x[i] = v;
+}
+
 LQ_EXPORT int lq_gate_mul(void* x, const void* gate, int gate_stride, int dtype, int gate_dtype, int rows, int cols, int act,
                           int group, cudaStream_t stream) {
     const size_t total = (size_t)rows * cols;
@@ -1259,6 +1291,14 @@ LQ_EXPORT int lq_gate_mul(void* x, const void* gate, int gate_stride, int dtype,
     if ((act != 1 && act != 2) || group < 1 || cols % group) return LQ_BAD_SIZE;
     unsigned blocks = (unsigned)((total + 255) / 256);
     typedef __nv_bfloat16 bf;
+    const int gate_piece = gate_dtype == LQ_F32 ? 4 : 8;
+    if (dtype == LQ_BF16 && group == 1 && cols % 8 == 0 && gate_stride % gate_piece == 0 && (((uintptr_t)x | (uintptr_t)gate) & 15) == 0) {
+        const dim3 grid((unsigned)((total / 8 + 255) / 256));
+        if (gate_dtype == LQ_F32)
+            return launch_pdl(gate_mul_vec_kernel<float>, grid, dim3(256), 0, stream, (uint4*)x, (const float*)gate, gate_stride, cols / 8, total / 8, act);
+        if (gate_dtype == LQ_BF16)
+            return launch_pdl(gate_mul_vec_kernel<bf>, grid, dim3(256), 0, stream, (uint4*)x, (const bf*)gate, gate_stride, cols / 8, total / 8, act);
+    }
     if (dtype == LQ_F32 && gate_dtype == LQ_F32)
         return launch_pdl(gate_mul_kernel<float, float>, dim3(blocks), dim3(256), 0, stream, (float*)x, (const float*)gate, gate_stride, cols, total, act, group);
     if (dtype == LQ_BF16 && gate_dtype == LQ_BF16)

@@ -1029,6 +1029,29 @@ def delta_prompt(rows: torch.Tensor, b_off: int, taps_w: torch.Tensor, ring: tor
     return raw
 
 
+def linear_prompt(rows: torch.Tensor, q_off: int, k_off: int, v_off: int, decay: torch.Tensor, state: torch.Tensor, cu_rows, slots, B: int,
+                  max_new: int, H: int, dk: int, dv: int) -> torch.Tensor:
+    """Linear attention with a fixed decay per head over a step's rows, by the records and the scan of the delta rule
+    (csrc/delta.cu): S_t = decay_h S_(t-1) + k_t v_t^T, o_t = S_t^T q_t with silu on q, k and v (heads side by side at their
+    columns of rows).  state [slots, H, dk, dv] float32 is moved on.  Returns S^T q, float32 [T, H, dv]."""
+    T = rows.shape[0]
+    if rows.stride(1) != 1 or rows.shape[1] < max(q_off, k_off) + H * dk or rows.shape[1] < v_off + H * dv or dk > 256:
+        raise KernelError("linear_prompt: rows with unit column stride that hold q, k and v; key size at most 256")
+    if state.dtype != torch.float32 or tuple(state.shape[1:]) != (H, dk, dv) or not state.is_contiguous():
+        raise KernelError(f"linear_prompt: the state must be contiguous float32 [slots, {H}, {dk}, {dv}]")
+    if decay.dtype != torch.float32 or decay.numel() != H:
+        raise KernelError("linear_prompt: the decays must be float32 [H]")
+    size = build.load("delta").lq_linear_record_floats
+    size.argtypes, size.restype = [c_int] * 5, c_longlong
+    records = torch.empty(int(size(T, B, H, dk, dv)), dtype=torch.float32, device=rows.device)
+    raw = torch.empty((T, H, dv), dtype=torch.float32, device=rows.device)
+    fn = _fn("delta", "lq_linear_prompt", [c_void_p, c_int, c_int, c_int, c_int, c_int, c_void_p, c_void_p, c_void_p, c_void_p, c_void_p,
+                                           c_void_p, c_int, c_int, c_int, c_int, c_int, c_void_p])
+    _check(fn(_p(rows), dtype_code(rows), rows.stride(0), q_off, k_off, v_off, _p(decay), _p(state), _p(cu_rows), _p(slots), _p(records),
+              _p(raw), B, max_new, H, dk, dv, _stream()), "linear_prompt", 2)
+    return raw
+
+
 def delta_single(rows: torch.Tensor, b_off: int, taps_w: torch.Tensor, ring: torch.Tensor, z_bias: torch.Tensor, rate: torch.Tensor,
                  state: torch.Tensor, cu_rows, slots, tok_pos, a_off: int, ra: int, a2: torch.Tensor, g_off: int, rg: int, g2: torch.Tensor,
                  norm_w: torch.Tensor, norm_eps: float, out_dtype: torch.dtype, B: int, H: int, G: int, dk: int, dv: int, q_scale: float,

@@ -30,7 +30,8 @@ Gates, decays, the state and the per-head norms are 32-bit in both precisions; t
 gates' pre-activations come from a 32-bit product of their own.  A sequence's tokens
 are walked in order from the state in its slot (`csrc/recurrent.cu`: one kernel for
 prompts and portions, one for steps of a single token per sequence), so a position's
-result does not depend on how its prompt was cut, beyond rounding.
+result does not depend on how its prompt was cut, beyond rounding.  ("lightning" walks prompts by records of four tokens,
+`csrc/delta.cu`.)
 """
 from __future__ import annotations
 
@@ -114,6 +115,8 @@ class Retention(_MatrixStateMixer):
 
 @register_part("mixer", "lightning")
 class Lightning(_MatrixStateMixer):
+    kernel_libraries = ("recurrent", "delta")
+
     def __init__(self, runtime: Runtime, hidden_size: int, n_heads: int, key_dim: int, value_dim: int, decay, eps: float,
                  names: dict | None = None):
         super().__init__(runtime, hidden_size, n_heads, key_dim, value_dim, eps, {"norm": "norm", **(names or {})})
@@ -136,9 +139,12 @@ class Lightning(_MatrixStateMixer):
     def forward(self, h, ctx: StepContext, cache_view, residual, writes_cache: bool = True):
         H, dk, dv = self.H, self.dk, self.dv
         rows = linear.linear(h, self.w_in, self.runtime.act_dtype)
-        # silu meets q, k and v in 32-bit as the scan reads them: nothing that enters the recurrence is rounded again.
-        raw, _ = ops.linear_scan(rows, 0, H * dk, 2 * H * dk, cache_view, ctx.cu_rows, ctx.slots, ctx.tok_pos, ctx.B,
-                                 H, dk, dv, decay=self.decay, single=ctx.decode, in_act="silu")
+        # silu meets q, k and v in 32-bit as they are read: nothing that enters the recurrence is rounded again.
+        if ctx.decode:
+            raw, _ = ops.linear_scan(rows, 0, H * dk, 2 * H * dk, cache_view, ctx.cu_rows, ctx.slots, ctx.tok_pos, ctx.B,
+                                     H, dk, dv, decay=self.decay, single=True, in_act="silu")
+        else:
+            raw = ops.linear_prompt(rows, 0, H * dk, 2 * H * dk, self.decay, cache_view, ctx.cu_rows, ctx.slots, ctx.B, ctx.max_new, H, dk, dv)
         g_off = 2 * H * dk + H * dv
         # One norm over all heads: the heads' outputs as a single "head" of H * dv numbers.
         out = ops.head_norm_gate(raw.view(raw.shape[0], 1, H * dv), H * dv, self.eps, self.runtime.act_dtype,

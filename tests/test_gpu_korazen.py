@@ -96,6 +96,22 @@ def test_one_layer_of_each_kind_whole_and_token_by_token(tmp_path, name, dtype):
 
 
 @pytest.mark.parametrize("dtype", DTYPES)
+@pytest.mark.parametrize("name", ["only_delta", "only_sides"])
+def test_a_checkpoint_stored_in_32_bit(tmp_path, name, dtype):
+    """Every tensor float32: the products keep them as they are, in either precision of the model."""
+    folder = make_folder(tmp_path, name, seed=6, dtype=torch.float32)
+    toks = tokens(70, CONFIGS[name]["vocab"], 9)
+    ref, tol, firm = _plain(folder, toks, dtype)
+    import warnings
+    with warnings.catch_warnings():
+        warnings.simplefilter("ignore")                      # (the loader says that such products run on the CUDA cores)
+        eng = _engine(folder, dtype, max_tokens=256)
+    s = eng.new_sequence()
+    assert row_errors(_rows(eng, s, toks, 40), ref)[firm].max() < tol
+    eng.close()
+
+
+@pytest.mark.parametrize("dtype", DTYPES)
 def test_a_block_ends_where_it_ends_when_one_token_outweighs_all_others(tmp_path, dtype):
     """The softmax side alone (the other side's norm weight is zero), in a prompt of one odd token among copies of another
     and with a flat softmax, so that one odd key shows.  With blocks of 4 an odd token at position 30 changes the logits
@@ -260,13 +276,15 @@ def test_a_slot_that_is_used_again_starts_from_nothing(tmp_path, dtype):
     last inputs or a page that outlived its request would show in the next one's first tokens."""
     folder = make_folder(tmp_path, "mixed", seed=21)
     eng = _engine(folder, dtype, max_tokens=192, max_batch=1)
+    rows, requests = {}, {}
     for i, n in enumerate([150, 3, 130, 66]):
-        toks = tokens(n, CONFIGS["mixed"]["vocab"], 300 + i)
+        toks = requests[i] = tokens(n, CONFIGS["mixed"]["vocab"], 300 + i)
         s = eng.new_sequence()
         assert s == 0
         got = _rows(eng, s, toks, max(1, n - 40))
         eng.end_sequence(s)
-        _check({(i, p): row for p, row in enumerate(got)}, {i: toks}, folder, dtype, f"request {i}")
+        rows.update({(i, p): row for p, row in enumerate(got)})
+    _check(rows, requests, folder, dtype, "one slot")
     assert eng.cache.pages_in_use() == 0
     eng.close()
 

@@ -418,3 +418,66 @@ def test_sizes_that_the_rule_does_not_take_are_refused():
     with pytest.raises(ops.KernelError):
         ops.attn_prefill(_rand((1, 64), torch.bfloat16, 1), _rand((1, 1, 64, 64), torch.bfloat16, 1), _rand((1, 1, 64, 264), torch.bfloat16, 2),
                          _i32([[0]]), _i32([0]), _i32([1]), _blocks([1], [0], 64), 1, 1, 64, 64, 1.0, None, vd=264)
+
+
+# ------------------------------------------------------------------ fixed decays through records, gates by pieces
+
+@pytest.mark.parametrize("dtype", [torch.float32, torch.bfloat16])
+@pytest.mark.parametrize("H,dk,dv", [(2, 16, 24), (3, 64, 64), (1, 20, 37), (2, 128, 48), (1, 256, 5), (2, 96, 200), (1, 161, 12)])
+def test_fixed_decay_records_whole_in_portions_and_beside_single_tokens(dtype, H, dk, dv):
+    """Decays of exactly one, close to one and far from it; whole, in portions, and going on from (and to) the kernel for
+    single tokens; a first token that stands out is still there behind a decay of one."""
+    ops = _ops()
+    lens, decays = [70, 3, 41], [1.0, 0.9995, 0.3][:H]
+    decay = torch.tensor(decays, device=DEV)
+    off, width = (3, 3 + H * dk, 3 + 2 * H * dk), 3 + 2 * H * dk + H * dv + 2
+    rows = [_rand((n, width), dtype, 60 + i) for i, n in enumerate(lens)]
+    for r in rows:
+        r[0, off[2]:off[2] + H * dv] = 25.0
+    ref = []
+    for r in rows:
+        x = _d(r)
+        x = x * torch.sigmoid(x)
+        n = x.shape[0]
+        q, k = x[:, off[0]:off[0] + H * dk].reshape(n, H, dk), x[:, off[1]:off[1] + H * dk].reshape(n, H, dk)
+        v = x[:, off[2]:off[2] + H * dv].reshape(n, H, dv)
+        S, o = torch.zeros(H, dk, dv, dtype=torch.float64), torch.zeros(n, H, dv, dtype=torch.float64)
+        for t in range(n):
+            S = _d(decay)[:, None, None] * S + k[t][:, :, None] * v[t][:, None, :]
+            o[t] = torch.einsum("hdv,hd->hv", S, q[t])
+        ref.append((o, S))
+    for cuts in ([[70], [3], [41]], [[1, 2, 5, 4, 58], [2, 1], [7, 1, 1, 32]], [[64, -6], [-3], [5, -1, 35]]):       # -n: n single tokens
+        state = torch.zeros((5, H, dk, dv), dtype=torch.float32, device=DEV)
+        slots, at, got = [4, 0, 2], [0, 0, 0], [[], [], []]
+        for i in range(3):
+            for c in cuts[i]:
+                for n in ([c] if c > 0 else [1] * -c):
+                    part = rows[i][at[i]:at[i] + n].contiguous()
+                    cu, sl = _i32([0, n]), _i32([slots[i]])
+                    if c > 0:
+                        out = ops.linear_prompt(part, *off, decay, state, cu, sl, 1, n, H, dk, dv)
+                    else:
+                        out, _ = ops.linear_scan(part, *off, state, cu, sl, _i32([at[i]]), 1, H, dk, dv, decay=decay, single=True, in_act="silu")
+                    got[i].append(out)
+                    at[i] += n
+        for i in range(3):
+            _close(torch.cat(got[i]), ref[i][0], 2e-5)
+            _close(state[slots[i]], ref[i][1], 2e-5)
+    # all three sequences in one step
+    state = torch.zeros((5, H, dk, dv), dtype=torch.float32, device=DEV)
+    out = ops.linear_prompt(torch.cat(rows).contiguous(), *off, decay, state, _i32([0, 70, 73, 114]), _i32([4, 0, 2]), 3, 70, H, dk, dv)
+    for i, (lo, hi) in enumerate(((0, 70), (70, 73), (73, 114))):
+        _close(out[lo:hi], ref[i][0], 2e-5)
+    assert float(state[1].abs().max()) == 0.0 and float(state[3].abs().max()) == 0.0
+
+
+@pytest.mark.parametrize("gdtype", [torch.bfloat16, torch.float32])
+@pytest.mark.parametrize("cols,off", [(64, 8), (64, 3), (20, 0), (1024, 16)])
+@pytest.mark.parametrize("act", ["sigmoid", "silu"])
+def test_gates_by_pieces_and_one_by_one(gdtype, cols, off, act):
+    ops = _ops()
+    x, wide = _rand((9, cols), torch.bfloat16, 1), _rand((9, cols + 32), gdtype, 2, 3.0)
+    gate = wide[:, off:off + cols]
+    g = _d(gate)
+    ref = _d(x) * (torch.sigmoid(g) if act == "sigmoid" else g * torch.sigmoid(g))
+    _close(ops.gate_mul(x.clone(), gate, act), ref, BF16_ULP, BF16_ULP)

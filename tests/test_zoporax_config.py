@@ -42,7 +42,7 @@ def test_configuration_round_trip_and_description():
     assert table["l0.mlp.shared.up"].shape == (48, 64) and table["l0.mlp.shared.sg"].shape == (1, 64)
     assert "l3.mlp.shared.up" not in table and "l2.norm2" not in table and "l2.mlp.up" not in table
     assert "head" not in table and "final.norm" in table
-    assert model.graph_safe and model.kernel_libraries() == ("latent_attn", "moe", "recurrent")
+    assert model.graph_safe and model.kernel_libraries() == ("delta", "latent_attn", "moe", "recurrent")
 
 
 @pytest.mark.parametrize("change,word", [
