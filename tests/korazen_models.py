@@ -53,7 +53,7 @@ CONFIGS = {
     "only_delta_odd": model(36, 77, [delta(3, 3, 20, 37, conv=7, rank=24, gate_rank=2)], logit_scale=0.5),
     "only_delta_no_past": model(32, 80, [delta(6, 2, 8, 5, conv=1, rank=3)]),
     "only_delta_two_taps": model(56, 80, [delta(1, 1, 96, 72, conv=2, rank=8, mlp=dense(40, 0.5))]),
-    "only_sides": model(64, 140, [sides((2, 1, 64, 64, None, 40, (64, 2e4)), (32, 48, (0.9, 1.0)), mlp=dense(40, 1.2))], logit_scale=3.0),
+    "only_sides": model(64, 140, [sides((2, 1, 64, 64, None, 40, (64, 3e4)), (32, 48, (0.9, 1.0)), mlp=dense(40, 1.2))], logit_scale=3.0),
     "only_sides_wide_values": model(48, 110, [sides((4, 2, 16, 32, 0.3, 24, (16, 100.0)), (24, 8, (0.5, 0.99, 0.2)))]),
     "only_sides_narrow_values": model(64, 110, [sides((2, 2, 128, 40, 0.08, 70, (32, 1e4)), (8, 72, (0.97,)))]),
     "only_sides_very_wide_values": model(64, 90, [sides((3, 1, 48, 160, None, 100, (8, 500.0)), (80, 40, (0.8, 0.999)))]),

@@ -128,9 +128,9 @@ def test_which_attention_kernel_takes_values_of_another_size():
     bf, f32 = torch.bfloat16, torch.float32
     kind = attention_kernels.prefill_kernel
     assert kind(bf, 128, vd=128) == kind(bf, 64) == "tc"
-    assert kind(bf, 64, vd=128) == kind(bf, 128, vd=256) == kind(bf, 96, vd=192) == kind(bf, 48, vd=40) == "mma"
+    assert kind(bf, 64, vd=128) == kind(bf, 128, vd=256) == kind(bf, 112, vd=224) == kind(bf, 48, vd=40) == "mma"
     assert kind(bf, 128, vd=264) is None and kind(bf, 128, vd=12) is None and kind(bf, 144, vd=64) is None and kind(f32, 64, vd=64) is None
-    assert attention_kernels.decode_kernel(bf, 96, 192) and not attention_kernels.decode_kernel(bf, 96, 300)
+    assert attention_kernels.decode_kernel(bf, 80, 160) and not attention_kernels.decode_kernel(bf, 96, 300)
     part = make_part("mixer", PartSpec("attention", {"hidden_size": 32, "n_heads": 4, "n_kv_heads": 2, "head_dim": 64, "scale": 0.1,
                                                      "value_dim": 128, "chunk": 70}), Runtime(CPU, bf, 64))
     assert set(part.step_needs()) == {"query_blocks64", attention_kernels.decode_work_name(4, 2, None, chunk=70)}
