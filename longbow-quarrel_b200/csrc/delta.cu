@@ -97,7 +97,7 @@ __device__ __forceinline__ int first_record(const int* cu_rows, int b) { return 
 // so every sum over them stays inside the warp.
 constexpr int DP_WARPS = 4;
 template <int CPL>
-__global__ void __launch_bounds__(DP_WARPS * 32, CPL == 3 || CPL == 4 ? 5 : 1) delta_prepare_kernel(DeltaArgs a) {
+__global__ void __launch_bounds__(DP_WARPS * 32, CPL <= 2 ? 6 : CPL <= 4 ? 5 : 1) delta_prepare_kernel(DeltaArgs a) {
     pdl_launch_dependents();
     const int dk = a.dk, dv = a.dv, lane = threadIdx.x & 31, h = blockIdx.z * DP_WARPS + (threadIdx.x >> 5), b = blockIdx.y;
     pdl_wait();

@@ -302,18 +302,27 @@ def test_long_decoding_from_the_first_token(tmp_path, dtype):
 
 # ------------------------------------------------------------------ generation through the entry point and the command line
 
-def _greedy_matches(folder, prompt, new, dtype):
+TOSS_UP = 0.005        # in router logits: what a bfloat16 run takes is as good as chance
+REACH = 24             # positions behind one for which the other row is still one of the few dozen keys that they see
+
+
+def _greedy_matches(folder, prompt, new, dtype) -> int:
+    """How many of the tokens could be held to the plain implementation's choice."""
     cfg, weights = load(folder)
-    seq = list(prompt)
+    seq, held = list(prompt), 0
     for tok in new:
-        logits = plain_lavutar.forward(cfg, weights, seq)[-1].numpy()
+        margins: list = []
+        logits = plain_lavutar.forward(cfg, weights, seq, margins=margins)[-1].numpy()
         best = int(np.argmax(logits))
         gap = (logits[best] - logits[tok]) / np.sqrt((logits ** 2).mean())
-        # Where a router's choice at this position is a close call, a bfloat16 run may take the other expert and
-        # so another token; the test goes on from the token that was generated.
-        if firm_rows(dtype, cfg, weights, seq)[-1]:
+        # Where a router's choice at this position is a close call, or was a toss-up a few positions back, a bfloat16 run
+        # may take the other expert and so another token; the test goes on from the token that was generated.
+        near = np.asarray(margins, dtype=np.float64).reshape(-1, len(seq))[:, -REACH:]
+        if dtype == "float32" or (firm_rows(dtype, cfg, weights, seq)[-1] and not (near < TOSS_UP).any()):
             assert tok == best or (dtype == "bfloat16" and gap < 5e-2), (dtype, len(seq), tok, best, gap)
+            held += 1
         seq.append(tok)
+    return held
 
 
 @pytest.mark.parametrize("dtype", DTYPES)
@@ -326,8 +335,8 @@ def test_greedy_generation_through_the_scheduler(tmp_path, dtype):
     eng = _engine(folder, dtype, max_tokens=3 * 128, max_batch=3)
     out = eng.generate(prompts, max_new_tokens=10, sampling=SamplingParams(temperature=0.0), stop_ids=[], batch_size=3)
     assert [len(o) for o in out] == [10] * 5
-    for prompt, new in zip(prompts, out):
-        _greedy_matches(folder, prompt, new, dtype)
+    held = sum(_greedy_matches(folder, prompt, new, dtype) for prompt, new in zip(prompts, out))
+    assert held == 50 or (dtype == "bfloat16" and held >= 10), held
     eng.close()
 
 
