@@ -91,25 +91,23 @@ def softplus(z: torch.Tensor) -> torch.Tensor:
     return torch.clamp(z, min=0.0) + torch.log1p(torch.exp(-z.abs()))
 
 
-def rotate_halves(x: torch.Tensor, pos: int, rot: dict) -> torch.Tensor:
-    """x [heads, dim] at position pos: pairs (i, i + dims/2) of the first dims dimensions turn by pos * base^(-2i/dims)."""
+def rotate_halves(x: torch.Tensor, rot: dict) -> torch.Tensor:
+    """x [T, heads, dim]: pairs (i, i + dims/2) of the first dims dimensions turn by t * base^(-2i/dims) at position t."""
     dims, base = rot["dims"], float(rot["base"])
     f = torch.tensor([base ** (-2.0 * i / dims) for i in range(dims // 2)], dtype=torch.float64)
-    a = pos * f
+    a = torch.arange(x.shape[0], dtype=torch.float64)[:, None, None] * f
     c, s = torch.cos(a).to(x.dtype), torch.sin(a).to(x.dtype)
-    u, v = x[:, :dims // 2], x[:, dims // 2:dims]
-    return torch.cat([u * c - v * s, v * c + u * s, x[:, dims:]], dim=1)
+    u, v = x[..., :dims // 2], x[..., dims // 2:dims]
+    return torch.cat([u * c - v * s, v * c + u * s, x[..., dims:]], dim=2)
 
 
 def causal_conv_silu(z: torch.Tensor, taps: torch.Tensor) -> torch.Tensor:
     """z [T, channels], taps [channels, n]: silu(sum_j taps[:, j] z_(t - n + 1 + j)), rows before the first one zero."""
     T, n = z.shape[0], taps.shape[1]
     out = torch.zeros_like(z)
-    for t in range(T):
-        for j in range(n):
-            s = t - n + 1 + j
-            if s >= 0:
-                out[t] += taps[:, j] * z[s]
+    for j in range(n):
+        back = n - 1 - j                       # tap j looks this many positions back
+        out[back:] += taps[:, j] * z[:max(T - back, 0)]
     return silu(out)
 
 
@@ -170,8 +168,7 @@ def block_attention(h: torch.Tensor, w: dict, m: dict, eps: float) -> torch.Tens
     k = unit_rms((h @ w["k"].T + w["k.b"]).reshape(T, G, dim), eps) * w["k.norm"]
     v = _st(h @ w["v"].T + w["v.b"]).reshape(T, G, vdim)
     if m.get("rot"):
-        q = torch.stack([rotate_halves(q[t], t, m["rot"]) for t in range(T)])
-        k = torch.stack([rotate_halves(k[t], t, m["rot"]) for t in range(T)])
+        q, k = rotate_halves(q, m["rot"]), rotate_halves(k, m["rot"])
     q, k = _st(q), _st(k)
     out = torch.zeros(T, H, vdim, dtype=h.dtype)
     for t in range(T):

@@ -34,10 +34,11 @@ def _plain(folder, toks, dtype=None):
     key = (str(folder), tuple(toks))
     if key not in _memo:
         cfg, weights = load(folder)
-        _memo[key] = {"ref": plain_korazen.forward(cfg, weights, toks).numpy()}
+        margins: list = []
+        _memo[key] = {"ref": plain_korazen.forward(cfg, weights, toks, margins=margins).numpy(), "margins": margins}
     entry = _memo[key]
     if dtype is not None and dtype not in entry:
-        firm = firm_rows(dtype, *load(folder), toks)
+        firm = firm_rows(dtype, *load(folder), toks, entry["margins"])
         entry[dtype] = (bound(dtype, *load(folder), toks, entry["ref"], firm), firm)
     return entry["ref"] if dtype is None else (entry["ref"], *entry[dtype])
 
@@ -220,7 +221,7 @@ def test_every_cut_of_every_request_matches_plain(tmp_path, name, dtype):
                         assert err < 2 * tol, f"{what} against whole: {rid} position {pos}: {err:.3g}, bound {2 * tol:.3g}"
 
 
-@pytest.mark.parametrize("seed", [3, 12, 29, 41])
+@pytest.mark.parametrize("seed", [3, 12])
 def test_configurations_drawn_at_random_match_plain(tmp_path, seed):
     """Sizes and options that nobody chose: whole, the last 30 tokens one by one and an unequal batch, in both precisions."""
     import random
@@ -316,10 +317,11 @@ def _greedy_matches(folder, prompt, new, dtype):
     cfg, weights = load(folder)
     seq = list(prompt)
     for tok in new:
-        logits = plain_korazen.forward(cfg, weights, seq)[-1].numpy()
+        margins: list = []
+        logits = plain_korazen.forward(cfg, weights, seq, margins=margins)[-1].numpy()
         best = int(np.argmax(logits))
         gap = (logits[best] - logits[tok]) / np.sqrt((logits ** 2).mean())
-        if not firm_rows(dtype, cfg, weights, seq)[-1]:
+        if not firm_rows(dtype, cfg, weights, seq, margins)[-1]:
             seq.append(tok)                                  # a read-out that nearly cancels: go on from what was generated
             continue
         assert tok == best or (dtype == "bfloat16" and gap < 5e-2), (dtype, len(seq), tok, best, gap)
