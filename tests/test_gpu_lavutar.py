@@ -318,7 +318,7 @@ def _greedy_matches(folder, prompt, new, dtype) -> int:
         # Where a router's choice at this position is a close call, or was a toss-up a few positions back, a bfloat16 run
         # may take the other expert and so another token; the test goes on from the token that was generated.
         near = np.asarray(margins, dtype=np.float64).reshape(-1, len(seq))[:, -REACH:]
-        if dtype == "float32" or (firm_rows(dtype, cfg, weights, seq)[-1] and not (near < TOSS_UP).any()):
+        if dtype == "float32" or (not (near < TOSS_UP).any() and firm_rows(dtype, cfg, weights, seq)[-1]):
             assert tok == best or (dtype == "bfloat16" and gap < 5e-2), (dtype, len(seq), tok, best, gap)
             held += 1
         seq.append(tok)
