@@ -1,1 +1,1 @@
-from . import fetorax, korazen, lavutar, llama, raritar, zoporax  # noqa: F401  (registers LlamaForCausalLM, Fetorax, Korazen, Lavutar, Raritar and Zoporax)
+from . import fetorax, gevipel, korazen, lavutar, llama, raritar, zoporax  # noqa: F401  (registers LlamaForCausalLM, Fetorax, Gevipel, Korazen, Lavutar, Raritar and Zoporax)

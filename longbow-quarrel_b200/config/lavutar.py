@@ -179,6 +179,14 @@ class Loop:
     stop: int
     times: int
 
+    @classmethod
+    def from_dict(cls, data: dict, n_layers: int) -> "Loop":
+        r = KeyReader(data, "config.json: loop")
+        loop = cls(r.integer("start", minimum=0), r.integer("stop", minimum=1), r.integer("times", minimum=1))
+        if not loop.start < loop.stop <= n_layers:
+            raise ConfigError(f"config.json: loop: layers {loop.start} .. {loop.stop - 1} are not a stretch of the {n_layers} layers")
+        return loop
+
 
 @dataclass(frozen=True)
 class LavutarConfig:
@@ -200,11 +208,7 @@ class LavutarConfig:
         loop = None
         ld = _object(data, "loop", "config.json", required=False)
         if ld is not None:
-            lr = KeyReader(ld, "config.json: loop")
-            loop = Loop(lr.integer("start", minimum=0), lr.integer("stop", minimum=1), lr.integer("times", minimum=1))
-            if not loop.start < loop.stop <= len(layers):
-                raise ConfigError(f"config.json: loop: layers {loop.start} .. {loop.stop - 1} are not a stretch of the "
-                                  f"{len(layers)} layers")
+            loop = Loop.from_dict(ld, len(layers))
         return cls(vocab=r.integer("vocab", minimum=1), width=r.integer("width", minimum=1),
                    norm_eps=KeyReader(norm, "config.json: norm").number("eps", positive=True),
                    layers=tuple(_layer(i, layer) for i, layer in enumerate(layers)), loop=loop,

@@ -80,7 +80,7 @@ attn_decode_kernel(const __nv_bfloat16* __restrict__ q, int q_stride, const __nv
                    float* __restrict__ part_o, float* __restrict__ part_ml, int* __restrict__ counters,
                    __nv_bfloat16* __restrict__ out, int H, int Hkv, int hd, int page_size, float scale, int window,
                    int n_splits, int part_stride, const int* __restrict__ work, const char* next_w, unsigned next_piece,
-                   int early_loads, const float* __restrict__ sink, float softcap, int keep_first, int vd) {
+                   int early_loads, const float* __restrict__ sink, float softcap, int keep_first, int vd, const float* __restrict__ slope) {
     constexpr int LD = HD + PAD, LV = VD + PAD;    // shared-memory row lengths in elements: keys, values
     constexpr int RING = ring_tiles(VD);
     constexpr int KD = HD / 16;                    // k16 steps over the head dimension
@@ -204,6 +204,8 @@ attn_decode_kernel(const __nv_bfloat16* __restrict__ q, int q_stride, const __nv
     // Query heads of the group as the rows of the mma tile (rows g and g + 8 of this thread).
     const int r0 = gt * 16 + g, r1 = r0 + 8;
     const bool r0ok = r0 < G, r1ok = r1 < G;
+    // What the rows' scores lose per position of distance.
+    const float fall0 = (slope && r0ok) ? slope[kvh * G + r0] : 0.f, fall1 = (slope && r1ok) ? slope[kvh * G + r1] : 0.f;
     const __nv_bfloat16* q0p = q + (size_t)tok * q_stride + (size_t)(kvh * G + (r0ok ? r0 : 0)) * hd;
     const __nv_bfloat16* q1p = q + (size_t)tok * q_stride + (size_t)(kvh * G + (r1ok ? r1 : 0)) * hd;
     uint32_t qf[KD][4];
@@ -258,6 +260,10 @@ attn_decode_kernel(const __nv_bfloat16* __restrict__ q, int q_stride, const __nv
                 if (softcap > 0.f) {              // score <- c tanh(score / c)
                     a = softcap * tanh_fast(a * inv_cap);
                     b = softcap * tanh_fast(b * inv_cap);
+                }
+                if (slope) {
+                    a = fmaf(fall0, (float)(key - pos), a);
+                    b = fmaf(fall1, (float)(key - pos), b);
                 }
                 s[nt][i] = ok ? a : -CUDART_INF_F;
                 s[nt][2 + i] = ok ? b : -CUDART_INF_F;
@@ -430,7 +436,7 @@ int launch(const void* q, int q_stride, const void* k_pages, const void* v_pages
            const int* tok_pos, const int* tok_seq, const int* slots, float* part_o, float* part_ml, int* counters,
            void* out, int T, int H, int Hkv, int hd, int page_size, float scale, int window, int n_splits,
            const int* work, int teams, const void* next_w, long next_bytes, int early_loads, const float* sink,
-           float softcap, int keep_first, int vd, cudaStream_t stream) {
+           float softcap, int keep_first, int vd, const float* slope, cudaStream_t stream) {
     int G = H / Hkv, gtiles = (G + 15) / 16;
     dim3 grid(n_splits, Hkv * gtiles, T);
     if (work) grid = dim3(Hkv * gtiles, teams, 1);      // n_splits is then the room for parts per token in the scratch
@@ -450,7 +456,7 @@ int launch(const void* q, int q_stride, const void* k_pages, const void* v_pages
     int rc = launch_pdl(attn_decode_kernel<HD, VD>, grid, dim3(DW * 32), smem, stream, (const __nv_bfloat16*)q, q_stride,
         (const __nv_bfloat16*)k_pages, (const __nv_bfloat16*)v_pages, page_table, pt_stride, tok_pos, tok_seq, slots,
         part_o, part_ml, counters, (__nv_bfloat16*)out, H, Hkv, hd, page_size, scale, window, n_splits, n_splits, work,
-        (const char*)next_w, (unsigned)piece, early_loads, sink, softcap, keep_first, vd);
+        (const char*)next_w, (unsigned)piece, early_loads, sink, softcap, keep_first, vd, slope);
     if (rc != LQ_OK || n_splits == 1 || counters != nullptr) return rc;
     return launch_pdl(attn_merge_kernel, dim3(T * H), dim3(128), 0, stream, (const float*)part_o, (const float*)part_ml,
                       (__nv_bfloat16*)out, vd, n_splits, H, sink);
@@ -491,12 +497,14 @@ bool sizes_ok(int H, int Hkv, int hd, int page_size, int q_stride, int n_splits)
 //
 // vd: the size of a value head (a multiple of 8, at most 256), where it is another than hd; out is [T, H*vd] and the
 // scratch holds rows of vd.
+//
+// slope (or null): float32 [H]; a score loses slope[h] times the distance to its key (after the scale and the cap).
 LQ_EXPORT int lq_attn_decode_vd(const void* q, int q_stride, const void* k_pages, const void* v_pages,
                                 const int* page_table, int pt_stride, const int* tok_pos, const int* tok_seq,
                                 const int* slots, float* part_o, float* part_ml, int* counters, void* out, int T,
                                 int H, int Hkv, int hd, int vd, int page_size, float scale, int window, int n_splits,
                                 const int* work, int teams, const void* next_w, long next_bytes, int early_loads,
-                                const float* sink, float softcap, int keep_first, cudaStream_t stream) {
+                                const float* sink, float softcap, int keep_first, const float* slope, cudaStream_t stream) {
     if (T <= 0) return LQ_OK;
     if (!sizes_ok(H, Hkv, hd, page_size, q_stride, n_splits) || vd <= 0 || vd % 8 || vd > 256) return LQ_BAD_SIZE;
     if (n_splits > 1 && (!part_o || !part_ml)) return LQ_BAD_SIZE;
@@ -504,7 +512,7 @@ LQ_EXPORT int lq_attn_decode_vd(const void* q, int q_stride, const void* k_pages
     if (softcap < 0.f || keep_first < 0) return LQ_BAD_SIZE;
 #define LQ_GO(HD, VD) return launch<HD, VD>(q, q_stride, k_pages, v_pages, page_table, pt_stride, tok_pos, tok_seq, slots, \
                                             part_o, part_ml, counters, out, T, H, Hkv, hd, page_size, scale, window, n_splits, \
-                                            work, teams, next_w, next_bytes, early_loads, sink, softcap, keep_first, vd, stream)
+                                            work, teams, next_w, next_bytes, early_loads, sink, softcap, keep_first, vd, slope, stream)
     if (vd > 128) LQ_GO(128, 256);
     if (hd <= 32 && vd <= 32) LQ_GO(32, 32);
     if (hd <= 64 && vd <= 64) LQ_GO(64, 64);
@@ -521,7 +529,7 @@ LQ_EXPORT int lq_attn_decode_capped(const void* q, int q_stride, const void* k_p
                                     const float* sink, float softcap, int keep_first, cudaStream_t stream) {
     return lq_attn_decode_vd(q, q_stride, k_pages, v_pages, page_table, pt_stride, tok_pos, tok_seq, slots, part_o, part_ml, counters,
                              out, T, H, Hkv, hd, hd, page_size, scale, window, n_splits, work, teams, next_w, next_bytes, early_loads,
-                             sink, softcap, keep_first, stream);
+                             sink, softcap, keep_first, nullptr, stream);
 }
 
 LQ_EXPORT int lq_attn_decode_sink(const void* q, int q_stride, const void* k_pages, const void* v_pages,

@@ -66,7 +66,7 @@ attn_prefill_kernel(const __nv_bfloat16* __restrict__ q, int q_stride, const __n
                     const int* __restrict__ slots, const int* __restrict__ kv_len, const int* __restrict__ qb_seq,
                     const int* __restrict__ qb_row, const int* __restrict__ qb_rows, const int* __restrict__ qb_pos,
                     __nv_bfloat16* __restrict__ out, int H, int Hkv, int hd, float scale_log2, int window, const float* __restrict__ sink,
-                    float cap_pre, int keep_first, int vd) {
+                    float cap_pre, int keep_first, int vd, const float* __restrict__ slope) {
     constexpr int LD = HD + PAD, LV = VD + PAD;        // shared-memory row lengths in elements: queries and keys, values
     constexpr int KD = HD / 16;                        // k16 steps over the head dimension
     extern __shared__ __align__(16) uint8_t smem_raw[];
@@ -136,6 +136,7 @@ attn_prefill_kernel(const __nv_bfloat16* __restrict__ q, int q_stride, const __n
     const bool row0ok = warp * 16 + g < n_rows, row1ok = warp * 16 + g + 8 < n_rows;
     const int warp_pos_hi = min(pos_last, pos0 + warp * 16 + 15);        // last position any row of the warp has
     const int warp_key_lo = lq_first_key(pos0 + warp * 16, window);
+    const float fall = slope ? slope[h] * 1.4426950408889634f : 0.f;     // what a score loses per position of distance
 
     for (int n = 0; n < n_tiles; ++n) {
         const int stage = n & 1, tile = tile_at(n);
@@ -189,8 +190,14 @@ attn_prefill_kernel(const __nv_bfloat16* __restrict__ q, int q_stride, const __n
                         a = tanh_fast(a * cap_pre);
                         b = tanh_fast(b * cap_pre);
                     }
-                    s[j][i] = ok0 ? a * scale_log2 : -CUDART_INF_F;
-                    s[j][2 + i] = ok1 ? b * scale_log2 : -CUDART_INF_F;
+                    a *= scale_log2;
+                    b *= scale_log2;
+                    if (slope) {
+                        a = fmaf(fall, (float)(key - prow0), a);
+                        b = fmaf(fall, (float)(key - prow1), b);
+                    }
+                    s[j][i] = ok0 ? a : -CUDART_INF_F;
+                    s[j][2 + i] = ok1 ? b : -CUDART_INF_F;
                     tm0 = fmaxf(tm0, s[j][i]);
                     tm1 = fmaxf(tm1, s[j][2 + i]);
                 }
@@ -266,7 +273,7 @@ template <int HD, int VD>
 int launch(const void* q, int q_stride, const void* k_pages, const void* v_pages, const int* page_table, int pt_stride,
            const int* slots, const int* kv_len, const int* qb_seq, const int* qb_row, const int* qb_rows,
            const int* qb_pos, void* out, int n_blocks, int H, int Hkv, int hd, float scale, int window,
-           const float* sink, float softcap, int keep_first, int vd, cudaStream_t stream) {
+           const float* sink, float softcap, int keep_first, int vd, const float* slope, cudaStream_t stream) {
     constexpr size_t smem = ((size_t)(BLOCK_M + 2 * BLOCK_N) * (HD + PAD) + (size_t)2 * BLOCK_N * (VD + PAD)) * 2;
     static bool configured = false;
     if (!configured) {
@@ -278,7 +285,7 @@ int launch(const void* q, int q_stride, const void* k_pages, const void* v_pages
     return launch_pdl(attn_prefill_kernel<HD, VD>, grid, dim3(NT), smem, stream, (const __nv_bfloat16*)q, q_stride,
         (const __nv_bfloat16*)k_pages, (const __nv_bfloat16*)v_pages, page_table, pt_stride, slots, kv_len, qb_seq, qb_row,
         qb_rows, qb_pos, (__nv_bfloat16*)out, H, Hkv, hd, (softcap > 0.f ? softcap : scale) * 1.4426950408889634f, window, sink,
-        softcap > 0.f ? scale / softcap : 0.f, keep_first, vd);
+        softcap > 0.f ? scale / softcap : 0.f, keep_first, vd, slope);
 }
 
 }  // namespace
@@ -288,19 +295,20 @@ int launch(const void* q, int q_stride, const void* k_pages, const void* v_pages
 // head_dim a multiple of 8 and at most 128, a value head's size vd one at most 256; the cache's page size must be 64.
 // sink (or null): float32 [H]; each head's softmax denominator gets one more term exp(sink[h]).
 // softcap c (0: none): score <- c tanh(score / c) after the scale.  keep_first n (0: none; with a window): a row's
-// first n keys stay visible when its window has moved past them.
+// first n keys stay visible when its window has moved past them.  slope (or null): float32 [H]; a score then loses slope[h]
+// times the distance to its key (after the scale and the cap).
 LQ_EXPORT int lq_attn_prefill_vd(const void* q, int q_stride, const void* k_pages, const void* v_pages,
                                  const int* page_table, int pt_stride, const int* slots, const int* kv_len,
                                  const int* qb_seq, const int* qb_row, const int* qb_rows, const int* qb_pos, void* out,
                                  int n_blocks, int H, int Hkv, int hd, int vd, int page_size, float scale, int window,
-                                 const float* sink, float softcap, int keep_first, cudaStream_t stream) {
+                                 const float* sink, float softcap, int keep_first, const float* slope, cudaStream_t stream) {
     if (n_blocks <= 0) return LQ_OK;
     if (softcap < 0.f || keep_first < 0) return LQ_BAD_SIZE;
     if (hd % 8 || hd > 128 || hd <= 0 || vd % 8 || vd > 256 || vd <= 0 || H % Hkv || page_size != BLOCK_N || q_stride % 8)
         return LQ_BAD_SIZE;
 #define LQ_GO(HD, VD) return launch<HD, VD>(q, q_stride, k_pages, v_pages, page_table, pt_stride, slots, kv_len, qb_seq, qb_row, \
                                             qb_rows, qb_pos, out, n_blocks, H, Hkv, hd, scale, window, sink, softcap, keep_first, \
-                                            vd, stream)
+                                            vd, slope, stream)
     if (vd > 128) LQ_GO(128, 256);
     if (hd <= 32 && vd <= 32) LQ_GO(32, 32);
     if (hd <= 64 && vd <= 64) LQ_GO(64, 64);
@@ -316,7 +324,7 @@ LQ_EXPORT int lq_attn_prefill_capped(const void* q, int q_stride, const void* k_
                                      int n_blocks, int H, int Hkv, int hd, int page_size, float scale, int window,
                                      const float* sink, float softcap, int keep_first, cudaStream_t stream) {
     return lq_attn_prefill_vd(q, q_stride, k_pages, v_pages, page_table, pt_stride, slots, kv_len, qb_seq, qb_row, qb_rows, qb_pos,
-                              out, n_blocks, H, Hkv, hd, hd, page_size, scale, window, sink, softcap, keep_first, stream);
+                              out, n_blocks, H, Hkv, hd, hd, page_size, scale, window, sink, softcap, keep_first, nullptr, stream);
 }
 
 LQ_EXPORT int lq_attn_prefill(const void* q, int q_stride, const void* k_pages, const void* v_pages,

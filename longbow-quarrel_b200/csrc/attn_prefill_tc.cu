@@ -100,7 +100,7 @@ attn_prefill_tc_kernel(const __grid_constant__ CUtensorMap map_q, const __grid_c
                        const int* __restrict__ slots, const int* __restrict__ kv_len, const int* __restrict__ qb_seq,
                        const int* __restrict__ qb_row, const int* __restrict__ qb_rows, const int* __restrict__ qb_pos,
                        __nv_bfloat16* __restrict__ out, int H, int Hkv, int oob_row, float scale_log2, int window,
-                       const float* __restrict__ sink, float cap_pre, int keep_first) {
+                       const float* __restrict__ sink, float cap_pre, int keep_first, const float* __restrict__ slope) {
     extern __shared__ uint8_t smem_raw[];
     constexpr int DH = HD / 64;                  // panels of 64 elements along the head dimension
     Smem<HD>& sm = *reinterpret_cast<Smem<HD>*>((reinterpret_cast<uintptr_t>(smem_raw) + 1023) & ~(uintptr_t)1023);
@@ -226,6 +226,8 @@ attn_prefill_tc_kernel(const __grid_constant__ CUtensorMap map_q, const __grid_c
         const uint32_t lane_base = (uint32_t)(quarter * 32) << 16;
         const int pos_r = pos0 + r;
         const int first_r = lq_first_key(pos_r, window);      // the first key this row sees
+        // What a raw score loses per position of distance (the exponent's scale is applied afterwards).
+        const float fall = slope ? slope[h] * 1.4426950408889634f / scale_log2 : 0.f;
         const bool row_ok = r < n_rows;
         constexpr int NC = BN / PARTS;                    // keys of a tile of this thread
         constexpr int OC = HD / PARTS;                    // output columns of this thread
@@ -247,6 +249,11 @@ attn_prefill_tc_kernel(const __grid_constant__ CUtensorMap map_q, const __grid_c
             if (cap_pre > 0.f) {                          // capped scores: t <- tanh(t scale / c); scale_log2 is then c log2(e)
 #pragma unroll
                 for (int c = 0; c < NC; ++c) t[c] = tanh_fast(t[c] * cap_pre);
+            }
+            if (slope) {
+                const float back = fall * (float)(kb - pos_r);
+#pragma unroll
+                for (int c = 0; c < NC; ++c) t[c] += fmaf(fall, (float)c, back);
             }
             // Tiles that lie wholly inside every row's range (most of them) need no mask.
             const bool whole = n_rows == BM && tb + BN - 1 <= pos0 && tb + BN <= len && tb >= first_last;
@@ -386,7 +393,7 @@ attn_prefill_two_kernel(const __grid_constant__ CUtensorMap map_q, const __grid_
                         const int* __restrict__ slots, const int* __restrict__ kv_len, const int* __restrict__ qb_seq,
                         const int* __restrict__ qb_row, const int* __restrict__ qb_rows, const int* __restrict__ qb_pos,
                         __nv_bfloat16* __restrict__ out, int H, int Hkv, int oob_row, float scale_log2, int window,
-                        const float* __restrict__ sink, float cap_pre, int keep_first) {
+                        const float* __restrict__ sink, float cap_pre, int keep_first, const float* __restrict__ slope) {
     extern __shared__ uint8_t smem_raw[];
     constexpr int DH = HD / 64;
     Smem2<HD>& sm = *reinterpret_cast<Smem2<HD>*>((reinterpret_cast<uintptr_t>(smem_raw) + 1023) & ~(uintptr_t)1023);
@@ -514,6 +521,8 @@ attn_prefill_two_kernel(const __grid_constant__ CUtensorMap map_q, const __grid_
         const uint32_t tmem_o = tmem_base + 2 * BN + chain * HD + lane_base;
         const int pos_r = pos0 + r;
         const int first_r = lq_first_key(pos_r, window);      // the first key this row sees
+        // What a raw score loses per position of distance (the exponent's scale is applied afterwards).
+        const float fall = slope ? slope[h] * 1.4426950408889634f / scale_log2 : 0.f;
         const bool row_ok = r < n_rows;
         float m_ref = -CUDART_INF_F, l = 0.f;
         bool ok = true;
@@ -529,6 +538,11 @@ attn_prefill_two_kernel(const __grid_constant__ CUtensorMap map_q, const __grid_
             if (cap_pre > 0.f) {                          // capped scores: t <- tanh(t scale / c); scale_log2 is then c log2(e)
 #pragma unroll
                 for (int c = 0; c < BN; ++c) t[c] = tanh_fast(t[c] * cap_pre);
+            }
+            if (slope) {
+                const float back = fall * (float)(kb - pos_r);
+#pragma unroll
+                for (int c = 0; c < BN; ++c) t[c] += fmaf(fall, (float)c, back);
             }
             const bool whole = n_rows == BM && kb + BN - 1 <= pos0 && kb + BN <= len && kb >= first_last;
             float mx[4] = {-CUDART_INF_F, -CUDART_INF_F, -CUDART_INF_F, -CUDART_INF_F};
@@ -619,7 +633,7 @@ template <int HD>
 int launch_hd(const void* q, int q_stride, int T, const void* k_pages, const void* v_pages, int n_pages,
               const int* page_table, int pt_stride, const int* slots, const int* kv_len, const int* qb_seq,
               const int* qb_row, const int* qb_rows, const int* qb_pos, void* out, int n_blocks, int H, int Hkv,
-              float scale, int window, const float* sink, float softcap, int keep_first, cudaStream_t stream) {
+              float scale, int window, const float* sink, float softcap, int keep_first, const float* slope, cudaStream_t stream) {
     CUtensorMap mq, mk, mv;
     // Capped scores: the kernels take tanh(s scale / c) and multiply by c log2(e) inside the exponent.
     const float cap_pre = softcap > 0.f ? scale / softcap : 0.f;
@@ -649,11 +663,11 @@ int launch_hd(const void* q, int q_stride, int T, const void* k_pages, const voi
         }
         return launch_pdl(attn_prefill_two_kernel<HD>, dim3(n_blocks * (H / 2)), dim3(N_THREADS2), smem2, stream, mq, mk, mv,
                           page_table, pt_stride, slots, kv_len, qb_seq, qb_row, qb_rows, qb_pos, (__nv_bfloat16*)out, H, Hkv,
-                          (int)kv_rows, scale_log2, window, sink, cap_pre, keep_first);
+                          (int)kv_rows, scale_log2, window, sink, cap_pre, keep_first, slope);
     }
     return launch_pdl(attn_prefill_tc_kernel<HD>, dim3(n_blocks * H), dim3(N_THREADS), smem, stream, mq, mk, mv, page_table,
                       pt_stride, slots, kv_len, qb_seq, qb_row, qb_rows, qb_pos, (__nv_bfloat16*)out, H, Hkv,
-                      (int)kv_rows, scale_log2, window, sink, cap_pre, keep_first);
+                      (int)kv_rows, scale_log2, window, sink, cap_pre, keep_first, slope);
 }
 }  // namespace
 
@@ -662,20 +676,21 @@ int launch_hd(const void* q, int q_stride, int T, const void* k_pages, const voi
 // qb_*: the work list, n_blocks entries: sequence, first packed row, rows (<= 128), position of the first row.
 // sink (or null): float32 [H]; each head's softmax denominator gets one more term exp(sink[h]).
 // softcap c (0: none): score <- c tanh(score / c) after the scale.  keep_first n (0: none; with a window): a row's
-// first n keys stay visible when its window has moved past them.
+// first n keys stay visible when its window has moved past them.  slope (or null): float32 [H]; a score then loses slope[h]
+// times the distance to its key (after the scale and the cap).
 LQ_EXPORT int lq_attn_prefill_tc_capped(const void* q, int q_stride, int T, const void* k_pages, const void* v_pages,
                                  int n_pages, const int* page_table, int pt_stride, const int* slots, const int* kv_len,
                                  const int* qb_seq, const int* qb_row, const int* qb_rows, const int* qb_pos, void* out,
                                  int n_blocks, int H, int Hkv, int hd, int page_size, float scale, int window,
-                                 const float* sink, float softcap, int keep_first, cudaStream_t stream) {
+                                 const float* sink, float softcap, int keep_first, const float* slope, cudaStream_t stream) {
     if (n_blocks <= 0) return LQ_OK;
     if (softcap < 0.f || keep_first < 0 || scale <= 0.f) return LQ_BAD_SIZE;
     if ((hd != 64 && hd != 128) || page_size != PAGE || H % Hkv || q_stride % 8 || ((uintptr_t)q & 15)) return LQ_BAD_SIZE;
     if (hd == 64)
         return launch_hd<64>(q, q_stride, T, k_pages, v_pages, n_pages, page_table, pt_stride, slots, kv_len, qb_seq, qb_row,
-                             qb_rows, qb_pos, out, n_blocks, H, Hkv, scale, window, sink, softcap, keep_first, stream);
+                             qb_rows, qb_pos, out, n_blocks, H, Hkv, scale, window, sink, softcap, keep_first, slope, stream);
     return launch_hd<128>(q, q_stride, T, k_pages, v_pages, n_pages, page_table, pt_stride, slots, kv_len, qb_seq, qb_row,
-                          qb_rows, qb_pos, out, n_blocks, H, Hkv, scale, window, sink, softcap, keep_first, stream);
+                          qb_rows, qb_pos, out, n_blocks, H, Hkv, scale, window, sink, softcap, keep_first, slope, stream);
 }
 
 LQ_EXPORT int lq_attn_prefill_tc(const void* q, int q_stride, int T, const void* k_pages, const void* v_pages,
@@ -685,7 +700,7 @@ LQ_EXPORT int lq_attn_prefill_tc(const void* q, int q_stride, int T, const void*
                                  const float* sink, cudaStream_t stream) {
     return lq_attn_prefill_tc_capped(q, q_stride, T, k_pages, v_pages, n_pages, page_table, pt_stride, slots, kv_len, qb_seq,
                                      qb_row, qb_rows, qb_pos, out, n_blocks, H, Hkv, hd, page_size, scale, window, sink, 0.f, 0,
-                                     stream);
+                                     nullptr, stream);
 }
 
 LQ_EXPORT int lq_attn_prefill_tc_status() { return tc::status_read(); }

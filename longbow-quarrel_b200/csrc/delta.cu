@@ -24,41 +24,17 @@
 //
 // Single tokens (one kernel, delta_single_kernel): convolution, unit vectors, the decays' and the output gate's second
 // products (over their small inner sizes), the recurrence, the head's norm and the gate; the state is read and written once.
+// The same kernel without the second products serves the rule with one decay per head (head_delta.cu has its prompts).
 //
 // The convolution's last inputs are kept per slot as a ring of `taps` rows, the row of position p at p % taps: a step
 // of one token writes a row that it does not read.
-#include "tcgen05.cuh"
+#include "delta.cuh"
 
 constexpr int DC = 4;                 // tokens of a record
 // Scalars of a record: b [4], M [4][4] (t, s), N [4][4]; or N alone.
 template <bool RULE> constexpr int scalars() { return RULE ? 4 + 16 + 16 : 16; }
 // Vectors of a record over the key channels: A_t k_t [DC], A_t q_t [DC], decayed k_s [DC], A_DC - 1; without the first DC.
 template <bool RULE> constexpr int vectors() { return RULE ? 3 * DC + 1 : 2 * DC + 1; }
-
-typedef unsigned long long f2;        // two float32 side by side
-__device__ __forceinline__ f2 fma2(f2 a, f2 b, f2 c) {
-    f2 d;
-    asm("fma.rn.f32x2 %0, %1, %2, %3;" : "=l"(d) : "l"(a), "l"(b), "l"(c));
-    return d;
-}
-__device__ __forceinline__ f2 pack2(float lo, float hi) {
-    f2 d;
-    asm("mov.b64 %0, {%1, %2};" : "=l"(d) : "f"(lo), "f"(hi));
-    return d;
-}
-__device__ __forceinline__ float2 unpack2(f2 v) {
-    float2 r;
-    asm("mov.b64 {%0, %1}, %2;" : "=f"(r.x), "=f"(r.y) : "l"(v));
-    return r;
-}
-// An untiled bulk copy into this block's shared memory; both addresses and the size in whole sixteens.
-__device__ __forceinline__ void bulk_load(uint32_t dst, const void* src, uint32_t bytes, uint32_t bar) {
-    asm volatile("cp.async.bulk.shared::cluster.global.mbarrier::complete_tx::bytes [%0], [%1], %2, [%3];"
-                 ::"r"(dst), "l"(src), "r"(bytes), "r"(bar) : "memory");
-}
-__device__ __forceinline__ float sigmoid_f(float x) { return __frcp_rn(1.f + expf(-x)); }
-__device__ __forceinline__ float silu_f(float x) { return x * sigmoid_f(x); }
-__device__ __forceinline__ float softplus_f(float x) { return fmaxf(x, 0.f) + log1pf(expf(-fabsf(x))); }
 
 struct DeltaArgs {
     const float* rows;           // [T, stride]: q at column 0, then k (G * dk each), v (H * dv), b (H), ...
@@ -634,6 +610,8 @@ struct DeltaSingleArgs {
     int out_bf16;
     int cg;                      // threads side by side along a row of the state
 };
+// With one decay per head a_off and g_off are the columns of the decays' pre-activations [H] and of the output gate [H, dv]
+// themselves, z_bias and rate are [H], and the gate is silu; there are no second products.
 
 template <typename TW> __device__ __forceinline__ float dot_row(const TW* w, const float* x, int n);
 template <> __device__ __forceinline__ float dot_row<float>(const float* w, const float* x, int n) {
@@ -664,7 +642,7 @@ template <> __device__ __forceinline__ float dot_row<__nv_bfloat16>(const __nv_b
 // neighbouring columns of up to KR rows in registers between the read and the write.  Columns beyond cg * VW take
 // another turn.
 constexpr int DT_THREADS = 256;
-template <typename TW, int KR, int VW>
+template <typename TW, int KR, int VW, bool HEAD>
 __global__ void __launch_bounds__(DT_THREADS) delta_single_kernel(DeltaSingleArgs s) {
     pdl_launch_dependents();
     extern __shared__ __align__(16) float sm[];
@@ -705,6 +683,7 @@ __global__ void __launch_bounds__(DT_THREADS) delta_single_kernel(DeltaSingleArg
         }
     };
     load_state(cl * VW);
+    if constexpr (!HEAD)
     for (int e = tid; e < dk + dv; e += DT_THREADS) {
         const TW* w = e < dk ? (const TW*)s.a2 + (size_t)(h * dk + e) * s.ra_ld : (const TW*)s.g2 + (size_t)(h * dv + e - dk) * s.rg_ld;
         asm volatile("prefetch.global.L2 [%0];" ::"l"(w));
@@ -722,6 +701,7 @@ __global__ void __launch_bounds__(DT_THREADS) delta_single_kernel(DeltaSingleArg
         sq[e < 2 * dk ? e : dk + e] = acc;                           // sq, sk, (sa), sv lie one after another
     }
     pdl_wait();
+    if constexpr (!HEAD)
     for (int i = tid; i < s.ra_ld + s.rg_ld; i += DT_THREADS)
         xa[i] = i < s.ra_ld ? (i < s.ra ? x[s.a_off + i] : 0.f) : (i - s.ra_ld < s.rg ? x[s.g_off + i - s.ra_ld] : 0.f);
     for (int e = tid; e < 2 * dk + dv; e += DT_THREADS) {
@@ -749,6 +729,11 @@ __global__ void __launch_bounds__(DT_THREADS) delta_single_kernel(DeltaSingleArg
             sums[2] = qk * sums[0] * sums[1];
         }
     }
+    float head_decay = 0.f;                      // less one
+    if constexpr (HEAD) {
+        head_decay = expm1f(-a.rate[h] * softplus_f(x[s.a_off + h] + a.z_bias[h]));
+        for (int e = tid; e < dv; e += DT_THREADS) sgate[e] = silu_f(x[s.g_off + h * dv + e]);
+    } else
     for (int e = tid; e < dk + dv; e += DT_THREADS) {
         if (e < dk) {
             const float z = dot_row<TW>((const TW*)s.a2 + (size_t)(h * dk + e) * s.ra_ld, xa, s.ra_ld) + a.z_bias[h * dk + e];
@@ -774,7 +759,7 @@ __global__ void __launch_bounds__(DT_THREADS) delta_single_kernel(DeltaSingleArg
         for (int i = 0; i < KR; ++i) {
             const int r = group + i * rg;
             if (live && r < dk) {
-                const float d = sa[r], k = sk[r], q = sq[r];
+                const float d = HEAD ? head_decay : sa[r], k = sk[r], q = sq[r];
 #pragma unroll
                 for (int v = 0; v < VW; ++v) {
                     S[i][v] = fmaf(S[i][v], d, S[i][v]);
@@ -841,7 +826,7 @@ __global__ void __launch_bounds__(DT_THREADS) delta_single_kernel(DeltaSingleArg
     }
 }
 
-template <typename TW>
+template <typename TW, bool HEAD = false>
 static int single_launch(DeltaSingleArgs& s, int B, cudaStream_t stream) {
     const int dk = s.d.dk, dv = s.d.dv, vw = dv % 4 == 0 ? 4 : 1;
     // As many threads along a row as there are columns, unless that leaves a thread too many rows.
@@ -858,11 +843,11 @@ static int single_launch(DeltaSingleArgs& s, int B, cudaStream_t stream) {
         return launch_pdl(kernel, dim3(B, s.d.H), dim3(DT_THREADS), smem, stream, s);
     };
     if (vw == 4) {
-        if (kr <= 4) return go(delta_single_kernel<TW, 4, 4>);
-        if (kr <= 8) return go(delta_single_kernel<TW, 8, 4>);
-        return go(delta_single_kernel<TW, 16, 4>);
+        if (kr <= 4) return go(delta_single_kernel<TW, 4, 4, HEAD>);
+        if (kr <= 8) return go(delta_single_kernel<TW, 8, 4, HEAD>);
+        return go(delta_single_kernel<TW, 16, 4, HEAD>);
     }
-    return go(delta_single_kernel<TW, 16, 1>);
+    return go(delta_single_kernel<TW, 16, 1, HEAD>);
 }
 
 // One token per sequence (row cu_rows[b] of rows): out [B, H dv], normed and gated.
@@ -881,4 +866,19 @@ LQ_EXPORT int lq_delta_single(const float* rows, int stride, int b_off, const fl
     if (w_dtype == LQ_F32) return single_launch<float>(s, B, stream);
     if (w_dtype == LQ_BF16) return single_launch<__nv_bfloat16>(s, B, stream);
     return LQ_BAD_DTYPE;
+}
+
+// The same with one decay per head (z_bias and rate [H]): rows hold the decays' pre-activations at column a_off [H] and the
+// output gate's at g_off [H, dv]; out [B, H dv] = the head over its root mean square times norm_w times silu(gate).
+LQ_EXPORT int lq_head_delta_single(const float* rows, int stride, int b_off, const float* taps_w, int taps, float* ring,
+                                   const float* z_bias, const float* rate, float* state, const int* cu_rows, const int* slots,
+                                   const int* tok_pos, int a_off, int g_off, const float* norm_w, float norm_eps, void* out, int out_dtype,
+                                   int B, int H, int G, int dk, int dv, float q_scale, float unit_eps, cudaStream_t stream) {
+    if (B <= 0) return LQ_OK;
+    if (dk < 1 || dk > 256 || dv < 1 || dv > 4096 || G < 1 || H % G || taps < 1) return LQ_BAD_SIZE;
+    if (out_dtype != LQ_F32 && out_dtype != LQ_BF16) return LQ_BAD_DTYPE;
+    DeltaSingleArgs s{{rows, stride, b_off, taps_w, taps, 2 * G * dk + H * dv, ring, nullptr, z_bias, rate, state, cu_rows, slots, tok_pos,
+                       nullptr, nullptr, H, G, dk, dv, q_scale, unit_eps},
+                      a_off, 0, g_off, 0, nullptr, nullptr, 0, 0, norm_w, norm_eps, out, out_dtype == LQ_BF16, 1};
+    return single_launch<float, true>(s, B, stream);
 }

@@ -44,13 +44,14 @@ __device__ __forceinline__ void mma_bf16(float (&c)[4], uint32_t a0, uint32_t a1
                  : "r"(a0), "r"(a1), "r"(a2), "r"(a3), "r"(b0), "r"(b1));
 }
 
-// act: 0 none, 1 gelu (erf), 2 gelu (tanh form), 3 silu, 4 relu
+// act: 0 none, 1 gelu (erf), 2 gelu (tanh form), 3 silu, 4 relu, 5 the square of relu
 __device__ __forceinline__ float gg_act(float v, int act) {
     switch (act) {
         case 1: return 0.5f * v * (1.f + erff(v * 0.70710678118654752f));
         case 2: return 0.5f * v * (1.f + tanhf(0.7978845608028654f * (v + 0.044715f * v * v * v)));
         case 3: return v / (1.f + expf(-v));
         case 4: return fmaxf(v, 0.f);
+        case 5: { const float r = fmaxf(v, 0.f); return r * r; }
         default: return v;
     }
 }
@@ -298,7 +299,7 @@ LQ_EXPORT int lq_grouped_gemm(const void* A, long long lda, long long a_group_st
                               const int* rows, const int* group_off, const int* tile_off, int n_listed, int G, int M, int N,
                               int K, int act, cudaStream_t stream) {
     if (G <= 0 || N <= 0) return LQ_OK;
-    if (K % 8 || lda % 8 || a_group_stride % 8 || w_group_stride % 8 || a_div < 1 || act < 0 || act > 4) return LQ_BAD_SIZE;
+    if (K % 8 || lda % 8 || a_group_stride % 8 || w_group_stride % 8 || a_div < 1 || act < 0 || act > 5) return LQ_BAD_SIZE;
     if (((uintptr_t)A | (uintptr_t)W) & 15) return LQ_BAD_SIZE;
     if (rows ? (!group_off || !tile_off || n_listed <= 0) : M <= 0) return LQ_BAD_SIZE;
     GroupedArgs a{(const __nv_bfloat16*)A, lda, a_group_stride, a_div, (const __nv_bfloat16*)W, w_group_stride, out, ldo,

@@ -177,6 +177,7 @@ LQ_EXPORT int lq_head_matmul(const void* in, int in_dtype, int in_stride, int in
 // (window 0: all).  grid = (T, ceil(H / LA_WARPS), splits): a block takes one row, up to LA_WARPS heads (a warp
 // each) and one slice of the row's keys; tiles of 32 keys are staged in shared memory as float32 once for all
 // the block's heads; lane j takes key j's score, then the lanes share out the R value columns.
+// sink (or null): [H], one more term exp(sink[h]) of each head's denominator, with no key and no value.
 // With splits > 1 a block leaves (max, sum, unnormalised mean) in scratch and lq_latent_merge finishes the row.
 constexpr int LA_WARPS = 8;
 constexpr int LA_KEYS = 32;
@@ -186,7 +187,7 @@ __global__ void __launch_bounds__(LA_WARPS * 32) latent_attention_kernel(
         const float* __restrict__ q, const TC* __restrict__ pages, const int* __restrict__ page_table, int pt_stride,
         const int* __restrict__ tok_pos, const int* __restrict__ tok_seq, const int* __restrict__ slots,
         float* __restrict__ out, float* __restrict__ part_o, float* __restrict__ part_ml,
-        int H, int R, int Dk, int page_size, float scale, int window, int splits) {
+        int H, int R, int Dk, int page_size, float scale, int window, int splits, const float* __restrict__ sink) {
     pdl_launch_dependents();
     extern __shared__ float sm[];
     const int ld = Dk | 1;                                  // odd: lane j's row starts in its own bank
@@ -249,6 +250,12 @@ __global__ void __launch_bounds__(LA_WARPS * 32) latent_attention_kernel(
     }
     if (!live) return;
     if (splits == 1) {
+        if (sink) {                                        // one more term of the denominator, without a key
+            const float s = sink[h], m_new = fmaxf(m, s), alpha = expf(m - m_new);
+            l = l * alpha + expf(s - m_new);
+#pragma unroll
+            for (int i = 0; i < NACC; ++i) acc[i] *= alpha;
+        }
         const float inv = 1.f / l;
         float* o = out + ((size_t)t * H + h) * R;
 #pragma unroll
@@ -269,15 +276,16 @@ __global__ void __launch_bounds__(LA_WARPS * 32) latent_attention_kernel(
 
 // One warp per (row, head): the slices' results combined in the order of the slices.
 __global__ void __launch_bounds__(128) latent_merge_kernel(const float* __restrict__ part_o, const float* __restrict__ part_ml,
-                                                           float* __restrict__ out, int n_pairs, int R, int splits) {
+                                                           float* __restrict__ out, int n_pairs, int R, int splits,
+                                                           const float* __restrict__ sink, int H) {
     pdl_launch_dependents();
     pdl_wait();
     const int pair = blockIdx.x * 4 + (threadIdx.x >> 5), lane = threadIdx.x & 31;
     if (pair >= n_pairs) return;
     const float* ml = part_ml + (size_t)pair * splits * 2;
-    float m = -CUDART_INF_F;
+    float m = sink ? sink[pair % H] : -CUDART_INF_F;
     for (int s = 0; s < splits; ++s) m = fmaxf(m, ml[2 * s]);
-    float l = 0.f;
+    float l = sink ? expf(sink[pair % H] - m) : 0.f;
     for (int s = 0; s < splits; ++s) l += ml[2 * s] == -CUDART_INF_F ? 0.f : ml[2 * s + 1] * expf(ml[2 * s] - m);
     const float inv = 1.f / l;
     for (int d = lane; d < R; d += 32) {
@@ -291,29 +299,29 @@ __global__ void __launch_bounds__(128) latent_merge_kernel(const float* __restri
 template <typename TC, int NACC>
 static int latent_attention_launch(const float* q, const void* pages, const int* page_table, int pt_stride, const int* tok_pos,
                                    const int* tok_seq, const int* slots, float* out, float* part_o, float* part_ml, int T, int H,
-                                   int R, int Dk, int page_size, float scale, int window, int splits, cudaStream_t stream) {
+                                   int R, int Dk, int page_size, float scale, int window, int splits, const float* sink, cudaStream_t stream) {
     const size_t smem = ((size_t)LA_WARPS * Dk + (size_t)LA_KEYS * (Dk + 1)) * sizeof(float);
     if (smem > 220 * 1024) return LQ_BAD_SIZE;
     auto kernel = latent_attention_kernel<TC, NACC>;
     if (smem > 48 * 1024) cudaFuncSetAttribute(kernel, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);
     dim3 grid(T, (H + LA_WARPS - 1) / LA_WARPS, splits);
     int rc = launch_pdl(kernel, grid, dim3(LA_WARPS * 32), smem, stream, q, (const TC*)pages, page_table, pt_stride, tok_pos,
-                        tok_seq, slots, out, part_o, part_ml, H, R, Dk, page_size, scale, window, splits);
+                        tok_seq, slots, out, part_o, part_ml, H, R, Dk, page_size, scale, window, splits, sink);
     if (rc != LQ_OK || splits == 1) return rc;
     const int n = T * H;
     return launch_pdl(latent_merge_kernel, dim3((n + 3) / 4), dim3(128), 0, stream, (const float*)part_o, (const float*)part_ml,
-                      out, n, R, splits);
+                      out, n, R, splits, sink, H);
 }
 
 LQ_EXPORT int lq_latent_attention(const float* q, const void* pages, int cache_dtype, const int* page_table, int pt_stride,
                                   const int* tok_pos, const int* tok_seq, const int* slots, float* out, float* part_o,
                                   float* part_ml, int T, int H, int R, int Dk, int page_size, float scale, int window,
-                                  int splits, cudaStream_t stream) {
+                                  int splits, const float* sink, cudaStream_t stream) {
     if (T <= 0) return LQ_OK;
     if (R < 1 || R > Dk || R > 1024 || splits < 1 || (splits > 1 && (!part_o || !part_ml))) return LQ_BAD_SIZE;
     typedef __nv_bfloat16 bf;
 #define LQ_GO(TC, NACC) return latent_attention_launch<TC, NACC>(q, pages, page_table, pt_stride, tok_pos, tok_seq, slots, out, \
-        part_o, part_ml, T, H, R, Dk, page_size, scale, window, splits, stream)
+        part_o, part_ml, T, H, R, Dk, page_size, scale, window, splits, sink, stream)
 #define LQ_BY_R(TC) do { if (R <= 64) LQ_GO(TC, 2); if (R <= 128) LQ_GO(TC, 4); if (R <= 256) LQ_GO(TC, 8); if (R <= 512) LQ_GO(TC, 16); LQ_GO(TC, 32); } while (0)
     if (cache_dtype == LQ_F32) LQ_BY_R(float);
     if (cache_dtype == LQ_BF16) LQ_BY_R(bf);

@@ -68,6 +68,7 @@ struct LatentArgs {
     int H, R, Dk, page_size, window, splits, head_blocks, chunks;
     int out_bf16;                    // the final rows go out as bfloat16 (the partial results of slices stay float32)
     float scale_log2;
+    const float* sink;               // [H] or null: one more term exp(sink[h]) of each head's denominator, with no key and no value
 };
 
 // CW: value columns that a group of four warps accumulates; NCH: groups (chunks of columns) of a block.
@@ -227,6 +228,14 @@ __global__ void __launch_bounds__(NT * NCH, 1) latent_attention_tc_kernel(Latent
     l1 += __shfl_xor_sync(0xffffffffu, l1, 1);
     l1 += __shfl_xor_sync(0xffffffffu, l1, 2);
     const bool whole = a.splits == 1;
+    if (a.sink && whole) {           // (slices get it when they are merged)
+        const float s0 = a.sink[h0 + r0 % Hb] * 1.4426950408889634f, s1 = a.sink[h0 + r1 % Hb] * 1.4426950408889634f;
+        const float n0 = fmaxf(m0, s0), n1 = fmaxf(m1, s1), f0 = exp2f(m0 - n0), f1 = exp2f(m1 - n1);
+        l0 = l0 * f0 + exp2f(s0 - n0);
+        l1 = l1 * f1 + exp2f(s1 - n1);
+#pragma unroll
+        for (int j = 0; j < CW / 8; ++j) { o[j][0] *= f0; o[j][1] *= f0; o[j][2] *= f1; o[j][3] *= f1; }
+    }
     const float i0 = whole ? 1.0f / l0 : 1.f, i1 = whole ? 1.0f / l1 : 1.f;
 #pragma unroll
     for (int half = 0; half < 2; ++half) {
@@ -262,7 +271,8 @@ __global__ void __launch_bounds__(NT * NCH, 1) latent_attention_tc_kernel(Latent
 // One block per (row, head): the slices' weights once, then a thread per value column, the slices added in their order.
 template <typename TO>
 __global__ void __launch_bounds__(128) latent_merge_tc_kernel(const float* __restrict__ part_o, const float* __restrict__ part_ml,
-                                                              TO* __restrict__ out, int n_pairs, int R, int splits) {
+                                                              TO* __restrict__ out, int n_pairs, int R, int splits,
+                                                              const float* __restrict__ sink, int H) {
     pdl_launch_dependents();
     pdl_wait();
     __shared__ float wgt[64];
@@ -270,7 +280,7 @@ __global__ void __launch_bounds__(128) latent_merge_tc_kernel(const float* __res
     const int pair = blockIdx.x, tid = threadIdx.x;
     const float* ml = part_ml + (size_t)pair * splits * 2;
     if (tid < 32) {
-        float m = -CUDART_INF_F;
+        float m = sink ? sink[pair % H] : -CUDART_INF_F;
         for (int s = tid; s < splits; s += 32) m = fmaxf(m, ml[2 * s]);
         m = warp_max(m);
         float l = 0.f;
@@ -280,7 +290,7 @@ __global__ void __launch_bounds__(128) latent_merge_tc_kernel(const float* __res
             l += w * ml[2 * s + 1];
         }
         l = warp_sum(l);
-        if (tid == 0) inv_s = 1.f / l;
+        if (tid == 0) inv_s = 1.f / (sink ? l + expf(sink[pair % H] - m) : l);
     }
     __syncthreads();
     const float inv = inv_s;
@@ -307,9 +317,9 @@ int launch(LatentArgs a, int n_blocks, int T, cudaStream_t stream) {
     const int n = T * a.H;
     if (a.out_bf16)
         return launch_pdl(latent_merge_tc_kernel<__nv_bfloat16>, dim3(n), dim3(128), 0, stream, (const float*)a.part_o,
-                          (const float*)a.part_ml, reinterpret_cast<__nv_bfloat16*>(a.out), n, a.R, a.splits);
+                          (const float*)a.part_ml, reinterpret_cast<__nv_bfloat16*>(a.out), n, a.R, a.splits, a.sink, a.H);
     return launch_pdl(latent_merge_tc_kernel<float>, dim3(n), dim3(128), 0, stream, (const float*)a.part_o,
-                      (const float*)a.part_ml, a.out, n, a.R, a.splits);
+                      (const float*)a.part_ml, a.out, n, a.R, a.splits, a.sink, a.H);
 }
 
 }  // namespace
@@ -324,14 +334,14 @@ LQ_EXPORT int lq_latent_attention_tc(const float* q, const void* pages, const in
                                      const int* qb_seq, const int* qb_row, const int* qb_rows, const int* qb_pos,
                                      const int* tok_pos, const int* tok_seq, void* out, int out_dtype, float* part_o, float* part_ml,
                                      int n_blocks, int T, int H, int R, int Dk, int page_size, float scale, int window,
-                                     int splits, cudaStream_t stream) {
+                                     int splits, const float* sink, cudaStream_t stream) {
     if (n_blocks <= 0) return LQ_OK;
     if (Dk % 8 || R < 1 || R > Dk || page_size % BN || splits < 1 || (splits > 1 && (!part_o || !part_ml)) || splits > 64) return LQ_BAD_SIZE;
     if (!qb_seq && (!tok_pos || !tok_seq)) return LQ_BAD_SIZE;
     if (out_dtype != LQ_F32 && out_dtype != LQ_BF16) return LQ_BAD_DTYPE;
     LatentArgs a{q, (const __nv_bfloat16*)pages, page_table, pt_stride, slots, qb_seq, qb_row, qb_rows, qb_pos, tok_pos, tok_seq,
                  (float*)out, part_o, part_ml, H, R, Dk, page_size, window, splits, (H + BM - 1) / BM, 1, out_dtype == LQ_BF16,
-                 scale * 1.4426950408889634f};
+                 scale * 1.4426950408889634f, sink};
     if (R <= 64) return launch<64, 1>(a, n_blocks, T, stream);
     if (R <= 128) return launch<128, 1>(a, n_blocks, T, stream);
     if (R <= 256) return launch<256, 1>(a, n_blocks, T, stream);

@@ -109,13 +109,14 @@ LQ_EXPORT int lq_moe_route(const float* z, int z_stride, int* ids, float* weight
                       weights, T, E, groups, keep, top, route_scale, score_fn, correction, group_rule, normalize);
 }
 
-// act: 0 none, 1 gelu (erf), 2 gelu (tanh form), 3 silu, 4 relu
+// act: 0 none, 1 gelu (erf), 2 gelu (tanh form), 3 silu, 4 relu, 5 the square of relu
 __device__ __forceinline__ float moe_act(float v, int act) {
     switch (act) {
         case 1: return 0.5f * v * (1.f + erff(v * 0.70710678118654752f));
         case 2: return 0.5f * v * (1.f + tanhf(0.7978845608028654f * (v + 0.044715f * v * v * v)));
         case 3: return v / (1.f + expf(-v));
         case 4: return fmaxf(v, 0.f);
+        case 5: { const float r = fmaxf(v, 0.f); return r * r; }
         default: return v;
     }
 }
@@ -244,7 +245,7 @@ __global__ void __launch_bounds__(MX_WARPS * 32) moe_down_kernel(const T* __rest
 LQ_EXPORT int lq_moe_up_rows(const void* h, const void* w_up, const int* ids, void* u, int dtype, int T, int top, int D, int F, int act,
                              int gated, int n_real, int block, cudaStream_t stream) {
     if (T <= 0) return LQ_OK;
-    if (act < 0 || act > 4 || (size_t)D * 4 > 200 * 1024) return LQ_BAD_SIZE;
+    if (act < 0 || act > 5 || (size_t)D * 4 > 200 * 1024) return LQ_BAD_SIZE;
     if (block < 0 || (block && (!gated || F % block))) return LQ_BAD_SIZE;
     dim3 grid(T * top, (F + MX_WARPS * MX_PER_WARP - 1) / (MX_WARPS * MX_PER_WARP));
     const size_t smem = (size_t)D * sizeof(float);

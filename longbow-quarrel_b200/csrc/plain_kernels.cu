@@ -20,23 +20,24 @@
 // ------------------------------------------------------------------ embedding
 template <typename TW>
 __global__ void embedding_kernel(const TW* __restrict__ table, const int* __restrict__ tokens,
-                                 float* __restrict__ out, int D, int V) {
+                                 float* __restrict__ out, int D, int V, float scale) {
     pdl_launch_dependents();
     pdl_wait();
     int t = blockIdx.x;
     int tok = tokens[t];
     if (tok < 0 || tok >= V) tok = 0;  // range is checked on the host before launch
     const TW* row = table + (size_t)tok * D;
-    for (int i = threadIdx.x; i < D; i += blockDim.x) out[(size_t)t * D + i] = to_f32(row[i]);
+    for (int i = threadIdx.x; i < D; i += blockDim.x) out[(size_t)t * D + i] = to_f32(row[i]) * scale;
 }
 
+// out[t] = table[tok_t] * scale
 LQ_EXPORT int lq_embedding(const void* table, int table_dtype, const int* tokens, float* out,
-                           int T, int D, int V, cudaStream_t stream) {
+                           int T, int D, int V, float scale, cudaStream_t stream) {
     if (T <= 0) return LQ_OK;
     if (table_dtype == LQ_F32)
-        return launch_pdl(embedding_kernel<float>, dim3(T), dim3(256), 0, stream, (const float*)table, tokens, out, D, V);
+        return launch_pdl(embedding_kernel<float>, dim3(T), dim3(256), 0, stream, (const float*)table, tokens, out, D, V, scale);
     else if (table_dtype == LQ_BF16)
-        return launch_pdl(embedding_kernel<__nv_bfloat16>, dim3(T), dim3(256), 0, stream, (const __nv_bfloat16*)table, tokens, out, D, V);
+        return launch_pdl(embedding_kernel<__nv_bfloat16>, dim3(T), dim3(256), 0, stream, (const __nv_bfloat16*)table, tokens, out, D, V, scale);
     else
         return LQ_BAD_DTYPE;
     return lq_launch_status();
@@ -1328,6 +1329,7 @@ LQ_EXPORT int lq_softcap(float* x, long long total, float cap, cudaStream_t stre
 // The same kernel serves a prompt's tokens and a decoded token, so both reduce in the
 // same order.  cap > 0: score <- cap * tanh(score / cap) after the scale.  keep_first: with a window, the first
 // keep_first positions of the sequence stay visible (at their own positions) when the window has moved past them.
+// slope (or null): [H], score <- score - slope[h] * (position - key), after the cap.
 constexpr int ATT_CHUNK = 128;
 
 template <typename T, typename TG>
@@ -1337,7 +1339,8 @@ attention_plain_kernel(const T* __restrict__ q, int q_stride, const T* __restric
                        const int* __restrict__ tok_pos, const int* __restrict__ tok_seq,
                        const int* __restrict__ slots, T* __restrict__ out, int H, int Hkv, int hd,
                        int page_size, float scale, int window, int vd, const float* __restrict__ sink,
-                       const TG* __restrict__ gate, int gate_stride, float cap, int keep_first, int gate_per_head) {
+                       const TG* __restrict__ gate, int gate_stride, float cap, int keep_first, int gate_per_head,
+                       const float* __restrict__ slope) {
     pdl_launch_dependents();
     pdl_wait();
     extern __shared__ float sm[];
@@ -1369,6 +1372,7 @@ attention_plain_kernel(const T* __restrict__ q, int q_stride, const T* __restric
             for (int i = 0; i < hd; ++i) d = fmaf(qs[i], to_f32(kr[i]), d);
             s = d * scale;
             if (cap > 0.f) s = cap * tanhf(s / cap);
+            if (slope) s = fmaf(-slope[h], (float)(pos - key), s);
         }
         sc[tid] = s;
         __syncthreads();
@@ -1425,7 +1429,7 @@ LQ_EXPORT int lq_attention_plain(const void* q, int q_stride, int dtype, const v
                                  const int* page_table, int pt_stride, const int* tok_pos, const int* tok_seq,
                                  const int* slots, void* out, int T, int H, int Hkv, int hd, int page_size,
                                  float scale, int window, int vd, const float* sink, const void* gate, int gate_stride,
-                                 int gate_dtype, float cap, int keep_first, int gate_per_head, cudaStream_t stream) {
+                                 int gate_dtype, float cap, int keep_first, int gate_per_head, const float* slope, cudaStream_t stream) {
     if (T <= 0) return LQ_OK;
     if (vd <= 0) vd = hd;
     if (vd > 2 * ATT_CHUNK || H % Hkv) return LQ_BAD_SIZE;
@@ -1434,15 +1438,15 @@ LQ_EXPORT int lq_attention_plain(const void* q, int q_stride, int dtype, const v
     if (dtype == LQ_F32)
         return launch_pdl(attention_plain_kernel<float, float>, grid, dim3(ATT_CHUNK), smem, stream, (const float*)q, q_stride, (const float*)k_pages,
             (const float*)v_pages, page_table, pt_stride, tok_pos, tok_seq, slots, (float*)out, H, Hkv, hd, page_size, scale, window,
-            vd, sink, (const float*)gate, gate_stride, cap, keep_first, gate_per_head);
+            vd, sink, (const float*)gate, gate_stride, cap, keep_first, gate_per_head, slope);
     else if (dtype == LQ_BF16 && gate && gate_dtype == LQ_F32)
         return launch_pdl(attention_plain_kernel<__nv_bfloat16, float>, grid, dim3(ATT_CHUNK), smem, stream, (const __nv_bfloat16*)q, q_stride,
             (const __nv_bfloat16*)k_pages, (const __nv_bfloat16*)v_pages, page_table, pt_stride, tok_pos, tok_seq, slots,
-            (__nv_bfloat16*)out, H, Hkv, hd, page_size, scale, window, vd, sink, (const float*)gate, gate_stride, cap, keep_first, gate_per_head);
+            (__nv_bfloat16*)out, H, Hkv, hd, page_size, scale, window, vd, sink, (const float*)gate, gate_stride, cap, keep_first, gate_per_head, slope);
     else if (dtype == LQ_BF16)
         return launch_pdl(attention_plain_kernel<__nv_bfloat16, __nv_bfloat16>, grid, dim3(ATT_CHUNK), smem, stream, (const __nv_bfloat16*)q, q_stride,
             (const __nv_bfloat16*)k_pages, (const __nv_bfloat16*)v_pages, page_table, pt_stride, tok_pos, tok_seq, slots,
-            (__nv_bfloat16*)out, H, Hkv, hd, page_size, scale, window, vd, sink, (const __nv_bfloat16*)gate, gate_stride, cap, keep_first, gate_per_head);
+            (__nv_bfloat16*)out, H, Hkv, hd, page_size, scale, window, vd, sink, (const __nv_bfloat16*)gate, gate_stride, cap, keep_first, gate_per_head, slope);
     else
         return LQ_BAD_DTYPE;
     return lq_launch_status();

@@ -4,7 +4,11 @@
 //   join    x += y / rms(y) * w,  y a branch, or the sum of two branches that are normed first:
 //           y = m1 (y1 + b1) / rms(y1 + b1) * w1 + m2 (y2 + b2) / rms(y2 + b2) * w2
 //
-// with rms(v) = sqrt(mean(v^2) + eps).  Either kernel also leaves what the next sublayer reads: the new stream in the
+// with rms(v) = sqrt(mean(v^2) + eps), and, for layers that norm a branch on both sides with norms of any kind,
+//
+//   join_branch   x += m norm_1(y) (+ e);  h = norm_2(x),   norm(v) = (v - c mean(v)) / sqrt(mean((v - c mean(v))^2) + eps) * w + b
+//
+// with c 1 for a layer norm and 0 for an RMS norm.  Every kernel also leaves what the next sublayer reads: the new stream in the
 // activations' dtype, or normed once more where the next layer has a norm of its own.  A block per row, the row held in
 // registers, everything in float32, sums in an order that the row's length alone fixes.
 #include "common.cuh"
@@ -205,6 +209,100 @@ __global__ void __launch_bounds__(MAX_THREADS) join_kernel(JoinArgs a) {
     }
 }
 
+struct AnyNorm {
+    const float *w, *b;              // b or null
+    float eps;
+    int center;
+};
+struct JoinBranchArgs {
+    const float* y;
+    AnyNorm n1;
+    float m;
+    const float* extra;              // joins the stream as well (or null)
+    float* x;
+    void* h;                         // the rows of the norm that reads the stream next, or null
+    AnyNorm n2;
+    int D;
+};
+
+// v <- norm(v) without weight and bias; returns the factor, the mean is taken off in place.
+template <int NV, int VW>
+__device__ __forceinline__ float norm_factor(Piece<VW> (&v)[NV], int D, const AnyNorm& n, float* red, int& turn) {
+    float s[1] = {0.f};
+    if (n.center) {
+#pragma unroll
+        for (int i = 0; i < NV; ++i)
+            if ((threadIdx.x + i * blockDim.x) * VW < D)
+#pragma unroll
+                for (int c = 0; c < VW; ++c) s[0] += v[i].v[c];
+        block_sums(s, red, turn);
+        const float mean = s[0] / (float)D;
+#pragma unroll
+        for (int i = 0; i < NV; ++i)
+#pragma unroll
+            for (int c = 0; c < VW; ++c) v[i].v[c] -= mean;
+    }
+    s[0] = 0.f;
+#pragma unroll
+    for (int i = 0; i < NV; ++i)
+        if ((threadIdx.x + i * blockDim.x) * VW < D)
+#pragma unroll
+            for (int c = 0; c < VW; ++c) s[0] = fmaf(v[i].v[c], v[i].v[c], s[0]);
+    block_sums(s, red, turn);
+    return 1.f / sqrtf(s[0] / (float)D + n.eps);
+}
+
+template <typename TO, int NV, int VW>
+__global__ void __launch_bounds__(MAX_THREADS) join_branch_kernel(const __grid_constant__ JoinBranchArgs a) {
+    __shared__ float red[2 * 32];
+    pdl_launch_dependents();
+    pdl_wait();
+    const int D = a.D;
+    const size_t at = (size_t)blockIdx.x * D;
+    int turn = 0;
+    Piece<VW> y[NV], x[NV];
+#pragma unroll
+    for (int i = 0; i < NV; ++i) {
+        const int d = (threadIdx.x + i * blockDim.x) * VW;
+        if (d < D) {
+            y[i] = load_piece<VW>(a.y + at + d);
+            x[i] = load_piece<VW>(a.x + at + d);
+        }
+    }
+    const float k = norm_factor<NV, VW>(y, D, a.n1, red, turn);
+#pragma unroll
+    for (int i = 0; i < NV; ++i) {
+        const int d = (threadIdx.x + i * blockDim.x) * VW;
+        if (d < D) {
+            const Piece<VW> w = load_piece<VW>(a.n1.w + d);
+            Piece<VW> b{};
+            if (a.n1.b) b = load_piece<VW>(a.n1.b + d);
+#pragma unroll
+            for (int c = 0; c < VW; ++c) x[i].v[c] = fmaf(a.m, fmaf(y[i].v[c] * k, w.v[c], b.v[c]), x[i].v[c]);
+            if (a.extra) {
+                const Piece<VW> e = load_piece<VW>(a.extra + at + d);
+#pragma unroll
+                for (int c = 0; c < VW; ++c) x[i].v[c] += e.v[c];
+            }
+            store_piece(a.x + at + d, x[i]);
+        }
+    }
+    if (!a.h) return;
+    const float kn = norm_factor<NV, VW>(x, D, a.n2, red, turn);
+#pragma unroll
+    for (int i = 0; i < NV; ++i) {
+        const int d = (threadIdx.x + i * blockDim.x) * VW;
+        if (d < D) {
+            const Piece<VW> w = load_piece<VW>(a.n2.w + d);
+            Piece<VW> b{};
+            if (a.n2.b) b = load_piece<VW>(a.n2.b + d);
+#pragma unroll
+            for (int c = 0; c < VW; ++c) x[i].v[c] = fmaf(x[i].v[c] * kn, w.v[c], b.v[c]);
+            store_piece((TO*)a.h + at + d, x[i]);
+        }
+    }
+}
+
 // Pieces a thread holds and threads of a block for rows of n pieces; 0 where the row is too long.
 int shape_of(int n, int& threads) {
     threads = n < 256 ? (n + 31) / 32 * 32 : (n <= 1024 ? 256 : (n <= 2048 ? 512 : MAX_THREADS));
@@ -218,6 +316,21 @@ int join_launch(const JoinArgs& a, int T, cudaStream_t stream) {
     const int nv = shape_of(a.D / VW, threads);
 #define LQ_GO(NV) (a.y2 ? launch_pdl(join_kernel<TO, NV, VW, true>, dim3(T), dim3(threads), 0, stream, a) \
                         : launch_pdl(join_kernel<TO, NV, VW, false>, dim3(T), dim3(threads), 0, stream, a))
+    switch (nv) {
+        case 1: return LQ_GO(1);
+        case 2: return LQ_GO(2);
+        case 4: return LQ_GO(4);
+        case 8: return LQ_GO(8);
+    }
+#undef LQ_GO
+    return LQ_BAD_SIZE;
+}
+
+template <typename TO, int VW>
+int join_branch_launch(const JoinBranchArgs& a, int T, cudaStream_t stream) {
+    int threads = 0;
+    const int nv = shape_of(a.D / VW, threads);
+#define LQ_GO(NV) launch_pdl(join_branch_kernel<TO, NV, VW>, dim3(T), dim3(threads), 0, stream, a)
     switch (nv) {
         case 1: return LQ_GO(1);
         case 2: return LQ_GO(2);
@@ -274,6 +387,22 @@ LQ_EXPORT int lq_join_normed(const float* y1, const float* b1, const float* w1, 
     typedef __nv_bfloat16 bf;
     if (h_dtype == LQ_F32) return vec ? join_launch<float, 4>(a, T, stream) : join_launch<float, 1>(a, T, stream);
     return vec ? join_launch<bf, 4>(a, T, stream) : join_launch<bf, 1>(a, T, stream);
+}
+
+// x += m norm(y; w1, b1, eps1) (+ extra), in place (float32 [T, D]); with h the rows of the norm (w2, b2, eps2) of the new
+// stream in h_dtype.  center1, center2: the mean is taken off first (layer norms).  Biases and extra may be null.
+LQ_EXPORT int lq_join_branch(const float* y, const float* w1, const float* b1, float eps1, int center1, float m, const float* extra, float* x,
+                             void* h, int h_dtype, const float* w2, const float* b2, float eps2, int center2, int T, int D,
+                             cudaStream_t stream) {
+    if (T <= 0) return LQ_OK;
+    if (h_dtype != LQ_F32 && h_dtype != LQ_BF16) return LQ_BAD_DTYPE;
+    if (!w1 || (h && !w2)) return LQ_BAD_SIZE;
+    JoinBranchArgs a{y, {w1, b1, eps1, center1}, m, extra, x, h, {w2, b2, eps2, center2}, D};
+    const uintptr_t all = (uintptr_t)y | (uintptr_t)w1 | (uintptr_t)b1 | (uintptr_t)extra | (uintptr_t)x | (uintptr_t)h | (uintptr_t)w2 | (uintptr_t)b2;
+    const bool vec = D % 4 == 0 && (all & 15) == 0;
+    typedef __nv_bfloat16 bf;
+    if (h_dtype == LQ_F32) return vec ? join_branch_launch<float, 4>(a, T, stream) : join_branch_launch<float, 1>(a, T, stream);
+    return vec ? join_branch_launch<bf, 4>(a, T, stream) : join_branch_launch<bf, 1>(a, T, stream);
 }
 
 // ------------------------------------------------------------------ columns of a product's rows as another product's input

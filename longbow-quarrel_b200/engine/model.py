@@ -138,8 +138,11 @@ class Model:
             probe(-1, x, ctx)
         # A block that reads the embedding's rows again later (`reads_embedding`) gets a copy: the stream changes in place.
         embedded = x.clone() if self._keeps_embedding else None
+        added = -1              # a run that only adds the embedding's rows and that the layer ahead has made already
         for i, entry in enumerate(schedule):
             block = self.blocks[entry.layer]
+            if i == added:
+                continue
             if getattr(block, "replaces_stream", False):
                 # A block that makes a new stream out of the old one (and the embedding's rows); it is no layer, and
                 # the probe is not called for it.
@@ -159,9 +162,17 @@ class Model:
                 if probe is not None:
                     probe(i, x, ctx)
                 continue
-            after = self.blocks[schedule[i + 1].layer] if i + 1 < len(schedule) else None
+            following = [self.blocks[e.layer] for e in schedule[i + 1:i + 3]]
+            more = {}
+            if following and probe is None and getattr(block, "takes_extra", False) and getattr(following[0], "adds_embedding", False):
+                more["extra"], added = embedded, i + 1
+                following.pop(0)
+            after = following[0] if following else None
             emit = after.input_norm(x.shape[0]) if getattr(after, "folds_norm", False) else None
-            more = {"emit_stream": True} if getattr(block, "emits_stream", False) and getattr(after, "reads_stream", False) else {}
+            if getattr(block, "emits_stream", False) and getattr(after, "reads_stream", False):
+                more["emit_stream"] = True
+            if getattr(block, "emits_any_norm", False) and hasattr(after, "first_norm"):
+                more["emit_norm"] = after.first_norm()
             normed = block.forward(x, ctx, cache.view(entry.cache), entry.writes_cache, normed=normed, emit=emit, **more)
             if probe is not None:
                 probe(i, x, ctx)

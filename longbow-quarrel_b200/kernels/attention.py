@@ -160,28 +160,29 @@ def _blocks(ctx, name):
 
 
 def attention(qkv, cache_view, ctx, H, Hkv, hd, scale, window, next_w=None, vd=None, sink=None, gate=None, softcap=None,
-              keep_first=0, chunk=None, gate_per_head=False):
+              keep_first=0, chunk=None, gate_per_head=False, slope=None):
     """Rows of qkv hold q in their left H*hd columns.  Returns [T, H*vd].  next_w: the weights the
     stream reads after the attention (the decode kernel asks for their first bytes as it ends).
     vd: size of a value head (default hd); sink: float32 [H], one more term of each head's softmax
     denominator; gate: [T, H*vd] whose sigmoid multiplies the output; softcap c: score <- c tanh(score / c);
     keep_first n: with a window, a sequence's first n positions stay visible.  chunk n (instead of a window): a position
-    sees only its own block of n positions.  gate_per_head: the gate is [T, H], one number for a head's values."""
+    sees only its own block of n positions.  gate_per_head: the gate is [T, H], one number for a head's values.
+    slope: float32 [H], a score loses slope[h] times the distance to its key (after the scale and the cap)."""
     vd = vd or hd
     keep_first = int(keep_first or 0) if window else 0
-    out = _attention(qkv, cache_view, ctx, H, Hkv, hd, scale, window, next_w, sink, gate, softcap, keep_first, chunk, vd)
+    out = _attention(qkv, cache_view, ctx, H, Hkv, hd, scale, window, next_w, sink, gate, softcap, keep_first, chunk, vd, slope)
     if gate is not None and out is not None:
         # The tensor-core kernels leave the gate to a kernel of its own.
         return ops.gate_mul(out, gate, "sigmoid", group=vd if gate_per_head else 1)
     return out if out is not None else general_attention(qkv, cache_view, ctx, H, Hkv, hd, vd, scale, window, sink, gate,
-                                                         softcap, keep_first, chunk, gate_per_head)
+                                                         softcap, keep_first, chunk, gate_per_head, slope)
 
 
-def _attention(qkv, cache_view, ctx, H, Hkv, hd, scale, window, next_w, sink, gate, softcap, keep_first, chunk, vd):
+def _attention(qkv, cache_view, ctx, H, Hkv, hd, scale, window, next_w, sink, gate, softcap, keep_first, chunk, vd, slope):
     """The tensor-core kernels where they take the sizes; None where only the plain kernel does and a gate
     is to be applied or values have a size of their own (the plain kernel does both itself)."""
     aligned = qkv.stride(0) % 8 == 0 and qkv.data_ptr() % 16 == 0
-    more = dict(sink=sink, softcap=softcap, keep_first=keep_first)
+    more = dict(sink=sink, softcap=softcap, keep_first=keep_first, slope=slope)
     mask = ops.span(window, chunk)          # the kernels take a window as w and blocks of n positions as -n
     if not ctx.decode and aligned:
         kind = prefill_kernel(qkv.dtype, hd, cache_view.page_size, vd)
@@ -213,14 +214,14 @@ def _attention(qkv, cache_view, ctx, H, Hkv, hd, scale, window, next_w, sink, ga
         return None
     return ops.attention_plain(qkv, cache_view.k_pages, cache_view.v_pages, cache_view.page_table, ctx.tok_pos,
                                ctx.tok_seq, ctx.slots, H, Hkv, hd, cache_view.page_size, scale, window, sink=sink,
-                               softcap=softcap, keep_first=keep_first, chunk=chunk)
+                               softcap=softcap, keep_first=keep_first, chunk=chunk, slope=slope)
 
 
 def general_attention(qkv, cache_view, ctx, H, Hkv, hd, vd, scale, window, sink, gate, softcap=None, keep_first=0, chunk=None,
-                      gate_per_head=False):
+                      gate_per_head=False, slope=None):
     """Attention through the plain kernel, which takes every option: a sink, a gate (per value or per head), values of
     another size than the keys, capped scores, kept first positions, blocks of positions."""
     return ops.attention_plain(qkv, cache_view.k_pages, cache_view.v_pages, cache_view.page_table, ctx.tok_pos,
                                ctx.tok_seq, ctx.slots, H, Hkv, hd, cache_view.page_size, scale, window, vd=vd,
                                sink=sink, gate=gate, softcap=softcap, keep_first=keep_first, chunk=chunk,
-                               gate_per_head=gate_per_head)
+                               gate_per_head=gate_per_head, slope=slope)

@@ -90,7 +90,8 @@ _WATCHED = {"gemm_tc": {1: "the TMA producer waited for a free stage", 2: "the p
                         3: "the product issuer waited for a stage's copies", 4: "the epilogue waited for an accumulator"},
             "gemm_pair": {1: "a TMA producer waited for a free stage", 2: "the product issuer waited for a free accumulator",
                           3: "the product issuer waited for a stage's copies", 4: "an epilogue waited for an accumulator"},
-            "attn_prefill_tc": {}, "delta": {1: "the copying warp waited for a free stage", 2: "a warp waited for a record"}}
+            "attn_prefill_tc": {}, "delta": {1: "the copying warp waited for a free stage", 2: "a warp waited for a record"},
+            "head_delta": {1: "the copying warp waited for a free stage", 2: "a warp waited for a chunk"}}
 _status_words: dict[str, object] = {}
 
 
@@ -150,14 +151,14 @@ def prepare(dtype: torch.dtype, verbose: bool = True, extra: tuple = ()) -> None
 
 # ------------------------------------------------------------------ plain kernels
 
-def embedding(table: torch.Tensor, tokens: torch.Tensor, out: torch.Tensor | None = None) -> torch.Tensor:
-    """out[t] = table[tokens[t]] as float32 (the residual stream starts in 32-bit)."""
+def embedding(table: torch.Tensor, tokens: torch.Tensor, out: torch.Tensor | None = None, scale: float = 1.0) -> torch.Tensor:
+    """out[t] = table[tokens[t]] * scale as float32 (the residual stream starts in 32-bit)."""
     V, D = table.shape
     T = tokens.numel()
     if out is None:
         out = torch.empty((T, D), dtype=torch.float32, device=table.device)
-    fn = _fn("plain_kernels", "lq_embedding", [c_void_p, c_int, c_void_p, c_void_p, c_int, c_int, c_int, c_void_p])
-    _check(fn(_p(_contig(table, "table")), dtype_code(table), _p(tokens), _p(out), T, D, V, _stream()), "embedding")
+    fn = _fn("plain_kernels", "lq_embedding", [c_void_p, c_int, c_void_p, c_void_p, c_int, c_int, c_int, c_float, c_void_p])
+    _check(fn(_p(_contig(table, "table")), dtype_code(table), _p(tokens), _p(out), T, D, V, float(scale), _stream()), "embedding")
     return out
 
 
@@ -334,15 +335,17 @@ def attention_plain(q: torch.Tensor, k_pages, v_pages, page_table, tok_pos, tok_
                     hd: int, page_size: int, scale: float, window: int | None,
                     out: torch.Tensor | None = None, vd: int | None = None, sink: torch.Tensor | None = None,
                     gate: torch.Tensor | None = None, softcap: float | None = None, keep_first: int = 0,
-                    chunk: int | None = None, gate_per_head: bool = False) -> torch.Tensor:
+                    chunk: int | None = None, gate_per_head: bool = False, slope: torch.Tensor | None = None) -> torch.Tensor:
     """Causal attention of every token over its own sequence's cache; q is the left
     H*hd columns of a [T, q_stride] buffer.  softcap c: score <- c tanh(score / c) after the scale.  keep_first: with a
     window, the sequence's first keep_first positions stay visible when the window has moved past them.  vd: size of a value head (default hd).  sink: float32 [H], one
     more term exp(sink) in each head's softmax denominator.  gate: a [T, H*vd] view (rows may be strided) whose
     sigmoid multiplies the output; with gate_per_head a [T, H] view, one number for all values of a head.
-    chunk n (instead of a window): a position sees only its own block of n positions."""
+    chunk n (instead of a window): a position sees only its own block of n positions.  slope: float32 [H], a score loses
+    slope[h] times the distance to its key, after the scale and the cap."""
     T = q.shape[0]
     vd = vd or hd
+    _check_slope(slope, H)
     if hd > 256 or vd > 256:
         raise KernelError(f"attention: head sizes {hd}, {vd} exceed 256")
     if sink is not None and (sink.dtype != torch.float32 or sink.numel() != H):
@@ -355,13 +358,18 @@ def attention_plain(q: torch.Tensor, k_pages, v_pages, page_table, tok_pos, tok_
     fn = _fn("plain_kernels", "lq_attention_plain", [c_void_p, c_int, c_int, c_void_p, c_void_p, c_void_p, c_int,
                                                      c_void_p, c_void_p, c_void_p, c_void_p, c_int, c_int, c_int, c_int,
                                                      c_int, c_float, c_int, c_int, c_void_p, c_void_p, c_int, c_int, c_float, c_int,
-                                                     c_int, c_void_p])
+                                                     c_int, c_void_p, c_void_p])
     _check(fn(_p(q), q.stride(0), dtype_code(q), _p(k_pages), _p(v_pages), _p(page_table), page_table.stride(0),
               _p(tok_pos), _p(tok_seq), _p(slots), _p(out), T, H, Hkv, hd, page_size, float(scale),
               span(window, chunk), vd, _p(sink), _p(gate), gate.stride(0) if gate is not None else 0,
               dtype_code(gate) if gate is not None else F32, float(softcap or 0.0), int(keep_first or 0),
-              int(bool(gate_per_head and gate is not None)), _stream()), "attention")
+              int(bool(gate_per_head and gate is not None)), _p(slope), _stream()), "attention")
     return out
+
+
+def _check_slope(slope, H: int) -> None:
+    if slope is not None and (slope.dtype != torch.float32 or slope.numel() != H or not slope.is_contiguous()):
+        raise KernelError("attention: the distance slopes must be contiguous float32 [H]")
 
 
 def span(window: int | None, chunk: int | None = None) -> int:
@@ -480,6 +488,30 @@ def join_normed(x: torch.Tensor, branches: tuple, gain: torch.Tensor, eps: float
               dtype_code(h) if own else F32, _p(next_gain), float(next_eps), T, D, _stream()), "join_normed", 1,
            "join_normed:two" if not one else None)
     return h if own else (x if rows_dtype is not None else None)
+
+
+def join_branch(x: torch.Tensor, y: torch.Tensor, norm: tuple, m: float, extra: torch.Tensor | None = None, next_norm: tuple | None = None,
+                rows_dtype: torch.dtype | None = None) -> torch.Tensor | None:
+    """x += m * norm(y) (+ extra), row by row, in place (float32 [T, D]): a branch joins the stream after a norm of its own and with
+    a multiplier.  next_norm: the norm that reads the stream next; its rows are made by the same kernel and returned in
+    rows_dtype.  A norm is (gain, bias or None, eps, center), as `Norm.affine` gives it: center takes the mean off (layer norm)."""
+    T, D = x.shape
+    for t in (y, extra):
+        if t is not None and (t.dtype != torch.float32 or t.shape != x.shape or not t.is_contiguous()):
+            raise KernelError("join_branch: a branch must be contiguous float32 of the stream's shape")
+    if x.dtype != torch.float32 or not x.is_contiguous():
+        raise KernelError("join_branch: the stream must be contiguous float32")
+    w1, b1, eps1, center1 = norm
+    w2, b2, eps2, center2 = next_norm if next_norm is not None else (None, None, 0.0, False)
+    for v in (w1, b1, w2, b2):
+        if v is not None and (v.dtype != torch.float32 or v.numel() != D or not v.is_contiguous()):
+            raise KernelError("join_branch: gains and biases must be contiguous float32 [D]")
+    h = torch.empty((T, D), dtype=rows_dtype, device=x.device) if next_norm is not None else None
+    fn = _fn("post_norm", "lq_join_branch", [c_void_p, c_void_p, c_void_p, c_float, c_int, c_float, c_void_p, c_void_p, c_void_p, c_int,
+                                             c_void_p, c_void_p, c_float, c_int, c_int, c_int, c_void_p])
+    _check(fn(_p(y), _p(w1), _p(b1), float(eps1), int(center1), float(m), _p(extra), _p(x), _p(h), dtype_code(h) if h is not None else F32,
+              _p(w2), _p(b2), float(eps2), int(center2), T, D, _stream()), "join_branch", 1, "join_branch:extra" if extra is not None else None)
+    return h
 
 
 def rope_partial(buf: torch.Tensor, bias: torch.Tensor | None, cos, sin, rot: int, tok_pos, tok_seq, slots,
@@ -641,10 +673,12 @@ def head_matmul(src: torch.Tensor, src_head: int, src_off: int, w: torch.Tensor,
 
 
 def latent_attention(q: torch.Tensor, pages: torch.Tensor, page_table, tok_pos, tok_seq, slots, H: int, R: int, page_size: int,
-                     scale: float, window: int | None, splits: int = 1) -> torch.Tensor:
+                     scale: float, window: int | None, splits: int = 1, sink: torch.Tensor | None = None) -> torch.Tensor:
     """Causal attention of every row's H wide queries q [T, H, Dk] (float32) over the latent rows of its sequence's cache
     (pages [pages, page_size, Dk]): scores over all Dk numbers, values the rows' first R numbers.  Returns float32
-    [T, H, R].  splits: slices that each row's keys are cut into (merged by a second kernel)."""
+    [T, H, R].  splits: slices that each row's keys are cut into (merged by a second kernel).  sink: float32 [H], one more
+    term exp(sink) in each head's denominator, with no key and no value."""
+    _check_sink(sink, H)
     T, Hq, Dk = q.shape
     if q.dtype != torch.float32 or not q.is_contiguous() or Hq != H or pages.shape[-1] != Dk or not pages.is_contiguous():
         raise KernelError("latent_attention: contiguous float32 queries [T, H, Dk] and cache rows of Dk numbers")
@@ -657,9 +691,9 @@ def latent_attention(q: torch.Tensor, pages: torch.Tensor, page_table, tok_pos, 
         part_ml = torch.empty((T, H, splits, 2), dtype=torch.float32, device=q.device)
     fn = _fn("latent_attn", "lq_latent_attention", [c_void_p, c_void_p, c_int, c_void_p, c_int, c_void_p, c_void_p, c_void_p,
                                                     c_void_p, c_void_p, c_void_p, c_int, c_int, c_int, c_int, c_int, c_float,
-                                                    c_int, c_int, c_void_p])
+                                                    c_int, c_int, c_void_p, c_void_p])
     _check(fn(_p(q), _p(pages), dtype_code(pages), _p(page_table), page_table.stride(0), _p(tok_pos), _p(tok_seq), _p(slots),
-              _p(out), _p(part_o), _p(part_ml), T, H, R, Dk, page_size, float(scale), int(window or 0), int(splits), _stream()),
+              _p(out), _p(part_o), _p(part_ml), T, H, R, Dk, page_size, float(scale), int(window or 0), int(splits), _p(sink), _stream()),
            "latent_attention", 2 if splits > 1 else 1, "latent_attention:slices" if splits > 1 else None)
     return out
 
@@ -676,11 +710,12 @@ def latent_attention_tc_takes(pages: torch.Tensor, page_size: int) -> bool:
 
 def latent_attention_tc(q: torch.Tensor, pages: torch.Tensor, page_table, slots, H: int, R: int, page_size: int, scale: float,
                         window: int | None, blocks: tuple | None = None, tok_pos=None, tok_seq=None, splits: int = 1,
-                        out_dtype: torch.dtype = torch.float32) -> torch.Tensor:
+                        out_dtype: torch.dtype = torch.float32, sink: torch.Tensor | None = None) -> torch.Tensor:
     """latent_attention on the tensor cores (mma.sync, bfloat16 cache rows).  blocks = (sequence, first row, tokens, first
     position) int32 tensors, one entry per block of at most latent_tc_tokens(H) consecutive tokens of one sequence, for
     a step with prompts; without it every row is its own block (tok_pos, tok_seq) and its keys may be cut into `splits`.
     Returns [T, H, R] in out_dtype (float32 or bfloat16)."""
+    _check_sink(sink, H)
     T, Hq, Dk = q.shape
     if q.dtype != torch.float32 or not q.is_contiguous() or Hq != H or pages.shape[-1] != Dk or not pages.is_contiguous():
         raise KernelError("latent_attention_tc: contiguous float32 queries [T, H, Dk] and cache rows of Dk numbers")
@@ -695,10 +730,10 @@ def latent_attention_tc(q: torch.Tensor, pages: torch.Tensor, page_table, slots,
         part_ml = torch.empty((T, H, splits, 2), dtype=torch.float32, device=q.device)
     qb = blocks if blocks is not None else (None, None, None, None)
     fn = _fn("latent_attn_tc", "lq_latent_attention_tc", [c_void_p, c_void_p, c_void_p, c_int] + [c_void_p] * 8 + [c_int, c_void_p, c_void_p]
-             + [c_int] * 6 + [c_float, c_int, c_int, c_void_p])
+             + [c_int] * 6 + [c_float, c_int, c_int, c_void_p, c_void_p])
     _check(fn(_p(q), _p(pages), _p(page_table), page_table.stride(0), _p(slots), _p(qb[0]), _p(qb[1]), _p(qb[2]), _p(qb[3]),
               _p(tok_pos), _p(tok_seq), _p(out), dtype_code(out), _p(part_o), _p(part_ml), qb[0].numel() if blocks is not None else T, T, H, R, Dk,
-              page_size, float(scale), int(window or 0), int(splits), _stream()),
+              page_size, float(scale), int(window or 0), int(splits), _p(sink), _stream()),
            "latent_attention_tc", 2 if splits > 1 else 1, "latent_attention_tc:slices" if splits > 1 else None)
     return out
 
@@ -815,7 +850,7 @@ def moe_combine(y: torch.Tensor, weights: torch.Tensor, x: torch.Tensor, accumul
 
 
 # ------------------------------------------------------------------ routed feed-forward
-MOE_ACTS = {None: 0, "gelu": 1, "gelu_tanh": 2, "silu": 3, "relu": 4}
+MOE_ACTS = {None: 0, "gelu": 1, "gelu_tanh": 2, "silu": 3, "relu": 4, "relu2": 5}
 
 
 SCORE_FNS = {"sigmoid": 0, "softmax": 1}
@@ -1072,6 +1107,59 @@ def delta_single(rows: torch.Tensor, b_off: int, taps_w: torch.Tensor, ring: tor
     _check(fn(_p(rows), rows.stride(0), b_off, _p(taps_w), taps, _p(ring), _p(z_bias), _p(rate), _p(state), _p(cu_rows), _p(slots),
               _p(tok_pos), a_off, ra, _p(a2), a2.shape[1], g_off, rg, _p(g2), g2.shape[1], dtype_code(a2), _p(norm_w), float(norm_eps),
               _p(out), dtype_code(out_dtype), B, H, G, dk, dv, float(q_scale), float(unit_eps), _stream()), "delta_single")
+    return out
+
+
+def _head_delta_sizes(what: str, rows, b_off, a_off, g_off, taps_w, ring, dt_bias, rate, state, norm_w, H, G, dk, dv):
+    C, taps = 2 * G * dk + H * dv, taps_w.shape[0]
+    for t, shape, name in ((taps_w, (taps, C), "taps"), (dt_bias, (H,), "bias"), (rate, (H,), "rates"), (norm_w, (dv,), "norm's weight")):
+        if t.dtype != torch.float32 or tuple(t.shape) != shape or not t.is_contiguous():
+            raise KernelError(f"{what}: the {name} must be contiguous float32 {list(shape)}")
+    for t, shape, name in ((ring, (taps, C), "convolution's state"), (state, (H, dk, dv), "state")):
+        if t.dtype != torch.float32 or tuple(t.shape[1:]) != shape or not t.is_contiguous():
+            raise KernelError(f"{what}: the {name} must be contiguous float32 [slots, {', '.join(map(str, shape))}]")
+    if rows.dtype != torch.float32 or not rows.is_contiguous() or min(b_off, a_off, g_off) < C \
+            or rows.shape[1] < max(b_off + H, a_off + H, g_off + H * dv):
+        raise KernelError(f"{what}: contiguous float32 rows of q, k, v ({C} columns), step sizes, decays and gates")
+    if dk > 256 or dv > 256 or H % G:
+        raise KernelError(f"{what}: key size {dk} and value size {dv} (at most 256), {H} heads on {G} key heads")
+    return taps
+
+
+def head_delta_prompt(rows: torch.Tensor, b_off: int, a_off: int, g_off: int, taps_w: torch.Tensor, ring: torch.Tensor, dt_bias: torch.Tensor,
+                      rate: torch.Tensor, state: torch.Tensor, cu_rows, slots, tok_pos, norm_w: torch.Tensor, norm_eps: float,
+                      out_dtype: torch.dtype, B: int, max_new: int, H: int, G: int, dk: int, dv: int, q_scale: float,
+                      unit_eps: float) -> torch.Tensor:
+    """The gated delta rule with one decay per head over a step's rows (csrc/head_delta.cu), with the norm and the gate behind it:
+    rows float32 [T, ...] hold q [G dk], k [G dk], v [H dv] side by side, the step sizes' pre-activations [H] at b_off, the decays'
+    at a_off (a = exp(-rate_h softplus(. + dt_bias_h))) and the gate's [H dv] at g_off.  state [slots, H, dk, dv] and ring (see
+    delta_prompt) are moved on.  Returns each head's S^T q over its root mean square, times norm_w [dv], times silu(gate): [T, H dv]."""
+    taps = _head_delta_sizes("head_delta_prompt", rows, b_off, a_off, g_off, taps_w, ring, dt_bias, rate, state, norm_w, H, G, dk, dv)
+    T = rows.shape[0]
+    size = build.load("head_delta").lq_head_delta_scratch_floats
+    size.argtypes, size.restype = [c_int] * 6, c_longlong
+    scratch = torch.empty(int(size(T, B, H, G, dk, dv)), dtype=torch.float32, device=rows.device)
+    out = torch.empty((T, H * dv), dtype=out_dtype, device=rows.device)
+    fn = _fn("head_delta", "lq_head_delta_prompt", [c_void_p, c_int, c_int, c_int, c_int, c_void_p, c_int, c_void_p, c_void_p, c_void_p, c_void_p,
+                                                    c_void_p, c_void_p, c_void_p, c_void_p, c_void_p, c_float, c_void_p] + [c_int] * 8
+             + [c_float, c_float, c_void_p])
+    _check(fn(_p(rows), rows.stride(0), b_off, a_off, g_off, _p(taps_w), taps, _p(ring), _p(dt_bias), _p(rate), _p(state), _p(cu_rows), _p(slots),
+              _p(tok_pos), _p(scratch), _p(norm_w), float(norm_eps), _p(out), dtype_code(out), T, B, max_new, H, G, dk, dv, float(q_scale),
+              float(unit_eps), _stream()), "head_delta_prompt", 3)
+    return out
+
+
+def head_delta_single(rows: torch.Tensor, b_off: int, a_off: int, g_off: int, taps_w: torch.Tensor, ring: torch.Tensor, dt_bias: torch.Tensor,
+                      rate: torch.Tensor, state: torch.Tensor, cu_rows, slots, tok_pos, norm_w: torch.Tensor, norm_eps: float,
+                      out_dtype: torch.dtype, B: int, H: int, G: int, dk: int, dv: int, q_scale: float, unit_eps: float) -> torch.Tensor:
+    """head_delta_prompt for a step of one token per sequence: one kernel (csrc/delta.cu) that reads and writes the state once."""
+    taps = _head_delta_sizes("head_delta_single", rows, b_off, a_off, g_off, taps_w, ring, dt_bias, rate, state, norm_w, H, G, dk, dv)
+    out = torch.empty((rows.shape[0], H * dv), dtype=out_dtype, device=rows.device)
+    fn = _fn("delta", "lq_head_delta_single", [c_void_p, c_int, c_int, c_void_p, c_int, c_void_p, c_void_p, c_void_p, c_void_p, c_void_p, c_void_p,
+                                               c_void_p, c_int, c_int, c_void_p, c_float, c_void_p] + [c_int] * 6 + [c_float, c_float, c_void_p])
+    _check(fn(_p(rows), rows.stride(0), b_off, _p(taps_w), taps, _p(ring), _p(dt_bias), _p(rate), _p(state), _p(cu_rows), _p(slots), _p(tok_pos),
+              a_off, g_off, _p(norm_w), float(norm_eps), _p(out), dtype_code(out), B, H, G, dk, dv, float(q_scale), float(unit_eps),
+              _stream()), "head_delta_single")
     return out
 
 
@@ -1332,14 +1420,16 @@ def _check_sink(sink, H: int):
 def attn_prefill(q: torch.Tensor, k_pages, v_pages, page_table, slots, kv_len, query_blocks, H: int, Hkv: int, hd: int,
                  page_size: int, scale: float, window: int | None, out: torch.Tensor | None = None,
                  sink: torch.Tensor | None = None, softcap: float | None = None, keep_first: int = 0,
-                 vd: int | None = None) -> torch.Tensor:
+                 vd: int | None = None, slope: torch.Tensor | None = None) -> torch.Tensor:
     """Causal attention of blocks of query rows over the paged bfloat16 cache (flash style:
     tensor-core products, online softmax in float32).  query_blocks = (sequence, first row,
     rows, first position) int32 tensors, one entry for each block of at most 64 rows.  softcap c: score <-
     c tanh(score / c) after the scale; keep_first n (with a window): a row's first n keys stay visible.  window: as `span`
-    makes it (w positions; -n for blocks of n positions; 0 or None for all).  vd: size of a value head (default hd)."""
+    makes it (w positions; -n for blocks of n positions; 0 or None for all).  vd: size of a value head (default hd).
+    slope: float32 [H], a score loses slope[h] times the distance to its key, after the scale and the cap."""
     T = q.shape[0]
     vd = vd or hd
+    _check_slope(slope, H)
     if q.dtype != torch.bfloat16 or k_pages.dtype != torch.bfloat16:
         raise KernelError("attn_prefill takes bfloat16 queries and cache")
     if hd % 16 or hd > 128 or vd % 8 or vd > 256 or page_size != 64:
@@ -1352,11 +1442,11 @@ def attn_prefill(q: torch.Tensor, k_pages, v_pages, page_table, slots, kv_len, q
     qb_seq, qb_row, qb_rows, qb_pos = query_blocks
     fn = _fn("attn_prefill", "lq_attn_prefill_vd", [c_void_p, c_int, c_void_p, c_void_p, c_void_p, c_int, c_void_p, c_void_p,
                                                     c_void_p, c_void_p, c_void_p, c_void_p, c_void_p, c_int, c_int, c_int, c_int,
-                                                    c_int, c_int, c_float, c_int, c_void_p, c_float, c_int, c_void_p])
+                                                    c_int, c_int, c_float, c_int, c_void_p, c_float, c_int, c_void_p, c_void_p])
     _check_sink(sink, H)
     _check(fn(_p(q), q.stride(0), _p(k_pages), _p(v_pages), _p(page_table), page_table.stride(0), _p(slots), _p(kv_len),
               _p(qb_seq), _p(qb_row), _p(qb_rows), _p(qb_pos), _p(out), qb_seq.numel(), H, Hkv, hd, vd, page_size,
-              float(scale), int(window or 0), _p(sink), float(softcap or 0.0), int(keep_first if window else 0), _stream()),
+              float(scale), int(window or 0), _p(sink), float(softcap or 0.0), int(keep_first if window else 0), _p(slope), _stream()),
            "attn_prefill", 1, "attn_prefill:vd" if vd != hd else None)
     return out
 
@@ -1364,10 +1454,10 @@ def attn_prefill(q: torch.Tensor, k_pages, v_pages, page_table, slots, kv_len, q
 def attn_prefill_tc(q: torch.Tensor, k_pages, v_pages, page_table, slots, kv_len, query_blocks128, H: int, Hkv: int,
                     hd: int, page_size: int, scale: float, window: int | None,
                     out: torch.Tensor | None = None, sink: torch.Tensor | None = None, softcap: float | None = None,
-                    keep_first: int = 0) -> torch.Tensor:
+                    keep_first: int = 0, slope: torch.Tensor | None = None) -> torch.Tensor:
     """attn_prefill on the tcgen05 tensor cores (TMA-fed, S and O in tensor memory): blocks of at
-    most 128 query rows, head_dim 64 or 128, pages of 64 keys, a cache that is finite everywhere.  softcap and
-    keep_first as in attn_prefill.  window: as `span` makes it (w positions; -n for blocks of n positions; 0 or None for all)."""
+    most 128 query rows, head_dim 64 or 128, pages of 64 keys, a cache that is finite everywhere.  softcap, keep_first
+    and slope as in attn_prefill.  window: as `span` makes it (w positions; -n for blocks of n positions; 0 or None for all)."""
     T = q.shape[0]
     if q.dtype != torch.bfloat16 or k_pages.dtype != torch.bfloat16:
         raise KernelError("attn_prefill_tc takes bfloat16 queries and cache")
@@ -1378,12 +1468,13 @@ def attn_prefill_tc(q: torch.Tensor, k_pages, v_pages, page_table, slots, kv_len
     qb_seq, qb_row, qb_rows, qb_pos = query_blocks128
     fn = _fn("attn_prefill_tc", "lq_attn_prefill_tc_capped",
              [c_void_p, c_int, c_int, c_void_p, c_void_p, c_int, c_void_p, c_int, c_void_p, c_void_p, c_void_p, c_void_p, c_void_p,
-              c_void_p, c_void_p, c_int, c_int, c_int, c_int, c_int, c_float, c_int, c_void_p, c_float, c_int, c_void_p])
+              c_void_p, c_void_p, c_int, c_int, c_int, c_int, c_int, c_float, c_int, c_void_p, c_float, c_int, c_void_p, c_void_p])
     _check_sink(sink, H)
+    _check_slope(slope, H)
     _check(fn(_p(q), q.stride(0), T, _p(_contig(k_pages, "k_pages")), _p(_contig(v_pages, "v_pages")), k_pages.shape[0],
               _p(page_table), page_table.stride(0), _p(slots), _p(kv_len), _p(qb_seq), _p(qb_row), _p(qb_rows), _p(qb_pos),
               _p(out), qb_seq.numel(), H, Hkv, hd, page_size, float(scale), int(window or 0), _p(sink), float(softcap or 0.0),
-              int(keep_first if window else 0), _stream()), "attn_prefill_tc")
+              int(keep_first if window else 0), _p(slope), _stream()), "attn_prefill_tc")
     return out
 
 
@@ -1398,7 +1489,8 @@ def attn_decode(q: torch.Tensor, k_pages, v_pages, page_table, tok_pos, tok_seq,
                 out: torch.Tensor | None = None, scratch: tuple | None = None,
                 next_w: torch.Tensor | None = None, early_loads: bool = False,
                 work: torch.Tensor | None = None, teams: int = 0, sink: torch.Tensor | None = None,
-                softcap: float | None = None, keep_first: int = 0, vd: int | None = None) -> torch.Tensor:
+                softcap: float | None = None, keep_first: int = 0, vd: int | None = None,
+                slope: torch.Tensor | None = None) -> torch.Tensor:
     """Attention of single query rows over the paged bfloat16 cache, the keys of each
     sequence cut into n_splits slices that are merged afterwards.  With `work` (int32: teams + 1 offsets,
     then (token, first tile, last tile + 1, part, parts) per segment) the grid is `teams` blocks per kv
@@ -1411,7 +1503,8 @@ def attn_decode(q: torch.Tensor, k_pages, v_pages, page_table, tok_pos, tok_seq,
     scale.  keep_first n (with a window): a token's first n keys stay visible once its window has moved past them;
     the tiles that a work list counts are then the kept tiles ahead of the window and after them the window's.
     window: as `span` makes it (w positions; -n for blocks of n positions, whose tiles a work list counts from the
-    block's first; 0 or None for all).  vd: size of a value head (default hd)."""
+    block's first; 0 or None for all).  vd: size of a value head (default hd).  slope: float32 [H], a score loses slope[h]
+    times the distance to its key, after the scale and the cap."""
     T = q.shape[0]
     vd = vd or hd
     if q.dtype != torch.bfloat16 or k_pages.dtype != torch.bfloat16:
@@ -1445,12 +1538,13 @@ def attn_decode(q: torch.Tensor, k_pages, v_pages, page_table, tok_pos, tok_seq,
     fn = _fn("attn_decode", "lq_attn_decode_vd", [c_void_p, c_int, c_void_p, c_void_p, c_void_p, c_int, c_void_p,
                                                   c_void_p, c_void_p, c_void_p, c_void_p, c_void_p, c_void_p, c_int,
                                                   c_int, c_int, c_int, c_int, c_int, c_float, c_int, c_int, c_void_p, c_int,
-                                                  c_void_p, c_long, c_int, c_void_p, c_float, c_int, c_void_p])
+                                                  c_void_p, c_long, c_int, c_void_p, c_float, c_int, c_void_p, c_void_p])
+    _check_slope(slope, H)
     next_p, next_n = _next(next_w, PREFETCH_BYTES_ATTN)
     _check(fn(_p(q), q.stride(0), _p(k_pages), _p(v_pages), _p(page_table), page_table.stride(0), _p(tok_pos),
               _p(tok_seq), _p(slots), _p(part_o), _p(part_ml), _p(counters), _p(out), T, H, Hkv, hd, vd, page_size,
               float(scale), int(window or 0), n_splits, _p(work), int(teams), next_p, next_n, int(early_loads), _p(sink),
-              float(softcap or 0.0), int(keep_first if window else 0), _stream()),
+              float(softcap or 0.0), int(keep_first if window else 0), _p(slope), _stream()),
            "attn_decode", 2 if n_splits > 1 and counters is None else 1,
            "attn_decode:teams" if work is not None else "attn_decode:one_slice" if n_splits == 1 else "attn_decode:slices")
     return out

@@ -33,7 +33,9 @@ the head's size that all heads share, one for q and one for k) or "all" (one nor
 query projection and one over the whole key projection, each with a weight of that size), in 32-bit on the
 products' 32-bit sums, ahead of the rotation; `q_temp` (coef, every): the queries times
 1 + coef ln(floor((p + 1) / every) + 1) at position p; `chunk` n (instead of a window): position i sees j <= i
-only in its own block of n positions, floor(i / n) = floor(j / n), and the cache gives back the pages below it.
+only in its own block of n positions, floor(i / n) = floor(j / n), and the cache gives back the pages below it;
+`distance_slopes` (one number per head: score_h(i, j) loses slope_h * (i - j), after the scale and the cap, in 32-bit); and
+`values="keys"` (no value projection: a head's values are its keys as projected, ahead of their norm and rotation).
 """
 from __future__ import annotations
 
@@ -67,7 +69,8 @@ class Attention(Mixer):
                  sink: bool = False, gate: str | None = None, softcap: float | None = None, keep_first: int = 0,
                  value_norm_eps: float | None = None, cache_window: int | None | str = "own",
                  cache_keep_first: int | None = None, qk_norm: str | None = None, norm_eps: float = 0.0,
-                 q_temp: tuple | None = None, chunk: int | None = None, out_bias: bool = False):
+                 q_temp: tuple | None = None, chunk: int | None = None, out_bias: bool = False,
+                 distance_slopes: tuple | None = None, values: str = "own"):
         if n_heads % n_kv_heads:
             raise ValueError(f"attention: {n_heads} heads are not a multiple of {n_kv_heads} kv heads")
         if (head_dim % 2 and position is not None) or not 1 <= head_dim <= 256:
@@ -86,6 +89,15 @@ class Attention(Mixer):
             raise ValueError(f"attention: qk_norm {qk_norm!r} is not supported (supported: 'head', 'head_gain', 'all')")
         if chunk is not None and (window is not None or int(chunk) < 1):
             raise ValueError("attention: blocks of positions (chunk >= 1) or a window, not both")
+        if values not in ("own", "keys"):
+            raise ValueError(f"attention: values {values!r} are not supported (supported: 'own', 'keys')")
+        if values == "keys" and (not own_kv or self.vd != head_dim):
+            raise ValueError(f"attention: values that are the keys need keys of their own and the keys' size {head_dim}, not {self.vd}")
+        if distance_slopes is not None and len(distance_slopes) != n_heads:
+            raise ValueError(f"attention: {len(distance_slopes)} distance slopes for {n_heads} heads")
+        self.own_values = values == "own"
+        self.distance_slopes = tuple(float(s) for s in distance_slopes) if distance_slopes is not None else None
+        self.slopes: torch.Tensor | None = None
         if q_temp is not None and not int(q_temp[1]) > 0:
             raise ValueError("attention: q_temp is (coef, every) with every >= 1")
         self.bias, self.sink, self.gate = bool(bias), bool(sink), gate
@@ -116,7 +128,8 @@ class Attention(Mixer):
         # kernels, know the plain form only; every option above takes the general kernels.
         self.general = self.bias or self.out_bias or self.sink or self.gate is not None or self.vd != head_dim or \
             (self.position is not None and self.rot != head_dim) or self.softcap is not None or self.keep_first > 0 or \
-            self.value_norm_eps is not None or self.qk_norm is not None or self.q_temp is not None or self.chunk is not None
+            self.value_norm_eps is not None or self.qk_norm is not None or self.q_temp is not None or self.chunk is not None or \
+            self.distance_slopes is not None or not self.own_values
         self.b_qkv = self.sinks = None
         self.w_qkv: linear.LinearWeight | None = None
         self.w_o: linear.LinearWeight | None = None
@@ -135,12 +148,14 @@ class Attention(Mixer):
         out = {n["q"]: WeightSpec((self.H * self.hd, self.D)), n["o"]: WeightSpec((self.D, self.H * self.vd))}
         if self.own_kv:
             out[n["k"]] = WeightSpec((self.Hkv * self.hd, self.D))
-            out[n["v"]] = WeightSpec((self.Hkv * self.vd, self.D))
+            if self.own_values:
+                out[n["v"]] = WeightSpec((self.Hkv * self.vd, self.D))
         if self.bias:
             out[n["q_bias"]] = WeightSpec((self.H * self.hd,), init="small", full_precision=True)
             if self.own_kv:
                 out[n["k_bias"]] = WeightSpec((self.Hkv * self.hd,), init="small", full_precision=True)
-                out[n["v_bias"]] = WeightSpec((self.Hkv * self.vd,), init="small", full_precision=True)
+                if self.own_values:
+                    out[n["v_bias"]] = WeightSpec((self.Hkv * self.vd,), init="small", full_precision=True)
         if self.out_bias:
             out[n["o_bias"]] = WeightSpec((self.D,), init="small", full_precision=True)
         if self.sink_learned:
@@ -175,14 +190,15 @@ class Attention(Mixer):
             for name in (n[key], n[key + "_bias"], n[key + "_norm"]):
                 if name in tensors and (key == "q" or self.own_kv):
                     tensors[name] = self._reordered(tensors[name], heads)
-        rows = [tensors[n["q"]]] + ([tensors[n["k"]], tensors[n["v"]]] if self.own_kv else [])
+        own = (["k", "v"] if self.own_values else ["k"]) if self.own_kv else []
+        rows = [tensors[n[k]] for k in ["q", *own]]
         if self.gate is not None:
             rows.append(tensors[n["g"]])               # the gate's rows ride in the same product, after q, k and v
         if len({r.dtype for r in rows}) > 1:
             rows = [r.to(torch.float32) for r in rows]
         self.w_qkv = linear.LinearWeight(torch.cat(rows, dim=0))
         if self.bias:
-            keys = ["q_bias"] + (["k_bias", "v_bias"] if self.own_kv else [])
+            keys = [k + "_bias" for k in ["q", *own]]
             self.b_qkv = torch.cat([tensors[n[k]].to(torch.float32) for k in keys]).contiguous()
         if self.sink:
             self.sinks = tensors[n["sink"]].to(torch.float32).contiguous() if self.sink_learned else \
@@ -192,6 +208,8 @@ class Attention(Mixer):
         if self.qk_norm in ("all", "head_gain"):
             keys = ["q_norm"] + (["k_norm"] if self.own_kv else [])
             self.norm_w = torch.cat([tensors[n[k]].to(torch.float32) for k in keys]).contiguous()
+        if self.distance_slopes is not None:
+            self.slopes = torch.tensor(self.distance_slopes, dtype=torch.float32, device=self.runtime.device)
         self.w_o = linear.LinearWeight(tensors[n["o"]])
         if self.position is not None and self.position.weights():
             self.position.load({name: tensors[name] for name in self.position.weights()})
@@ -211,17 +229,18 @@ class Attention(Mixer):
         if self.position is not None and tables is None:
             raise ValueError("attention: a position part without tables cannot be combined with the layer's options")
         cos, sin = tables if tables is not None else (None, None)
-        v_off = (H + G) * hd
+        v_off = (H + G) * hd if self.own_values else H * hd       # values that are the keys: the keys' own columns
         ops.rope_partial(rows, self.b_qkv, cos, sin, self.rot if tables is not None else 0, ctx.tok_pos, ctx.tok_seq,
                          ctx.slots, cache_view.page_table if store else None, cache_view.k_pages if store else None,
                          cache_view.v_pages if store else None, H + (G if self.own_kv else 0), H, G, hd, vd, v_off,
                          cache_view.page_size, qout=q if wide else None, v_unit_eps=self.value_norm_eps,
                          unit_norm="head" if self.qk_norm == "head_gain" else self.qk_norm, norm_weight=self.norm_w, norm_eps=self.norm_eps, q_temp=self.q_temp)
-        g_off = H * hd + (G * (hd + vd) if self.own_kv else 0)
+        g_off = H * hd + (G * (hd + (vd if self.own_values else 0)) if self.own_kv else 0)
         gate = rows[:, g_off:g_off + (H if self.gate_per_head else H * vd)] if self.gate is not None else None
         out = attention_kernels.attention(q, cache_view, ctx, H, G, hd, self.scale, self.window,
                                           next_w=self.w_o.tensor, vd=vd, sink=self.sinks, gate=gate, softcap=self.softcap,
-                                          keep_first=self.keep_first, chunk=self.chunk, gate_per_head=self.gate_per_head)
+                                          keep_first=self.keep_first, chunk=self.chunk, gate_per_head=self.gate_per_head,
+                                          slope=self.slopes)
         out = self._project(out, residual, None)
         if self.out_bias and bias:
             ops.add_bias(out if residual is None else residual, self.branch_bias)

@@ -197,6 +197,11 @@ class Norm(Part):
         do its work for `n_rows` rows (see Mixer.folds_norm); None otherwise."""
         return None
 
+    def affine(self) -> tuple | None:
+        """(gain, bias or None, eps, center): (x - center * mean(x)) over its root mean square, times gain, plus bias -- for
+        kernels that make this norm's rows as they leave the stream (ops.join_branch); None for a norm of another form."""
+        return None
+
 
 class PositionEncoding(Part):
     """Either gives cos/sin tables for the fused rotate-and-store kernel, or rotates

@@ -11,7 +11,8 @@ steps kept as the layer's own state; and `residual_scale` m, x += m * mixer(...)
 the mixer and the feed-forward hand back their branches as float32 rows.
 
 "stream_mix": no mixer and no feed-forward; the stream is replaced by a product over the stream and the embedding's
-rows side by side, x <- W [x; e] (what a pass over repeated layers starts with).
+rows side by side, x <- W [x; e] (what a pass over repeated layers starts with).  "stream_add": the same place without a
+product, x <- x + e.
 
 "post_norm": the sublayers read the stream itself and what they return is normed, x += norm1(mixer(x));
 x += norm2(ffn(x)), a layer may have no feed-forward.  The branch's norm (and, for a mixer of two sides whose outputs are
@@ -19,7 +20,9 @@ normed first, theirs and the sum), the addition and the rows that the next subla
 
 "sandwich_norm": every branch is normed on both sides, x += norm1b(mixer(norm1(x)));
 x += norm2b(ffn(norm2(x))), and a layer may have no feed-forward.  The branch's own norm,
-the addition and the norm that reads the stream next are one kernel."""
+the addition and the norm that reads the stream next are one kernel.  The norms may be RMS norms or layer norms, and
+`residual_scale` m multiplies a branch as it joins, x += m norm1b(...); that kernel also makes the addition of a
+"stream_add" that follows."""
 from __future__ import annotations
 
 import torch
@@ -27,7 +30,7 @@ import torch
 from ..kernels import linear, ops
 from ..weights.spec import WeightSpec
 from .base import Part, Runtime, StepContext
-from .norm import RMSNorm
+from .norm import LayerNorm, RMSNorm
 from .registry import make_part, register_part
 from .spec import LayerSpec
 
@@ -156,8 +159,8 @@ class SandwichNormBlock(Part):
 
     folds_norm = True
 
-    def __init__(self, runtime: Runtime, layer: LayerSpec):
-        self.prefix, self.runtime = layer.prefix, runtime
+    def __init__(self, runtime: Runtime, layer: LayerSpec, residual_scale: float = 1.0):
+        self.prefix, self.runtime, self.scale = layer.prefix, runtime, float(residual_scale)
         places = set(layer.parts)
         unknown = places - {"norm1", "mixer", "norm1b", "norm2", "ffn", "norm2b"}
         if unknown:
@@ -175,8 +178,13 @@ class SandwichNormBlock(Part):
             raise ValueError(f"layer {layer.prefix!r}: the mixer {layer.part('mixer').kind!r} cannot hand back its "
                              f"output for a norm of its own")
         for norm in self.norms():
-            if not hasattr(norm, "gain") or not hasattr(norm, "eps"):
-                raise ValueError(f"layer {layer.prefix!r}: the arrangement 'sandwich_norm' needs RMS norms with a gain")
+            if not isinstance(norm, (RMSNorm, LayerNorm)):
+                raise ValueError(f"layer {layer.prefix!r}: the arrangement 'sandwich_norm' needs RMS norms or layer norms")
+        # Layer norms and a multiplier on the branches take the kernel for norms of any kind; that one also makes the rows of
+        # whatever norm comes next (`emits_any_norm`) and adds the embedding's rows on the way (`takes_extra`).
+        self.general = self.scale != 1.0 or any(isinstance(norm, LayerNorm) for norm in self.norms())
+        self.emits_any_norm = self.takes_extra = self.general
+        self.kernel_libraries = ("post_norm",) if self.general else ()
 
     def norms(self):
         return tuple(n for n in (self.norm1, self.norm1b, self.norm2, self.norm2b) if n is not None)
@@ -212,15 +220,31 @@ class SandwichNormBlock(Part):
 
     def input_norm(self, n_rows: int):
         """(gain, eps) of norm1: the layer ahead may make its rows in the kernel that ends it."""
-        return (self.norm1.gain, self.norm1.eps) if self.norm1.gain is not None else None
+        return (self.norm1.gain, self.norm1.eps) if isinstance(self.norm1, RMSNorm) and self.norm1.gain is not None else None
 
-    def forward(self, x, ctx: StepContext, cache_view, writes_cache: bool = True, normed=None, emit=None):
+    def first_norm(self):
+        """The norm whose rows the layer starts from, as `Norm.affine` gives it: for a layer ahead that can make any norm's rows."""
+        return self.norm1.affine()
+
+    def _forward_general(self, x, ctx, cache_view, writes_cache, h, emit_norm, extra):
+        act = self.runtime.act_dtype
+        y = self.mixer.forward(h, ctx, cache_view, None, writes_cache)
+        if not self.has_ffn:
+            return ops.join_branch(x, y, self.norm1b.affine(), self.scale, extra, emit_norm, act)
+        h = ops.join_branch(x, y, self.norm1b.affine(), self.scale, None, self.norm2.affine(), act)
+        y = self.ffn.forward(h, ctx, None)
+        return ops.join_branch(x, y, self.norm2b.affine(), self.scale, extra, emit_norm, act)
+
+    def forward(self, x, ctx: StepContext, cache_view, writes_cache: bool = True, normed=None, emit=None, emit_norm=None, extra=None):
         """`normed`: the rows of norm1 when the layer ahead made them; `emit`: the next layer's
-        input_norm().  Returns the next layer's rows, or None."""
+        input_norm(); with `emits_any_norm`, `emit_norm`: its first_norm(); with `takes_extra`, `extra`: rows that join the
+        stream as the layer ends.  Returns the next layer's rows, or None."""
         act = self.runtime.act_dtype
         if isinstance(normed, ops.NormedRows):
             normed = normed.finish()
         h = normed if normed is not None else self.norm1.forward(x)
+        if self.general:
+            return self._forward_general(x, ctx, cache_view, writes_cache, h, emit_norm, extra)
         y = self.mixer.forward(h, ctx, cache_view, None, writes_cache)
         if not self.has_ffn:
             return ops.rmsnorm_add(y, self.norm1b.gain, self.norm1b.eps, x, emit, act)
@@ -337,3 +361,28 @@ class StreamMixBlock(Part):
 
     def forward(self, x, ctx: StepContext, embedded):
         return linear.linear(ops.side_by_side(x, embedded, self.runtime.act_dtype), self.w, torch.float32)
+
+
+@register_part("block", "stream_add")
+class StreamAddBlock(Part):
+    """x <- x + e, e the embedding's output for the same rows (what a pass over repeated layers starts with).  Where the layer
+    ahead can (`takes_extra`), its last kernel makes the addition and this block does not run.  It keeps nothing in the cache."""
+    graph_safe = True
+    folds_norm = False
+    replaces_stream = True
+    reads_embedding = True
+    adds_embedding = True        # nothing but x += e
+
+    def __init__(self, runtime: Runtime, layer: LayerSpec):
+        if layer.parts:
+            raise ValueError(f"layer {layer.prefix!r}: the arrangement 'stream_add' has no places for parts")
+        self.prefix = layer.prefix
+
+    def parts(self):
+        return ()
+
+    def cache_need(self):
+        return None
+
+    def forward(self, x, ctx: StepContext, embedded):
+        return ops.add_scaled(x, embedded, 1.0)

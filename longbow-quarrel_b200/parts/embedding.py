@@ -1,6 +1,6 @@
 """Token embedding and output head.
 
-Embedding: row `token` of the table, no multiplier, promoted to the 32-bit residual
+Embedding: row `token` of the table, no multiplier unless asked for, promoted to the 32-bit residual
 stream (internal/device/kernels.metal:465-467; internal/engine/engine.go:1365-1375).
 Head: logits = n . W^T in 32-bit (internal/engine/engine.go:1561;
 internal/device/kernels.metal:1172-1194), reading the embedding table when the
@@ -21,8 +21,12 @@ from .spec import PartSpec
 class TokenEmbedding(Part):
     graph_safe = True
 
-    def __init__(self, runtime: Runtime, vocab_size: int, hidden_size: int, name: str, norm: PartSpec | None = None):
-        """norm: an RMS norm with a gain that the rows pass before they become the stream."""
+    def __init__(self, runtime: Runtime, vocab_size: int, hidden_size: int, name: str, norm: PartSpec | None = None, scale: float = 1.0):
+        """norm: an RMS norm with a gain that the rows pass before they become the stream.  scale: the rows are multiplied by
+        this constant, in 32-bit (without a norm)."""
+        self.scale = float(scale)
+        if norm is not None and self.scale != 1.0:
+            raise ValueError("token_embedding: a multiplier on the rows or a norm, not both")
         self.runtime, self.vocab_size, self.hidden_size, self.name = runtime, vocab_size, hidden_size, name
         self.norm = make_part("norm", norm, runtime) if norm is not None else None
         if self.norm is not None and not (hasattr(self.norm, "gain") and hasattr(self.norm, "eps") and not hasattr(self.norm, "bias")):
@@ -44,7 +48,7 @@ class TokenEmbedding(Part):
 
     def forward(self, tokens: torch.Tensor, emit_stream: bool = False):
         if self.norm is None:
-            return ops.embedding(self.table, tokens)
+            return ops.embedding(self.table, tokens, scale=self.scale)
         x, rows = ops.embedding_norm(self.table, tokens, self.norm.gain, self.norm.eps, self.runtime.act_dtype if emit_stream else None)
         return (x, rows) if emit_stream else x
 

@@ -6,7 +6,7 @@
     g_e = s_e / (sum of the chosen s + 1e-20) * route_scale
     y = sum_e g_e W_down,e act(W_up,e h)  [ + sigmoid(w_sg . h) * shared(h) ]
 
-The experts have no gate and no bias.  A shared expert (a `dense_mlp` of its own size) runs for every
+The experts have no gate and no bias; act is any of `ops.MOE_ACTS` (gelu in two forms, silu, relu, the square of relu).  A shared expert (a `dense_mlp` of its own size) runs for every
 token behind one sigmoid number per token.
 
 Options that other designs use, each a parameter: `score` "softmax" (over all router outputs) instead of "sigmoid";

@@ -38,6 +38,9 @@ class RMSNorm(Norm):
     def forward(self, x, rows=None):
         return ops.rmsnorm(x, self.gain, self.eps, self.runtime.act_dtype, rows)
 
+    def affine(self):
+        return self.gain, None, self.eps, False
+
     def foldable(self, n_rows):
         if self.gain is None or not linear.can_defer_norm(n_rows, self.size, self.runtime.act_dtype):
             return None
@@ -67,5 +70,8 @@ class LayerNorm(Norm):
     def forward(self, x, rows=None, add=()):
         """add: ((y, m), ...) branches that join the stream (x += m * y, in place) in the same pass."""
         return ops.layernorm(x, self.gain, self.bias, self.eps, self.runtime.act_dtype, rows, add=add)
+
+    def affine(self):
+        return self.gain, self.bias, self.eps, True
 
     takes_branches = True       # forward(add=...) adds a mixer's branches as it norms
