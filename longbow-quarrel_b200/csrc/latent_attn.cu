@@ -163,6 +163,7 @@ LQ_EXPORT int lq_head_matmul(const void* in, int in_dtype, int in_stride, int in
         return launch_pdl(head_matmul_kernel<TI, TW, TO>, grid, dim3(256), smem, stream, (const TI*)in, in_stride, in_head, in_off, \
                           (const TW*)w, (TO*)out, out_stride, out_head, out_off, T, K, N); } while (0)
     if (in_dtype == LQ_F32 && w_dtype == LQ_F32 && out_dtype == LQ_F32) LQ_GO(float, float, float);
+    if (in_dtype == LQ_F32 && w_dtype == LQ_F32 && out_dtype == LQ_BF16) LQ_GO(float, float, bf);
     if (in_dtype == LQ_F32 && w_dtype == LQ_BF16 && out_dtype == LQ_F32) LQ_GO(float, bf, float);
     if (in_dtype == LQ_F32 && w_dtype == LQ_BF16 && out_dtype == LQ_BF16) LQ_GO(float, bf, bf);
     if (in_dtype == LQ_BF16 && w_dtype == LQ_BF16 && out_dtype == LQ_F32) LQ_GO(bf, bf, float);
