@@ -402,6 +402,8 @@ def design_bench(args) -> int:
         return lavutar_bench(args)
     if args.design == "korazen":
         return korazen_bench(args)
+    if args.design == "gevipel":
+        return gevipel_bench(args)
     return fetorax_bench(args)
 
 
@@ -910,6 +912,119 @@ def korazen_bench(args) -> int:
     return 0
 
 
+def gevipel_config(size: str, window: int) -> dict:
+    """Four layers, each with routed experts: the gated delta rule with one decay per head, windowed attention whose values are
+    the keys, the delta rule, latent attention with a sink."""
+    width, heads, kv, dim, _ = DESIGN_SIZES[size]
+    _, zh, dn, dr, dv, _, rkv, _, experts, top, eff, _ = ZOPORAX_SIZES[size]
+    moe = {"kind": "moe", "expert": {"ff": eff}, "router": {"experts": experts, "top": top}}
+    delta = {"type": "delta", "mlp": moe, "mixer": {"heads": heads, "kv_heads": heads, "dim": dim, "vdim": dim, "conv": 4}}
+    att = {"type": "attention", "mlp": moe, "mixer": {"heads": heads, "kv_heads": kv, "dim": dim, "vdim": dim, "scale": dim ** -0.5,
+                                                      "mask": {"size": window}, "q_temp": {"coef": 0.1, "every": 512}}}
+    lat = {"type": "latent_attention", "mlp": moe, "mixer": {"heads": zh, "dim": dn, "rot_dim": dr, "vdim": dv, "kv_rank": rkv,
+                                                             "scale": (dn + dr) ** -0.5, "rot": {"dims": dr, "base": 1e4}}}
+    return {"architecture": "Gevipel", "vocab": DESIGN_VOCAB, "width": width, "embedding": {"scale": 2.0}, "norm": {"eps": 1e-5},
+            "residual_mult": 0.5, "layers": [delta, att, delta, lat], "max_positions": 8192}
+
+
+def zoporax_twin(size: str) -> dict:
+    """A Zoporax model of the same width, depth, latent attention and experts for `gevipel_config`: lightning and latent
+    attention over all positions by turns, each with routed experts and no shared one."""
+    cfg = zoporax_config(size, 8192)
+    lat, lig = cfg["layers"][2], cfg["layers"][1]
+    moe = {k: v for k, v in lig["mlp"].items() if k != "shared"}
+    lat, lig = {**lat, "mlp": moe, "mixer": {k: v for k, v in lat["mixer"].items() if k != "mask"}}, {**lig, "mlp": moe}
+    return {**cfg, "layers": [lig, lat, lig, lat]}
+
+
+def gevipel_bench(args) -> int:
+    """Prefill and decode of a Gevipel model of realistic layer sizes beside the closest models the library has, a Zoporax
+    model (latent attention and experts of the same sizes) and, for the delta rule and the attention, a Korazen model of the
+    same width and heads (random weights, vocabulary 32,000): tokens a second, what every kind of kernel adds to a prompt
+    step and to a decode step, and how many times their roofline the design's kernels take, beside the like kernels."""
+    import numpy as np
+    import torch
+
+    from longbow_quarrel_b200.engine import Engine
+    peaks, peaks_from = load_peaks()
+    K, W = args.steps, max(3, args.warmup)
+    T, B, ctx, window = PREFILL_TOKENS, BATCH, 2048, 1280
+    hbm, tensor = peaks["hbm_gbs"] * 1e9, peaks["bf16_tflops"] * 1e12
+    rng = np.random.default_rng(0)
+    sampler = ClockSampler()
+    sampler.start()
+    out = {}
+    for size in args.sizes.split(","):
+        width, heads, kv, dim, _ = DESIGN_SIZES[size]
+        _, zh, dn, dr, dv, _, rkv, _, experts, top, eff, _ = ZOPORAX_SIZES[size]
+        configs = {"gevipel": gevipel_config(size, window), "zoporax": zoporax_twin(size), "korazen": korazen_config(size, window)}
+        res = {name: _design_run(torch, np, Engine, cfg, name, T, B, ctx, K, W, rng) for name, cfg in configs.items()}
+
+        def each(kinds, launches, *names):
+            """us of one application of an operation that these kernels make together, `launches` times in the step"""
+            us = sum(kinds[k][1] for k in names if k in kinds)
+            return us / launches if us else None
+
+        def roof(us, nbytes, flops=0.0):
+            """(us, times the roofline)"""
+            return [round(us, 1), round(us / (max(nbytes / hbm, flops / tensor) * 1e6), 2)] if us else None
+        (gp, gd), (zp, zd), (kp, kd) = ((res[n]["prefill_kernels_us"], res[n]["decode_kernels_us"]) for n in ("gevipel", "zoporax", "korazen"))
+        full = T * (T + 1) / 2
+        seen = window * (window + 1) / 2 + (T - window) * window
+        blocks = window * (window + 1) / 2 + (T - window) * (T - window + 1) / 2
+        per_head, state = T * heads * dim, B * heads * dim * dim * 4.0 * 2
+        Dk = rkv + dr
+        latent = T * zh * (Dk + rkv) * 4.0 + T * Dk * 2.0, 2.0 * zh * (Dk + rkv) * full
+        chosen = min(B * top, experts) * eff * width * 2.0
+        attn = ("attn_prefill_two", "attn_prefill_tc")
+        times = {
+            "prefill": {
+                # q, k, v, the gate and the outputs, 32-bit each but the last; read-out, correction and write of a state per head and token.
+                "delta rule, one decay per head (with norm and gate)": roof(each(gp, 2, "prepare", "scan", "output"), per_head * (4 * 4 + 2.0), 6.0 * per_head * dim),
+                "korazen delta rule, channel decays (with norm and gate)": roof(each(kp, 2, "delta_prepare", "delta_scan") and each(kp, 2, "delta_prepare", "delta_scan")
+                                                                                + each(kp, 4, "head_norm_gate", "head_norm_gate_wide"),
+                                                                                per_head * (5 * 4 + 2 + 2.0), 6.0 * per_head * dim),
+                "attention, window and slopes": roof(each(gp, 1, *attn), T * (2 * heads + 2 * kv) * dim * 2.0, 4.0 * heads * dim * seen),
+                "korazen attention, blocks": roof(each(kp, 1, *attn), T * (2 * heads + 2 * kv) * dim * 2.0, 4.0 * heads * dim * blocks),
+                "unit norms + temperature + cache write": roof(each(gp, 1, "rope_partial"), T * (heads + kv) * dim * 6.0 + T * kv * dim * 2.0),
+                "korazen biases + unit norms + rotation + cache write": roof(each(kp, 2, "rope_partial"), T * (heads + 1.5 * kv) * dim * 6.0 + T * kv * dim * 3.0),
+                "latent attention with sink": roof(each(gp, 1, "latent_attention_tc", "latent_attention"), *latent),
+                "zoporax latent attention": roof(each(zp, 2, "latent_attention_tc", "latent_attention"), *latent),
+                "branch norm + multiplier + add + next norm": roof(each(gp, 8, "join_branch"), T * width * (4 + 8 + 2.0)),
+                "korazen branch norm + add + rows": roof(each(kp, 8, "join"), (6 * T * width * 14.0 + 2 * T * width * 18.0) / 8),
+                # The experts' eight products are launches of gemm_tc, which also serves small products of the step (an upper bound).
+                "experts, either product": roof(each(gp, 8, "gemm_tc"), experts * eff * width * 2.0, 2.0 * T * top * eff * width),
+                "zoporax experts, either product": roof(each(zp, 8, "gemm_tc"), experts * eff * width * 2.0, 2.0 * T * top * eff * width),
+                "experts' activation": roof(each(gp, 4, "activation", "activation_vec"), T * top * eff * 4.0),
+                "zoporax experts' activation": roof(each(zp, 4, "activation", "activation_vec"), T * top * eff * 4.0),
+            },
+            "decode": {
+                "delta rule, one decay per head (one kernel)": roof(each(gd, 2, "delta_single"), state),
+                "korazen delta rule, channel decays (one kernel)": roof(each(kd, 2, "delta_single"), state + 2 * heads * dim * 64 * 2.0),
+                "attention, window and slopes": roof(each(gd, 1, "attn_decode"), B * window * 2 * kv * dim * 2.0),
+                "korazen attention (both value sizes)": roof(each(kd, 2, "attn_decode"), B * ((ctx + W + K // 2) % window + 1) * kv * dim * 5.0),
+                "latent attention with sink": roof(each(gd, 1, "latent_attention_tc", "latent_merge_tc", "latent_attention"), B * ctx * Dk * 2.0),
+                "zoporax latent attention": roof(each(zd, 2, "latent_attention_tc", "latent_merge_tc", "latent_attention"), B * ctx * Dk * 2.0),
+                "branch norm + multiplier + add + next norm": roof(each(gd, 8, "join_branch"), B * width * 14.0),
+                "korazen branch norm + add + rows": roof(each(kd, 8, "join"), B * width * 14.0),
+                "experts, first product": roof(each(gd, 4, "moe_up"), chosen),
+                "zoporax experts, first product": roof(each(zd, 4, "moe_up"), chosen),
+                "experts, second product": roof(each(gd, 4, "moe_down"), chosen),
+                "zoporax experts, second product": roof(each(zd, 4, "moe_down"), chosen),
+            },
+        }
+        out[size] = {**res, "us_and_times_the_roofline": times,
+                     "gevipel_over_zoporax": {"prefill": round(res["gevipel"]["prefill_tokens_per_s"] / res["zoporax"]["prefill_tokens_per_s"], 3),
+                                              "decode": round(res["gevipel"]["decode_tokens_per_s"] / res["zoporax"]["decode_tokens_per_s"], 3)}}
+    clocks = sampler.stop()
+    print(json.dumps({"design": "gevipel", "beside": "zoporax and korazen", "dtype": "bf16", "data": "synthetic", "layers": 4,
+                      "layer_order": "delta rule, windowed attention, delta rule, latent attention; beside lightning, latent attention, lightning, latent "
+                                     "attention; each + experts; and beside delta rule, two sides, delta rule, two sides, each + gated ff",
+                      "vocab": DESIGN_VOCAB, "prefill_tokens": T, "decode_batch": B, "decode_context": ctx, "steps": K,
+                      "warmup": W, "peaks": peaks, "peaks_from": peaks_from, "clocks": clocks, "sizes": out}))
+    return 0
+
+
 def fetorax_bench(args) -> int:
     """Prefill and decode of a Fetorax model of the 1B and 8B layer sizes beside a Llama model of the same sizes
     (random weights, vocabulary cut to 32,000): tokens a second, the device time of every kind of kernel in one
@@ -1019,7 +1134,7 @@ def fetorax_bench(args) -> int:
 
 def main() -> int:
     ap = argparse.ArgumentParser()
-    ap.add_argument("--design", default="", choices=["", "fetorax", "zoporax", "raritar", "lavutar", "korazen"],
+    ap.add_argument("--design", default="", choices=["", "fetorax", "zoporax", "raritar", "lavutar", "korazen", "gevipel"],
                     help="instead of the default workload: this design beside the closest model the library has, at equal layer "
                          "sizes (prefill, decode, kernel by kernel): fetorax beside Llama, zoporax beside Fetorax, raritar beside Llama, lavutar beside Fetorax, korazen beside Lavutar")
     ap.add_argument("--sizes", default="1b,8b", help="--design: layer sizes to run, of " + ", ".join(DESIGN_SIZES))
