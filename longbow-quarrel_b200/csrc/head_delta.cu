@@ -88,37 +88,52 @@ __global__ void __launch_bounds__(NT, NT == 128 ? 4 : 2) prepare_kernel(const __
         const int p = pos0 + t0 + i;
         return p >= 0 ? ring[(size_t)(p % taps) * a.C + c] : 0.f;
     };
-    // Convolution and silu of channel c for the tokens t .. t + 3; zero behind the chunk's last one.
-    auto conv4 = [&](int c, int t) -> float4 {
-        float y[4] = {0.f, 0.f, 0.f, 0.f};
-        if (taps == 4 && t0 + t >= 3 && t + 4 <= n) {
-            const float* p = a.rows + (ptrdiff_t)(row0 + t - 3) * a.stride + c;
-            float x[7];
+    // Convolution and silu of channel c for the tokens t .. t + 15 (zero behind the chunk's last one), to dst[0 .. 15].
+    auto conv16 = [&](int c, int t, float* dst) {
+        float y[16];
 #pragma unroll
-            for (int i = 0; i < 7; ++i, p += a.stride) x[i] = *p;
+        for (int i = 0; i < 16; ++i) y[i] = 0.f;
+        if (taps <= 4) {
+            float x[19], w[4];                   // rows t - 3 .. t + 15; fewer taps leave the first weights at zero
 #pragma unroll
-            for (int j = 0; j < 4; ++j) {
-                const float w = a.taps_w[(size_t)j * a.C + c];
+            for (int j = 0; j < 4; ++j) w[j] = j >= 4 - taps ? a.taps_w[(size_t)(j - (4 - taps)) * a.C + c] : 0.f;
+            if (t0 + t >= 3 && t + 16 <= n) {
+                const float* p = a.rows + (ptrdiff_t)(row0 + t - 3) * a.stride + c;
 #pragma unroll
-                for (int i = 0; i < 4; ++i) y[i] = fmaf(w, x[i + j], y[i]);
+                for (int i = 0; i < 19; ++i) x[i] = p[(ptrdiff_t)i * a.stride];
+            } else {
+#pragma unroll
+                for (int i = 0; i < 19; ++i) x[i] = i >= 4 - taps && t - 3 + i < n ? input(t - 3 + i, c) : 0.f;
             }
+#pragma unroll
+            for (int j = 0; j < 4; ++j)
+#pragma unroll
+                for (int i = 0; i < 16; ++i) y[i] = fmaf(w[j], x[i + j], y[i]);
         } else {
             for (int j = 0; j < taps; ++j) {
                 const float w = a.taps_w[(size_t)j * a.C + c];
 #pragma unroll
-                for (int i = 0; i < 4; ++i)
+                for (int i = 0; i < 16; ++i)
                     if (t + i < n) y[i] = fmaf(w, input(t + i - keep + j, c), y[i]);
             }
         }
 #pragma unroll
-        for (int i = 0; i < 4; ++i) y[i] = t + i < n ? silu_f(y[i]) : 0.f;
-        return make_float4(y[0], y[1], y[2], y[3]);
+        for (int i = 0; i < 16; i += 4) {
+#pragma unroll
+            for (int k = 0; k < 4; ++k) y[i + k] = t + i + k < n ? __fdividef(y[i + k], 1.f + __expf(-y[i + k])) : 0.f;
+            *reinterpret_cast<float4*>(dst + i) = make_float4(y[i], y[i + 1], y[i + 2], y[i + 3]);
+        }
     };
 
-    for (int j = tid; j < 2 * dk4 * (HC / 4); j += NT) {
-        const int c = j % (2 * dk4), t = j / (2 * dk4) * 4, r = c % dk4;
-        const float4 y = r < dk ? conv4((c < dk4 ? 0 : a.G * dk) + g * dk + r, t) : make_float4(0.f, 0.f, 0.f, 0.f);
-        *reinterpret_cast<float4*>((c < dk4 ? qT : kT) + (size_t)r * LT + t) = y;
+    for (int j = tid; j < 2 * dk4 * (HC / 16); j += NT) {
+        const int c = j % (2 * dk4), t = j / (2 * dk4) * 16, r = c % dk4;
+        float* dst = (c < dk4 ? qT : kT) + (size_t)r * LT + t;
+        if (r < dk) {
+            conv16((c < dk4 ? 0 : a.G * dk) + g * dk + r, t, dst);
+        } else {
+#pragma unroll
+            for (int i = 0; i < 16; i += 4) *reinterpret_cast<float4*>(dst + i) = make_float4(0.f, 0.f, 0.f, 0.f);
+        }
     }
     if (tid < HC) {
         const bool in = tid < n;
@@ -190,6 +205,7 @@ __global__ void __launch_bounds__(NT, NT == 128 ? 4 : 2) prepare_kernel(const __
             while (PER * (ti + 1) * (ti + 2) / 2 <= j) ++ti;
             const int si = j - PER * ti * (ti + 1) / 2, t = ti * TM, s = si * 4;
             float kk[TM][4] = {}, qk[TM][4] = {};
+#pragma unroll 2
             for (int r = 0; r < dk4; ++r) {
                 const float* kr = kT + r * LT;
                 const float4 x = *reinterpret_cast<const float4*>(kr + s);
@@ -229,52 +245,79 @@ __global__ void __launch_bounds__(NT, NT == 128 ? 4 : 2) prepare_kernel(const __
         }
     }
     __syncthreads();
-    for (int j = tid; j < dv * (HC / 4); j += NT) {
-        const int e = j % dv, t = j / dv * 4;
-        *reinterpret_cast<float4*>(qT + (size_t)e * LT + t) = conv4(2 * a.G * dk + h * dv + e, t);
+    for (int j = tid; j < dv * (HC / 16); j += NT) {
+        const int e = j % dv, t = j / dv * 16;
+        conv16(2 * a.G * dk + h * dv + e, t, qT + (size_t)e * LT + t);
     }
     __syncthreads();
-    // The triangle's solutions, a thread per column: W's columns from b e^l k, V' columns from b v.
-    const int cols = a.ld + a.tiles * a.n;
-    for (int col = tid; col < cols; col += NT) {
-        const bool key = col < a.ld;
-        const int e = key ? col : col - a.ld;
-        const bool in = key ? e < dk4 : e < dv;
-        const float* src = (key ? kT : qT) + (size_t)(in ? e : 0) * LT;
-        float x[HC];
+    // The triangle's solutions, where the columns lie: W's from b e^l k, V' from b v.  Two columns a thread (an entry of the
+    // triangle read from shared memory serves both; four leave too few warps), sixteen rows at a time: what the rows above them
+    // leave, then the rows themselves one after the other.  (What lies between dk4 and ld, and behind dv, is never read into anything that counts.)
+    constexpr int CT = 2;
+    const int cols = dk4 + dv, per = (cols + CT - 1) / CT;
+    for (int c = tid; c < per; c += NT) {
+        float* src[CT];
+        float* dst[CT];
+        int step[CT];
+        bool key[CT];
 #pragma unroll
-        for (int t = 0; t < HC; t += 4) {
-            const float4 v = *reinterpret_cast<const float4*>(src + t), bt = *reinterpret_cast<const float4*>(sb + t);
-            const float4 et = *reinterpret_cast<const float4*>(se + t);
-            x[t] = in ? v.x * bt.x * (key ? et.x : 1.f) : 0.f;
-            x[t + 1] = in ? v.y * bt.y * (key ? et.y : 1.f) : 0.f;
-            x[t + 2] = in ? v.z * bt.z * (key ? et.z : 1.f) : 0.f;
-            x[t + 3] = in ? v.w * bt.w * (key ? et.w : 1.f) : 0.f;
+        for (int j = 0; j < CT; ++j) {
+            const int col = min(c + j * per, cols - 1);
+            key[j] = col < dk4;
+            const int e = key[j] ? col : col - dk4;
+            src[j] = (key[j] ? kT : qT) + (size_t)e * LT;
+            dst[j] = key[j] ? a.W + (chunk * a.H + h) * HC * a.ld + e : a.V + ((chunk * a.H + h) * a.tiles + e / a.n) * HC * a.n + e % a.n;
+            step[j] = key[j] ? a.ld : a.n;
         }
+#pragma unroll 1
+        for (int r0 = 0; r0 < HC; r0 += 16) {
+            float x[CT][16];
 #pragma unroll
-        for (int t = 1; t < HC; ++t) {
-            float s0 = 0.f, s1 = 0.f, s2 = 0.f, s3 = 0.f;
+            for (int t = 0; t < 16; t += 4) {
+                const float4 bt = *reinterpret_cast<const float4*>(sb + r0 + t), et = *reinterpret_cast<const float4*>(se + r0 + t);
 #pragma unroll
-            for (int s = 0; s < t; s += 4) {
-                const float4 m = *reinterpret_cast<const float4*>(M + t * LT + s);       // zero on and above the diagonal
-                s0 = fmaf(m.x, x[s], s0);
-                if (s + 1 < t) s1 = fmaf(m.y, x[s + 1], s1);
-                if (s + 2 < t) s2 = fmaf(m.z, x[s + 2], s2);
-                if (s + 3 < t) s3 = fmaf(m.w, x[s + 3], s3);
+                for (int j = 0; j < CT; ++j) {
+                    const float4 v = *reinterpret_cast<const float4*>(src[j] + r0 + t);
+                    x[j][t] = v.x * bt.x * (key[j] ? et.x : 1.f);
+                    x[j][t + 1] = v.y * bt.y * (key[j] ? et.y : 1.f);
+                    x[j][t + 2] = v.z * bt.z * (key[j] ? et.z : 1.f);
+                    x[j][t + 3] = v.w * bt.w * (key[j] ? et.w : 1.f);
+                }
             }
-            x[t] -= (s0 + s1) + (s2 + s3);
-        }
-        float* dst;
-        int step;
-        if (key) {
-            dst = a.W + (chunk * a.H + h) * HC * a.ld + e;
-            step = a.ld;
-        } else {
-            dst = a.V + ((chunk * a.H + h) * a.tiles + e / a.n) * HC * a.n + e % a.n;
-            step = a.n;
-        }
+#pragma unroll 1
+            for (int s0 = 0; s0 < r0; s0 += 4) {
+                float4 y[CT];
 #pragma unroll
-        for (int t = 0; t < HC; ++t) dst[(size_t)t * step] = x[t];
+                for (int j = 0; j < CT; ++j) y[j] = *reinterpret_cast<const float4*>(src[j] + s0);
+#pragma unroll
+                for (int i = 0; i < 16; ++i) {
+                    const float4 m = *reinterpret_cast<const float4*>(M + (r0 + i) * LT + s0);
+#pragma unroll
+                    for (int j = 0; j < CT; ++j)
+                        x[j][i] = fmaf(-m.w, y[j].w, fmaf(-m.z, y[j].z, fmaf(-m.y, y[j].y, fmaf(-m.x, y[j].x, x[j][i]))));
+                }
+            }
+#pragma unroll
+            for (int i = 1; i < 16; ++i)
+#pragma unroll
+                for (int q = 0; q < i; q += 4) {
+                    const float4 m = *reinterpret_cast<const float4*>(M + (r0 + i) * LT + r0 + q);       // zero on and above the diagonal
+                    const float mv[4] = {m.x, m.y, m.z, m.w};
+#pragma unroll
+                    for (int k = 0; k < 4; ++k)
+                        if (q + k < i)
+#pragma unroll
+                            for (int j = 0; j < CT; ++j) x[j][i] = fmaf(-mv[k], x[j][q + k], x[j][i]);
+                }
+#pragma unroll
+            for (int j = 0; j < CT; ++j) {
+                if (c + j * per >= cols) break;
+#pragma unroll
+                for (int t = 0; t < 16; ++t) dst[j][(size_t)(r0 + t) * step[j]] = x[j][t];
+#pragma unroll
+                for (int t = 0; t < 16; t += 4) *reinterpret_cast<float4*>(src[j] + r0 + t) = make_float4(x[j][t], x[j][t + 1], x[j][t + 2], x[j][t + 3]);
+            }
+        }
     }
 }
 
@@ -420,14 +463,16 @@ __global__ void __launch_bounds__((2 * WC + 1) * 32, 1) scan_kernel(const __grid
 #pragma unroll
                 for (int c = 0; c < 2; ++c)
                     A[i][p][c] = pack2(fmaf(S[i][2 * p][c], E, S[i][2 * p][c]), fmaf(S[i][2 * p + 1][c], E, S[i][2 * p + 1][c]));
+        const float* kp[RI];                     // rows behind the last key channel repeat the last ones and are not used
+#pragma unroll
+        for (int i = 0; i < RI; ++i) kp[i] = k + min(row_of(i), dk4 - 4);
 #pragma unroll 8
         for (int t = 0; t < HC; ++t) {
             const float2 u = *reinterpret_cast<const float2*>(us + t * N + c0);
             const f2 u0 = pack2(u.x, u.x), u1 = pack2(u.y, u.y);
 #pragma unroll
             for (int i = 0; i < RI; ++i) {
-                if (row_of(i) >= dk4) continue;
-                const ulonglong2 x = *reinterpret_cast<const ulonglong2*>(k + (size_t)t * ld + row_of(i));
+                const ulonglong2 x = *reinterpret_cast<const ulonglong2*>(kp[i] + t * ld);
                 A[i][0][0] = fma2(x.x, u0, A[i][0][0]);
                 A[i][1][0] = fma2(x.y, u0, A[i][1][0]);
                 A[i][0][1] = fma2(x.x, u1, A[i][0][1]);
