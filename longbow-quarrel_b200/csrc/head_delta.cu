@@ -322,12 +322,13 @@ __global__ void __launch_bounds__(NT, NT == 128 ? 4 : 2) prepare_kernel(const __
 }
 
 // ------------------------------------------------------------------ scan
-// 8 WC value columns of a head; 2 WC warps work, one more brings the chunks' vectors into shared memory by bulk copies.  RI:
-// key channels in groups of 64.  A thread holds 4 RI rows and 2 columns of the state.
-template <int RI, int WC>
+// 4 WC J value columns of a head; 2 WC warps work, one more brings the chunks' vectors into shared memory by bulk copies.  RI:
+// key channels in groups of 64.  A thread holds 4 RI rows and J columns of the state.  (What the lanes read from shared memory
+// bounds the two products: wide tiles of few threads read less.)
+template <int RI, int WC, int J>
 __global__ void __launch_bounds__((2 * WC + 1) * 32, 1) scan_kernel(const __grid_constant__ HeadDeltaArgs a, int stages) {
     using namespace tc;
-    constexpr int N = 8 * WC, WORKERS = 2 * WC * 32;
+    constexpr int N = 4 * WC * J, WORKERS = 2 * WC * 32;
     pdl_launch_dependents();
     extern __shared__ __align__(16) float sm[];
     __shared__ __align__(8) uint64_t full[4], empty[4];
@@ -378,9 +379,9 @@ __global__ void __launch_bounds__((2 * WC + 1) * 32, 1) scan_kernel(const __grid
         }
     }
     const int wr = warp & 1, wc = warp >> 1, l8 = lane & 7, l4 = lane >> 3;
-    // This thread's part of the state: rows 4 (l8 + 8 wr + 16 i) .. + 3, columns c0, c0 + 1.
-    const int c0 = 2 * (l4 + 4 * wc);
-    float S[RI][4][2];
+    // This thread's part of the state: rows 4 (l8 + 8 wr + 16 i) .. + 3, columns c0 .. c0 + J - 1.
+    const int c0 = J * (l4 + 4 * wc);
+    float S[RI][4][J];
     float* st = a.state + ((size_t)a.slots[b] * H + h) * dk * dv;
     auto row_of = [&](int i) { return 4 * (l8 + 8 * wr + 16 * i); };
 #pragma unroll
@@ -388,7 +389,7 @@ __global__ void __launch_bounds__((2 * WC + 1) * 32, 1) scan_kernel(const __grid
 #pragma unroll
         for (int r = 0; r < 4; ++r)
 #pragma unroll
-            for (int c = 0; c < 2; ++c) {
+            for (int c = 0; c < J; ++c) {
                 const int row = row_of(i) + r, col = col0 + c0 + c;
                 S[i][r][c] = row < dk && col < dv ? st[(size_t)row * dv + col] : 0.f;
             }
@@ -397,7 +398,7 @@ __global__ void __launch_bounds__((2 * WC + 1) * 32, 1) scan_kernel(const __grid
         for (int i = 0; i < RI; ++i)
             if (row_of(i) < dk4)
 #pragma unroll
-                for (int c = 0; c < 2; ++c)
+                for (int c = 0; c < J; ++c)
                     *reinterpret_cast<float4*>(sT + (c0 + c) * ld + row_of(i)) = make_float4(S[i][0][c], S[i][1][c], S[i][2][c], S[i][3][c]);
     };
     share_state();
@@ -413,27 +414,33 @@ __global__ void __launch_bounds__((2 * WC + 1) * 32, 1) scan_kernel(const __grid
             for (int i = 0; i < RI; ++i)
 #pragma unroll
                 for (int r = 0; r < 4; ++r)
-                    if (row_of(i) + r < dk) *reinterpret_cast<float2*>(S0 + (size_t)(row_of(i) + r) * a.tiles * N) = make_float2(S[i][r][0], S[i][r][1]);
+                    if (row_of(i) + r < dk) {
+                        float* at = S0 + (size_t)(row_of(i) + r) * a.tiles * N;
+                        if constexpr (J == 4) *reinterpret_cast<float4*>(at) = make_float4(S[i][r][0], S[i][r][1], S[i][r][2], S[i][r][3]);
+                        else *reinterpret_cast<float2*>(at) = make_float2(S[i][r][0], S[i][r][1]);
+                    }
         }
         const unsigned bad = mbar_wait(smem_u32(&full[s]), (ch / stages) & 1) ? 0u : 1u;
         if (bad) give_up(2);
         // u = V' - W S_0: rows l8 + 8 wr + 16 i, columns l4 + 4 wc + 4 WC j.
-        f2 acc[4][2];
+        f2 acc[4][J];
 #pragma unroll
-        for (int i = 0; i < 4; ++i) acc[i][0] = acc[i][1] = 0ull;
+        for (int i = 0; i < 4; ++i)
+#pragma unroll
+            for (int j = 0; j < J; ++j) acc[i][j] = 0ull;
         const float* wp = w + (size_t)(l8 + 8 * wr) * ld;
         const float* sp = sT + (size_t)(l4 + 4 * wc) * ld;
 #pragma unroll 4
         for (int r = 0; r < dk4; r += 4) {
-            ulonglong2 x[4], y[2];
+            ulonglong2 x[4], y[J];
 #pragma unroll
             for (int i = 0; i < 4; ++i) x[i] = *reinterpret_cast<const ulonglong2*>(wp + 16 * i * ld + r);
 #pragma unroll
-            for (int j = 0; j < 2; ++j) y[j] = *reinterpret_cast<const ulonglong2*>(sp + 4 * WC * j * ld + r);
+            for (int j = 0; j < J; ++j) y[j] = *reinterpret_cast<const ulonglong2*>(sp + 4 * WC * j * ld + r);
 #pragma unroll
             for (int i = 0; i < 4; ++i)
 #pragma unroll
-                for (int j = 0; j < 2; ++j) {
+                for (int j = 0; j < J; ++j) {
                     acc[i][j] = fma2(x[i].x, y[j].x, acc[i][j]);
                     acc[i][j] = fma2(x[i].y, y[j].y, acc[i][j]);
                 }
@@ -442,7 +449,7 @@ __global__ void __launch_bounds__((2 * WC + 1) * 32, 1) scan_kernel(const __grid
 #pragma unroll
         for (int i = 0; i < 4; ++i)
 #pragma unroll
-            for (int j = 0; j < 2; ++j) {
+            for (int j = 0; j < J; ++j) {
                 const int t = l8 + 8 * wr + 16 * i, c = l4 + 4 * wc + 4 * WC * j;
                 const float2 f = unpack2(acc[i][j]);
                 const float u = v[t * N + c] - (f.x + f.y);
@@ -455,28 +462,35 @@ __global__ void __launch_bounds__((2 * WC + 1) * 32, 1) scan_kernel(const __grid
         if (any) break;                          // every worker leaves together
         // S_64 = S_0 + (e^l - 1) S_0 + sum_s k_s (u_s e^(l_64 - l_s))^T
         const float E = sc[2 * HC];
-        f2 A[RI][2][2];                          // rows in pairs
+        f2 A[RI][2][J];                          // rows in pairs
 #pragma unroll
         for (int i = 0; i < RI; ++i)
 #pragma unroll
             for (int p = 0; p < 2; ++p)
 #pragma unroll
-                for (int c = 0; c < 2; ++c)
+                for (int c = 0; c < J; ++c)
                     A[i][p][c] = pack2(fmaf(S[i][2 * p][c], E, S[i][2 * p][c]), fmaf(S[i][2 * p + 1][c], E, S[i][2 * p + 1][c]));
         const float* kp[RI];                     // rows behind the last key channel repeat the last ones and are not used
 #pragma unroll
         for (int i = 0; i < RI; ++i) kp[i] = k + min(row_of(i), dk4 - 4);
 #pragma unroll 8
         for (int t = 0; t < HC; ++t) {
-            const float2 u = *reinterpret_cast<const float2*>(us + t * N + c0);
-            const f2 u0 = pack2(u.x, u.x), u1 = pack2(u.y, u.y);
+            f2 u[J];
+            if constexpr (J == 4) {
+                const float4 f = *reinterpret_cast<const float4*>(us + t * N + c0);
+                u[0] = pack2(f.x, f.x); u[1] = pack2(f.y, f.y); u[2] = pack2(f.z, f.z); u[3] = pack2(f.w, f.w);
+            } else {
+                const float2 f = *reinterpret_cast<const float2*>(us + t * N + c0);
+                u[0] = pack2(f.x, f.x); u[1] = pack2(f.y, f.y);
+            }
 #pragma unroll
             for (int i = 0; i < RI; ++i) {
                 const ulonglong2 x = *reinterpret_cast<const ulonglong2*>(kp[i] + t * ld);
-                A[i][0][0] = fma2(x.x, u0, A[i][0][0]);
-                A[i][1][0] = fma2(x.y, u0, A[i][1][0]);
-                A[i][0][1] = fma2(x.x, u1, A[i][0][1]);
-                A[i][1][1] = fma2(x.y, u1, A[i][1][1]);
+#pragma unroll
+                for (int c = 0; c < J; ++c) {
+                    A[i][0][c] = fma2(x.x, u[c], A[i][0][c]);
+                    A[i][1][c] = fma2(x.y, u[c], A[i][1][c]);
+                }
             }
         }
 #pragma unroll
@@ -484,7 +498,7 @@ __global__ void __launch_bounds__((2 * WC + 1) * 32, 1) scan_kernel(const __grid
 #pragma unroll
             for (int p = 0; p < 2; ++p)
 #pragma unroll
-                for (int c = 0; c < 2; ++c) {
+                for (int c = 0; c < J; ++c) {
                     const float2 f = unpack2(A[i][p][c]);
                     S[i][2 * p][c] = f.x;
                     S[i][2 * p + 1][c] = f.y;
@@ -498,7 +512,7 @@ __global__ void __launch_bounds__((2 * WC + 1) * 32, 1) scan_kernel(const __grid
 #pragma unroll
         for (int r = 0; r < 4; ++r)
 #pragma unroll
-            for (int c = 0; c < 2; ++c) {
+            for (int c = 0; c < J; ++c) {
                 const int row = row_of(i) + r, col = col0 + c0 + c;
                 if (row < dk && col < dv) st[(size_t)row * dv + col] = S[i][r][c];
             }
@@ -650,14 +664,15 @@ template <int NT, int TM> int go_prepare(const HeadDeltaArgs& a, dim3 grid, cuda
     return launch_pdl(prepare_kernel<NT, TM>, grid, dim3(NT), smem, stream, a);
 }
 
-template <int RI, int WC> int go_scan(const HeadDeltaArgs& a, int B, cudaStream_t stream) {
-    const size_t stage = (size_t)(2 * HC * a.ld + HC * 8 * WC + SC) * sizeof(float), rest = (size_t)(8 * WC * a.ld + HC * 8 * WC) * sizeof(float);
+template <int RI, int WC, int J> int go_scan(const HeadDeltaArgs& a, int B, cudaStream_t stream) {
+    constexpr int N = 4 * WC * J;
+    const size_t stage = (size_t)(2 * HC * a.ld + HC * N + SC) * sizeof(float), rest = (size_t)(N * a.ld + HC * N) * sizeof(float);
     int stages = 3;
     while (stages > 1 && stages * stage + rest > MOST_SMEM) --stages;
     const size_t smem = stages * stage + rest;
     if (smem > MOST_SMEM) return LQ_BAD_SIZE;
-    if (!allow_smem(scan_kernel<RI, WC>, smem)) return lq_launch_status();
-    return launch_after(scan_kernel<RI, WC>, dim3(B, a.H, a.tiles), dim3((2 * WC + 1) * 32), smem, stream, a, stages);
+    if (!allow_smem(scan_kernel<RI, WC, J>, smem)) return lq_launch_status();
+    return launch_after(scan_kernel<RI, WC, J>, dim3(B, a.H, a.tiles), dim3((2 * WC + 1) * 32), smem, stream, a, stages);
 }
 
 template <typename TO, int CJ> int go_output(const HeadDeltaArgs& a, dim3 grid, cudaStream_t stream) {
@@ -704,7 +719,7 @@ LQ_EXPORT int lq_head_delta_prompt(const float* rows, int stride, int b_off, int
     int rc = dk + dv <= 160 ? go_prepare<128, 8>(a, grid, stream) : go_prepare<256, 4>(a, grid, stream);
     if (rc != LQ_OK) return rc;
     const int ri = (pad4(dk) + 63) / 64, cj = (a.tiles * n + 63) / 64;
-#define LQ_GO(RI) case RI: rc = n == 32 ? go_scan<RI, 4>(a, B, stream) : go_scan<RI, 2>(a, B, stream); break;
+#define LQ_GO(RI) case RI: rc = n == 32 ? go_scan<RI, RI <= 2 ? 2 : 4, RI <= 2 ? 4 : 2>(a, B, stream) : go_scan<RI, 2, 2>(a, B, stream); break;
     switch (ri) { LQ_GO(1) LQ_GO(2) LQ_GO(3) LQ_GO(4) default: rc = LQ_BAD_SIZE; }
 #undef LQ_GO
     if (rc != LQ_OK) return rc;
