@@ -71,8 +71,8 @@ __device__ __forceinline__ float tanh_fast(float x) {
     return fmaf(-2.0f, r, 1.0f);
 }
 
-// VD: a value head's size rounded up; its real size vd may be another than hd.
-template <int HD, int VD>
+// VD: a value head's size rounded up; its real size vd may be another than hd.  FAR: scores fall with the distance (slope).
+template <int HD, int VD, bool FAR>
 __global__ void __launch_bounds__(DW * 32, HD <= 64 && VD <= 64 ? 2 : 1)
 attn_decode_kernel(const __nv_bfloat16* __restrict__ q, int q_stride, const __nv_bfloat16* __restrict__ k_pages,
                    const __nv_bfloat16* __restrict__ v_pages, const int* __restrict__ page_table, int pt_stride,
@@ -205,7 +205,7 @@ attn_decode_kernel(const __nv_bfloat16* __restrict__ q, int q_stride, const __nv
     const int r0 = gt * 16 + g, r1 = r0 + 8;
     const bool r0ok = r0 < G, r1ok = r1 < G;
     // What the rows' scores lose per position of distance.
-    const float fall0 = (slope && r0ok) ? slope[kvh * G + r0] : 0.f, fall1 = (slope && r1ok) ? slope[kvh * G + r1] : 0.f;
+    const float fall0 = (FAR && r0ok) ? slope[kvh * G + r0] : 0.f, fall1 = (FAR && r1ok) ? slope[kvh * G + r1] : 0.f;
     const __nv_bfloat16* q0p = q + (size_t)tok * q_stride + (size_t)(kvh * G + (r0ok ? r0 : 0)) * hd;
     const __nv_bfloat16* q1p = q + (size_t)tok * q_stride + (size_t)(kvh * G + (r1ok ? r1 : 0)) * hd;
     uint32_t qf[KD][4];
@@ -261,7 +261,7 @@ attn_decode_kernel(const __nv_bfloat16* __restrict__ q, int q_stride, const __nv
                     a = softcap * tanh_fast(a * inv_cap);
                     b = softcap * tanh_fast(b * inv_cap);
                 }
-                if (slope) {
+                if constexpr (FAR) {
                     a = fmaf(fall0, (float)(key - pos), a);
                     b = fmaf(fall1, (float)(key - pos), b);
                 }
@@ -431,7 +431,7 @@ __global__ void attn_merge_kernel(const float* __restrict__ part_o, const float*
     }
 }
 
-template <int HD, int VD>
+template <int HD, int VD, bool FAR>
 int launch(const void* q, int q_stride, const void* k_pages, const void* v_pages, const int* page_table, int pt_stride,
            const int* tok_pos, const int* tok_seq, const int* slots, float* part_o, float* part_ml, int* counters,
            void* out, int T, int H, int Hkv, int hd, int page_size, float scale, int window, int n_splits,
@@ -449,11 +449,11 @@ int launch(const void* q, int q_stride, const void* k_pages, const void* v_pages
     constexpr size_t smem = ring > merge ? ring : merge;
     static bool configured = false;
     if (!configured) {
-        if (cudaFuncSetAttribute(attn_decode_kernel<HD, VD>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem) != cudaSuccess)
+        if (cudaFuncSetAttribute(attn_decode_kernel<HD, VD, FAR>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem) != cudaSuccess)
             return lq_launch_status();
         configured = true;
     }
-    int rc = launch_pdl(attn_decode_kernel<HD, VD>, grid, dim3(DW * 32), smem, stream, (const __nv_bfloat16*)q, q_stride,
+    int rc = launch_pdl(attn_decode_kernel<HD, VD, FAR>, grid, dim3(DW * 32), smem, stream, (const __nv_bfloat16*)q, q_stride,
         (const __nv_bfloat16*)k_pages, (const __nv_bfloat16*)v_pages, page_table, pt_stride, tok_pos, tok_seq, slots,
         part_o, part_ml, counters, (__nv_bfloat16*)out, H, Hkv, hd, page_size, scale, window, n_splits, n_splits, work,
         (const char*)next_w, (unsigned)piece, early_loads, sink, softcap, keep_first, vd, slope);
@@ -510,15 +510,17 @@ LQ_EXPORT int lq_attn_decode_vd(const void* q, int q_stride, const void* k_pages
     if (n_splits > 1 && (!part_o || !part_ml)) return LQ_BAD_SIZE;
     if (work && (teams < 1 || teams > 65535 || (n_splits > 1 && !counters))) return LQ_BAD_SIZE;
     if (softcap < 0.f || keep_first < 0) return LQ_BAD_SIZE;
-#define LQ_GO(HD, VD) return launch<HD, VD>(q, q_stride, k_pages, v_pages, page_table, pt_stride, tok_pos, tok_seq, slots, \
-                                            part_o, part_ml, counters, out, T, H, Hkv, hd, page_size, scale, window, n_splits, \
-                                            work, teams, next_w, next_bytes, early_loads, sink, softcap, keep_first, vd, slope, stream)
+#define LQ_GO(HD, VD) return slope ? launch<HD, VD, true> LQ_ARGS : launch<HD, VD, false> LQ_ARGS
+#define LQ_ARGS (q, q_stride, k_pages, v_pages, page_table, pt_stride, tok_pos, tok_seq, slots, \
+                part_o, part_ml, counters, out, T, H, Hkv, hd, page_size, scale, window, n_splits, \
+                work, teams, next_w, next_bytes, early_loads, sink, softcap, keep_first, vd, slope, stream)
     if (vd > 128) LQ_GO(128, 256);
     if (hd <= 32 && vd <= 32) LQ_GO(32, 32);
     if (hd <= 64 && vd <= 64) LQ_GO(64, 64);
     if (hd <= 64) LQ_GO(64, 128);
     LQ_GO(128, 128);
 #undef LQ_GO
+#undef LQ_ARGS
 }
 
 LQ_EXPORT int lq_attn_decode_capped(const void* q, int q_stride, const void* k_pages, const void* v_pages,
